@@ -118,7 +118,8 @@ class CacheManager:
     def __init__(self, needs: Sequence[object], cache_of: Sequence[Optional[int]], page_size: int,
                  num_pages: int, max_requests: int):
         """``needs[i]`` is what schedule entry ``i`` keeps (None if nothing or if it reads
-        ``cache_of[i]``'s cache); ``num_pages`` pages are given to every group."""
+        ``cache_of[i]``'s cache); needs beyond ``cache_of`` are those of parts that are no schedule entry (an embedding that
+        keeps a state) and own what they keep; ``num_pages`` pages are given to every group."""
         if page_size <= 0 or page_size > 64 or (page_size & (page_size - 1)) != 0:
             raise ValueError(f"page_size must be a power of two up to 64, got {page_size}")
         if num_pages <= 0:
@@ -133,7 +134,7 @@ class CacheManager:
         self.place: Dict[int, tuple] = {}
         self.state_needs: Dict[object, StateNeed] = {}
         self.state: Dict[object, torch.Tensor] = {}
-        self.cache_of = list(cache_of)
+        self.cache_of = list(cache_of) + [None] * (len(needs) - len(cache_of))
         by_need: Dict[PagedKV, int] = {}
 
         def put(need, key):
@@ -159,7 +160,8 @@ class CacheManager:
             if where is not None:
                 self.place[i] = where
         windows = (ctypes.c_int * max(1, len(self.groups)))(*[g.need.window if g.need.window else -1 for g in self.groups])
-        self._handle = self._lib.mbh_cache_create(self.page_size, self.num_pages, self.max_requests, len(self.groups), windows)
+        keeps = (ctypes.c_int * max(1, len(self.groups)))(*[g.need.keep_first if g.need.window else 0 for g in self.groups])
+        self._handle = self._lib.mbh_cache_create(self.page_size, self.num_pages, self.max_requests, len(self.groups), windows, keeps)
         if not self._handle:
             raise ValueError("the cache core refused these sizes")
         self.slots = SlotsView(self._lib, self._core, self.max_requests)

@@ -29,7 +29,7 @@ def host_lib() -> ctypes.CDLL:
         "mbh_pool_create": (vp, [i32]), "mbh_pool_destroy": (None, [vp]), "mbh_pool_num_free": (i32, [vp]),
         "mbh_pool_num_held": (i32, [vp]), "mbh_pool_alloc": (i32, [vp, i32, pi32]), "mbh_pool_free": (i32, [vp, i32]),
         "mbh_pool_check": (i32, [vp, text, i32]),
-        "mbh_cache_create": (vp, [i32, i32, i32, i32, pi32]), "mbh_cache_destroy": (None, [vp]),
+        "mbh_cache_create": (vp, [i32, i32, i32, i32, pi32, pi32]), "mbh_cache_destroy": (None, [vp]),
         "mbh_admit": (i32, [vp, pi64, pi32]), "mbh_length": (i32, [vp, i64]), "mbh_pages_missing": (i32, [vp, i64, i32, pi32]),
         "mbh_can_reserve": (i32, [vp, i32, pi64, pi32]), "mbh_reserve": (i32, [vp, i64, i32]), "mbh_commit": (i32, [vp, i64, i32]),
         "mbh_release": (i32, [vp, i64]), "mbh_block_table": (i32, [vp, i64, i32, pi32, i32]),

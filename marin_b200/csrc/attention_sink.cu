@@ -2,12 +2,14 @@
 //   * keys of `d` elements, values of `dv` (they may differ): K pages [page][kv_head][offset][d], V pages [..][dv];
 //   * which keys a position sees: all before it, the last `window`, or those of its own chunk of `chunk` positions
 //     (chunks counted from position 0 of the sequence, wherever a prompt was cut);
+//   * the sequence's first `keep` positions, visible however far behind the window or chunk they lie;
+//   * scores capped: s <- cap tanh(s / cap), the sink's score is not;
 //   * a sink: one more term in the softmax's denominator, a key without a value whose score is 0 or a learned number per
 //     query head (not scaled),  p_j = exp(s_j) / (exp(sink_h) + sum_j exp(s_j));
 //   * values that are the leading `dv` elements of the key rows (a latent shared by keys and values): the value pointer is
 //     the key pointer and `v_stride`, the distance between two positions' values, is the key rows' width;
 //   * an output gate: the result is multiplied element by element with sigmoid(g), g a column block of the fused
-//     projection.
+//     projection; and a plain factor `out_scale`.
 // This file holds the head preparation (biases, RMS norm of q and k per head or over the whole projection, partial
 // rotation with scaled sines and cosines, value mixing with the values an earlier layer left for the same tokens, cache
 // write) and the plain attention kernel that serves any size in both dtypes.  Sums, norms, angles, scores and weights
@@ -367,7 +369,7 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
     const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
     const int* __restrict__ block_table, int max_pages, const int* __restrict__ req_index, const int* __restrict__ positions,
     int H, int K, int d, int dv, int page_size, float scale, int window, int chunk, int sink, const float* __restrict__ sink_logit,
-    int v_stride, const T* __restrict__ gate, int gate_stride) {
+    int v_stride, const T* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride) {
     PDL_ENTER();
     q = pdl_fresh(q); k_cache = pdl_fresh(k_cache); v_cache = pdl_fresh(v_cache); gate = pdl_fresh(gate);
     extern __shared__ float smem[];
@@ -380,6 +382,8 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
     const int pos = positions[t];
     int lo = window > 0 ? max(0, pos - window + 1) : 0;
     if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
+    // the keys in order: the kept ones before lo, then lo .. pos; key number j is j or lo + j - kept
+    const int kept = min(keep, lo), keys = kept + pos - lo + 1;
     const int* table = block_table + (size_t)req * max_pages;
     const T* qrow = q + ((size_t)t * H + head) * d;
     for (int i = threadIdx.x; i < d; i += SK_THREADS) qs[i] = to_f32(qrow[i]);
@@ -392,33 +396,35 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
 #pragma unroll
     for (int r = 0; r < SK_MAX_PER_THREAD; ++r) acc[r] = 0.0f;
 
-    for (int base = lo; base <= pos; base += SK_THREADS) {
-        const int key = base + threadIdx.x;
+    for (int base = 0; base < keys; base += SK_THREADS) {
+        const int at = base + threadIdx.x;
         float s = -INFINITY;
-        if (key <= pos) {
+        if (at < keys) {
+            const int key = at < kept ? at : lo + at - kept;
             const size_t page = (size_t)table[key / page_size];
             const T* krow = k_cache + ((page * K + kh) * page_size + (size_t)(key % page_size)) * d;
             float dot = 0.0f;
             for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_f32(krow[i]), dot);
             s = dot * scale;
+            if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
         }
         const float block_top = block_max(s, scratch);
         const float m_new = fmaxf(m, block_top);
         const float corr = expf(m - m_new);   // exp(-inf) = 0 on the first block without a sink
-        const float p = key <= pos ? expf(s - m_new) : 0.0f;
+        const float p = at < keys ? expf(s - m_new) : 0.0f;
         __syncthreads();
         ps[threadIdx.x] = p;
         const float block_total = block_sum(p, scratch);  // has the barriers that publish ps
         l = l * corr + block_total;
         m = m_new;
-        const int count = min(SK_THREADS, pos - base + 1);
+        const int count = min(SK_THREADS, keys - base);
 #pragma unroll
         for (int r = 0; r < SK_MAX_PER_THREAD; ++r) {
             const int dd = threadIdx.x + r * SK_THREADS;
             if (dd < dv) {
                 float a = acc[r] * corr;
                 for (int j = 0; j < count; ++j) {
-                    const int kj = base + j;
+                    const int kj = base + j < kept ? base + j : lo + base + j - kept;
                     const size_t page = (size_t)table[kj / page_size];
                     const T* vrow = v_cache + ((page * K + kh) * page_size + (size_t)(kj % page_size)) * v_stride;
                     a = fmaf(ps[j], to_f32(vrow[dd]), a);
@@ -428,13 +434,13 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
         }
         __syncthreads();
     }
-    T* orow = out + ((size_t)t * H + head) * dv;
+    T* orow = out + (size_t)t * out_stride + (size_t)head * dv;
     const T* grow = gate != nullptr ? gate + (size_t)t * gate_stride + (size_t)head * dv : nullptr;
 #pragma unroll
     for (int r = 0; r < SK_MAX_PER_THREAD; ++r) {
         const int dd = threadIdx.x + r * SK_THREADS;
         if (dd < dv) {
-            float o = acc[r] / l;
+            float o = acc[r] / l * out_scale;
             if (grow != nullptr) o *= 1.0f / (1.0f + expf(-to_f32(grow[dd])));
             orow[dd] = from_f32<T>(o);
         }
@@ -444,12 +450,13 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
 // gate: null, or the first gate column of token 0 (rows `gate_stride` elements apart, H heads of dv side by side).
 // sink_logit: null (a sink of score 0, if `sink`) or a float32 score per query head.  v_stride: elements between the values of
 // two positions of a page (dv for value pages of their own; the key rows' width where values are the start of the key rows).
+// keep: first positions that are always seen; softcap 0: scores are not capped; out rows are out_stride elements apart.
 MB_API int mb_attention_sink(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype, const int* block_table,
                              int max_pages, const int* req_index, const int* positions, int tokens, int H, int K, int d, int dv,
                              int page_size, float scale, int window, int chunk, int sink, const float* sink_logit, int v_stride,
-                             const void* gate, int gate_stride, cudaStream_t s) {
+                             const void* gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
     if (tokens <= 0) return 0;
-    if (v_stride < dv) return MB_ERR_BAD_SIZE;
+    if (v_stride < dv || keep < 0 || softcap < 0.0f || out_stride < H * dv) return MB_ERR_BAD_SIZE;
     if (d <= 0 || dv <= 0 || dv > SK_THREADS * SK_MAX_PER_THREAD || K <= 0 || H % K != 0 || window < 0 || chunk < 0) return MB_ERR_BAD_SIZE;
     dim3 grid(tokens, H);
     const size_t smem = (size_t)(d + SK_THREADS + 32) * sizeof(float);
@@ -457,10 +464,10 @@ MB_API int mb_attention_sink(const void* q, const void* k_cache, const void* v_c
     if (dtype == MB_F32)
         return launch_kernel(attention_sink_kernel<float>, grid, SK_THREADS, smem, s, 0, (const float*)q, (const float*)k_cache,
                              (const float*)v_cache, (float*)out, block_table, max_pages, req_index, positions, H, K, d, dv, page_size,
-                             scale, window, chunk, sink, sink_logit, v_stride, (const float*)gate, gate_stride);
+                             scale, window, chunk, sink, sink_logit, v_stride, (const float*)gate, gate_stride, keep, softcap, out_scale, out_stride);
     if (dtype == MB_BF16)
         return launch_kernel(attention_sink_kernel<bf16>, grid, SK_THREADS, smem, s, 0, (const bf16*)q, (const bf16*)k_cache,
                              (const bf16*)v_cache, (bf16*)out, block_table, max_pages, req_index, positions, H, K, d, dv, page_size,
-                             scale, window, chunk, sink, sink_logit, v_stride, (const bf16*)gate, gate_stride);
+                             scale, window, chunk, sink, sink_logit, v_stride, (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
     return MB_ERR_BAD_DTYPE;
 }

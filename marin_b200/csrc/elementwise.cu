@@ -34,6 +34,61 @@ MB_API int mb_embed(const int* ids, const void* table, int table_dtype, const vo
     return mb_last_error();
 }
 
+// ---- token embedding plus a bigram embedding ----------------------------------------------------------------------------
+// out[t, :] = float(table[ids[t], :]) * scale + float(pairs[r, :]), r = (before * mul_before + ids[t] * mul_now) mod buckets with
+// `before` the token ahead in the same sequence, or row `buckets` (the last) for a sequence's first token.  The token ahead of a
+// request's first token of the step is what its state keeps (last: int32 [slot]).  `store`: every request brings one token and
+// its block also keeps it; otherwise last_token_kernel does, once all blocks have read.
+template <typename TW>
+__global__ void embed_bigram_kernel(const int* __restrict__ ids, const TW* __restrict__ table, const TW* __restrict__ pairs,
+                                    const int* __restrict__ positions, const int* __restrict__ req_index, const int* __restrict__ cu_tokens,
+                                    const int* __restrict__ slots, int* last, float* __restrict__ out, int h, float scale, long long mul_before,
+                                    long long mul_now, int buckets, int store) {
+    PDL_ENTER();
+    ids = pdl_fresh(ids); last = pdl_fresh(last);
+    const int t = blockIdx.x;
+    const int req = req_index[t], id = ids[t];
+    int* kept = last + slots[req];
+    long long at = buckets;
+    if (positions[t] > 0) at = ((long long)(t > cu_tokens[req] ? ids[t - 1] : *kept) * mul_before + (long long)id * mul_now) % buckets;
+    if (store) {
+        __syncthreads();                                       // every thread has read the token ahead
+        if (threadIdx.x == 0) *kept = id;
+    }
+    const TW* row = table + (size_t)id * h;
+    const TW* pair = pairs + (size_t)at * h;
+    float* dst = out + (size_t)t * h;
+    for (int i = threadIdx.x; i < h; i += blockDim.x) dst[i] = to_f32(row[i]) * scale + to_f32(pair[i]);
+}
+
+__global__ void last_token_kernel(const int* __restrict__ ids, const int* __restrict__ cu_tokens, const int* __restrict__ slots,
+                                  int* __restrict__ last, int requests) {
+    PDL_ENTER();
+    ids = pdl_fresh(ids);
+    const int r = blockIdx.x * blockDim.x + threadIdx.x;
+    if (r < requests && cu_tokens[r + 1] > cu_tokens[r]) last[slots[r]] = ids[cu_tokens[r + 1] - 1];
+}
+
+MB_API int mb_embed_bigram(const int* ids, const void* table, const void* pairs, int table_dtype, const int* positions, const int* req_index,
+                           const int* cu_tokens, const int* slots, int* last, float* out, int tokens, int requests, int h, float scale,
+                           long long mul_before, long long mul_now, int buckets, int store, cudaStream_t s) {
+    if (tokens <= 0) return 0;
+    if (buckets <= 0 || mul_before < 0 || mul_now < 0) return MB_ERR_BAD_SIZE;
+    int rc = MB_ERR_BAD_DTYPE;
+    if (table_dtype == MB_F32)
+        rc = launch_kernel(embed_bigram_kernel<float>, tokens, 256, 0, s, 0, ids, (const float*)table, (const float*)pairs, positions, req_index,
+                           cu_tokens, slots, last, out, h, scale, mul_before, mul_now, buckets, store);
+    else if (table_dtype == MB_BF16)
+        rc = launch_kernel(embed_bigram_kernel<bf16>, tokens, 256, 0, s, 0, ids, (const bf16*)table, (const bf16*)pairs, positions, req_index,
+                           cu_tokens, slots, last, out, h, scale, mul_before, mul_now, buckets, store);
+    return rc;
+}
+
+MB_API int mb_last_token(const int* ids, const int* cu_tokens, const int* slots, int* last, int requests, cudaStream_t s) {
+    if (requests <= 0) return 0;
+    return launch_kernel(last_token_kernel, (requests + 127) / 128, 128, 0, s, 0, ids, cu_tokens, slots, last, requests);
+}
+
 // ---- RMSNorm over rows of a float32 matrix ---------------------------------------------------------
 template <typename TO>
 __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, int unit_offset,
@@ -295,9 +350,9 @@ MB_API int mb_qk_norm_rope_write(const void* qkv, int dtype, void* q_out, const 
 }
 
 // ---- SwiGLU: out[t, i] = g / (1 + exp(-g)) * u with g = gu[t, i], u = gu[t, I + i]; or, interleaved, with gate and
-// up in alternating blocks of 16 columns: g = gu[t, 32 (i / 16) + i % 16], u = 16 columns further -----------------
+// up in alternating blocks of 16 columns: g = gu[t, 32 (i / 16) + i % 16], u = 16 columns further.  act 1: max(g, 0) * u ----
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t total, int interleaved) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t total, int interleaved, int act) {
     PDL_ENTER();
     gu = pdl_fresh(gu);
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -307,7 +362,7 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const size_t gi = interleaved ? (i >> 4) * 32 + (i & 15) : i;
         const size_t ui = interleaved ? gi + 16 : I + i;
         const float g = to_f32(gu[t * 2 * I + gi]), u = to_f32(gu[t * 2 * I + ui]);
-        out[idx] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+        out[idx] = from_f32<T>((act == 1 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g))) * u);
     }
 }
 
@@ -330,13 +385,13 @@ MB_API int mb_rope_table(const int* positions, const float* inv_freq, int half, 
     return launch_kernel(rope_table_kernel, dim3((total + 255) / 256), dim3(256), 0, s, 0, positions, inv_freq, half, out, T);
 }
 
-MB_API int mb_swiglu(const void* gate_up, void* out, int dtype, int tokens, int I, int interleaved, cudaStream_t s) {
+MB_API int mb_swiglu(const void* gate_up, void* out, int dtype, int tokens, int I, int interleaved, int act, cudaStream_t s) {
     const size_t total = (size_t)tokens * I;
     if (total == 0) return 0;
     const int threads = 256;
     const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
-    if (dtype == MB_F32) return launch_kernel(swiglu_kernel<float>, blocks, threads, 0, s, 0, (const float*)gate_up, (float*)out, I, total, interleaved);
-    else if (dtype == MB_BF16) return launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, s, 0, (const bf16*)gate_up, (bf16*)out, I, total, interleaved);
+    if (dtype == MB_F32) return launch_kernel(swiglu_kernel<float>, blocks, threads, 0, s, 0, (const float*)gate_up, (float*)out, I, total, interleaved, act);
+    else if (dtype == MB_BF16) return launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, s, 0, (const bf16*)gate_up, (bf16*)out, I, total, interleaved, act);
     else return MB_ERR_BAD_DTYPE;
     return mb_last_error();
 }

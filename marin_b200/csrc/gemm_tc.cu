@@ -554,8 +554,8 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
         }
         if (direct && norm.weight != nullptr) {
             store_chunk_norm(out, t0 + c0, n, n < N, T, N, v, norm, norm.sumsq + (size_t)(blockIdx.x * 4 + warp) * T, lane);
-        } else if (direct && mode == TC_OUT_SWIGLU) {
-            if (n0 + warp * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + warp * 32, lane, T, N, v);
+        } else if (direct && (mode == TC_OUT_SWIGLU || mode == TC_OUT_REGLU)) {
+            if (n0 + warp * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + warp * 32, lane, T, N, v, mode == TC_OUT_REGLU);
         } else if (n < N) {
             if (direct) store_chunk(out, mode, t0 + c0, n, T, N, v);
             else {
@@ -930,8 +930,8 @@ __global__ void __launch_bounds__(320) gemm_tc_persistent_kernel(const __grid_co
                 }
                 if (norm.weight != nullptr) {
                     store_chunk_norm(out, t0 + c0, n, n < N, T, N, v, norm, norm.sumsq + (size_t)(tile_row * 4 + quarter) * T, lane);
-                } else if (mode == TC_OUT_SWIGLU) {
-                    if (n0 + quarter * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + quarter * 32, lane, T, N, v);
+                } else if (mode == TC_OUT_SWIGLU || mode == TC_OUT_REGLU) {
+                    if (n0 + quarter * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + quarter * 32, lane, T, N, v, mode == TC_OUT_REGLU);
                 } else if (reduce_out) {
                     // "+=" into float32 without reading the old values: the four warps that share this half of the columns
                     // lay sixteen tokens of the tile into shared memory and one thread hands them to a TMA reduction
@@ -1126,7 +1126,7 @@ static int persistent_dispatch(const void* x, const void* w, void* out, int mode
                                const TcHeadsOut& heads = TcHeadsOut{}, const float* rope = nullptr) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ctas <= 0) return MB_ERR_BAD_SIZE;
-    if (mode < 0 || mode > 4 || (mode == 3 && N % 32 != 0)) return MB_ERR_BAD_DTYPE;
+    if (mode < 0 || mode > 5 || ((mode == 3 || mode == 5) && N % 32 != 0)) return MB_ERR_BAD_DTYPE;
     if (norm.weight != nullptr && (mode != TC_OUT_F32_ACC || norm.scaled == nullptr || norm.sumsq == nullptr)) return MB_ERR_BAD_DTYPE;
     if (scale.sumsq != nullptr && (scale.slots <= 0 || scale.dim <= 0)) return MB_ERR_BAD_SIZE;
     CUtensorMap mw, mx;
@@ -1227,7 +1227,7 @@ static int gemm_tc_dispatch(const void* x, const void* w, void* out, int mode, i
     if (norm.weight != nullptr && !cluster_reduce && splits > 1) return MB_ERR_BAD_SIZE;
     if (scale.sumsq != nullptr && (scale.slots <= 0 || scale.dim <= 0 || (!cluster_reduce && splits > 1))) return MB_ERR_BAD_SIZE;
     if (K <= 0 || K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return MB_ERR_BAD_SIZE;
-    if (mode < 0 || mode > 4 || (mode == 3 && (splits > 1 || N % 32 != 0))) return MB_ERR_BAD_DTYPE;
+    if (mode < 0 || mode > 5 || ((mode == 3 || mode == 5) && (splits > 1 || N % 32 != 0))) return MB_ERR_BAD_DTYPE;
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     if (splits < 1) splits = 1;
     if (splits > total_kb) splits = total_kb;

@@ -40,10 +40,12 @@ MBH_API int mbh_pool_check(void* p, char* msg, int cap) {
 }
 
 // ---- the cache manager ----------------------------------------------------------------------------------------------
-// windows[g] < 0: group g keeps all keys.
-MBH_API void* mbh_cache_create(int page_size, int num_pages, int max_requests, int n_groups, const int* windows) {
+// windows[g] < 0: group g keeps all keys.  keeps[g]: its first positions whose pages a window never gives back (0: none).
+MBH_API void* mbh_cache_create(int page_size, int num_pages, int max_requests, int n_groups, const int* windows, const int* keeps) {
     if (page_size <= 0 || num_pages <= 0 || max_requests <= 0 || n_groups < 0) return nullptr;
-    return new Cache(page_size, num_pages, max_requests, n_groups, windows);
+    for (int g = 0; g < n_groups; ++g)
+        if (keeps[g] < 0) return nullptr;
+    return new Cache(page_size, num_pages, max_requests, n_groups, windows, keeps);
 }
 MBH_API void mbh_cache_destroy(void* c) { delete static_cast<Cache*>(c); }
 MBH_API int mbh_admit(void* c, int64_t* handle, int* slot) { return static_cast<Cache*>(c)->admit(handle, slot); }

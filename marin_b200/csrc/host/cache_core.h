@@ -86,10 +86,12 @@ struct Request {
 
 class Cache {
   public:
-    Cache(int page_size, int num_pages, int max_requests, int n_groups, const int* windows)
+    // windows[g]: the latest positions group g keeps (-1: all); keeps[g]: its first positions that stay however old they are
+    Cache(int page_size, int num_pages, int max_requests, int n_groups, const int* windows, const int* keeps)
         : page_size_(page_size), slots_(max_requests) {
         for (int g = 0; g < n_groups; ++g) {
             windows_.push_back(windows[g]);
+            kept_pages_.push_back((keeps[g] + page_size - 1) / page_size);
             pools_.emplace_back(num_pages);
         }
     }
@@ -127,7 +129,8 @@ class Cache {
         for (size_t g = 0; g < pools_.size(); ++g) pools_[g].alloc(need[g], &r.pages[g]);
         return MBH_OK;
     }
-    // The step succeeded: the request holds new_len positions; pages a window has passed go back to their pool.
+    // The step succeeded: the request holds new_len positions; pages a window has passed go back to their pool, all but
+    // those that hold the first positions a group keeps for good.
     int commit(Request& r, int new_len) {
         if (new_len < r.length) return MBH_BAD_ARG;
         r.length = new_len;
@@ -135,7 +138,7 @@ class Cache {
             if (windows_[g] < 0) continue;
             const int first = std::max(0, new_len - windows_[g] + 1) / page_size_;   // the next token's first needed page
             std::vector<int>& table = r.pages[g];
-            for (int logical = 0; logical < std::min(first, (int)table.size()); ++logical) {
+            for (int logical = kept_pages_[g]; logical < std::min(first, (int)table.size()); ++logical) {
                 if (table[logical] != DROPPED) {
                     const int rc = pools_[g].free_page(table[logical]);
                     if (rc != MBH_OK) return rc;
@@ -190,6 +193,7 @@ class Cache {
   private:
     int page_size_;
     std::vector<int> windows_;               // per group, -1: all keys are kept
+    std::vector<int> kept_pages_;            // per group: how many pages from the sequence's start are never given back
     std::vector<PagePool> pools_;
     PagePool slots_;
     std::unordered_map<int64_t, Request> reqs_;

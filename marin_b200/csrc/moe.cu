@@ -5,7 +5,11 @@
 // The gated form is g sigmoid(alpha g) (u + shift) with g = gate x and u = up x, both capped where `act_limit` > 0
 // (g <- min(g, limit), u <- clamp(u, -limit, limit)); alpha 1, shift 0 and no limit is silu(gate x) * (up x).
 //   * router: z = W_r h in float32, score = sigmoid(z) or the softmax of z over the experts; the chosen experts' scores are
-//     the weights, renormalised to sum 1 over the chosen ones if asked;
+//     the weights, renormalised to sum 1 over the chosen ones if asked, times a factor;
+//   * the choice may see more than the scores: a correction per expert is added for it (the weights stay without), and where
+//     the experts form groups of neighbours only those of the best `keep` groups (by their largest choice score) can be chosen;
+//   * the router may have more outputs than there are experts: the last ones stand for the identity (a pair's result is the
+//     input itself times its weight, no matrix is read);
 //   * the weight multiplies the expert's input (x = w h, the activation sees it) or its output (x = h, result times w).
 // Kernels: the router with its top-k (a warp per token), the grouping of (token, choice) pairs by expert (offsets and an
 // order), and the plain expert products for any size in both dtypes (a pair per block).  A pair's result never depends on
@@ -32,12 +36,15 @@ __host__ __device__ __forceinline__ int gate_up_row(int c, int which, int ff, in
 template <typename T>
 __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T* __restrict__ h_rows, const float* __restrict__ router,
                                                                const float* __restrict__ router_bias, int* __restrict__ expert_out, float* __restrict__ weight_out,
-                                                               int tokens, int h, int E, int top, int score_mode, int renorm) {
+                                                               int tokens, int h, int E, int top, int score_mode, int renorm,
+                                                               const float* __restrict__ correction, int groups, int keep, float factor) {
     PDL_ENTER();
     h_rows = pdl_fresh(h_rows);
     extern __shared__ float smem[];
     float* xrow = smem;                        // [h] (first: 16-byte aligned)
-    float* z = smem + h;                       // [E]
+    float* z = smem + h;                       // [E]: logits, and what the choice goes by
+    float* score_of = z + E;                   // [E] (with a correction)
+    float* group_top = score_of + E;           // [groups]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
     const T* x = h_rows + (size_t)t * h;
@@ -85,6 +92,30 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T* __restri
         for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
         denom = warp_sum(sum);
     }
+    if (correction != nullptr) {                               // the choice goes by score + correction, the weights by the score
+        for (int e = lane; e < E; e += 32) {
+            const float s = score_mode == 1 ? expf(z[e] - zmax) / denom : 1.0f / (1.0f + expf(-z[e]));
+            score_of[e] = s;
+            z[e] = s + correction[e];
+        }
+        __syncwarp();
+    }
+    if (keep < groups) {                                       // what lies outside the best groups cannot be chosen
+        const int per = E / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float mx = -INFINITY;
+            for (int e = g * per; e < (g + 1) * per; ++e) mx = fmaxf(mx, z[e]);
+            group_top[g] = mx;
+        }
+        __syncwarp();
+        for (int g = lane; g < groups; g += 32) {              // a group's rank: how many come before it (the lower group among equals)
+            int ahead = 0;
+            for (int o = 0; o < groups; ++o) ahead += group_top[o] > group_top[g] || (group_top[o] == group_top[g] && o < g);
+            if (ahead >= keep)
+                for (int e = g * per; e < (g + 1) * per; ++e) z[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
     float chosen_sum = 0.0f;
     for (int c = 0; c < top; ++c) {
         float best = -INFINITY;
@@ -100,7 +131,7 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T* __restri
             if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
         }
         if (at >= E) at = c;                                   // logits that are not numbers order nothing: stay inside the table
-        const float score = score_mode == 1 ? expf(best - zmax) / denom : 1.0f / (1.0f + expf(-best));
+        const float score = correction != nullptr ? score_of[at] : score_mode == 1 ? expf(best - zmax) / denom : 1.0f / (1.0f + expf(-best));
         chosen_sum += score;
         if (lane == 0) {
             expert_out[(size_t)t * top + c] = at;
@@ -109,22 +140,27 @@ __global__ void __launch_bounds__(MR_THREADS) moe_route_kernel(const T* __restri
         }
         __syncwarp();
     }
-    if (renorm && lane == 0)
-        for (int c = 0; c < top; ++c) weight_out[(size_t)t * top + c] /= chosen_sum;
+    if ((renorm || factor != 1.0f) && lane == 0)
+        for (int c = 0; c < top; ++c) {
+            const float w = weight_out[(size_t)t * top + c];
+            weight_out[(size_t)t * top + c] = (renorm ? w / (chosen_sum + 1e-20f) : w) * factor;
+        }
 }
 
+// E: all outputs of the router (identity outputs included).  groups 1: no groups; correction null: none; factor: on the weights.
 MB_API int mb_moe_route(const void* h_rows, int dtype, const float* router, const float* router_bias, int* expert_out, float* weight_out, int tokens, int h,
-                        int E, int top, int score_mode, int renorm, cudaStream_t s) {
+                        int E, int top, int score_mode, int renorm, const float* correction, int groups, int keep, float factor, cudaStream_t s) {
     if (tokens <= 0) return 0;
     if (E <= 0 || top <= 0 || top > E || h <= 0 || score_mode < 0 || score_mode > 1) return MB_ERR_BAD_SIZE;
-    const size_t smem = (size_t)(E + h) * sizeof(float);
+    if (groups <= 0 || E % groups != 0 || keep <= 0 || keep > groups || (keep < groups && top > E / groups * keep)) return MB_ERR_BAD_SIZE;
+    const size_t smem = (size_t)(2 * E + groups + h) * sizeof(float);
     if (smem > 48 * 1024) return MB_ERR_BAD_SIZE;
     if (dtype == MB_F32)
         return launch_kernel(moe_route_kernel<float>, tokens, MR_THREADS, smem, s, 0, (const float*)h_rows, router, router_bias, expert_out,
-                             weight_out, tokens, h, E, top, score_mode, renorm);
+                             weight_out, tokens, h, E, top, score_mode, renorm, correction, groups, keep, factor);
     if (dtype == MB_BF16)
         return launch_kernel(moe_route_kernel<bf16>, tokens, MR_THREADS, smem, s, 0, (const bf16*)h_rows, router, router_bias, expert_out,
-                             weight_out, tokens, h, E, top, score_mode, renorm);
+                             weight_out, tokens, h, E, top, score_mode, renorm, correction, groups, keep, factor);
     return MB_ERR_BAD_DTYPE;
 }
 
@@ -188,13 +224,14 @@ __global__ void __launch_bounds__(ME_THREADS) moe_gate_up_kernel(const T* __rest
                                                                  const int* __restrict__ expert_of, const float* __restrict__ weight_of,
                                                                  T* __restrict__ act, int h, int ff, int top, int weight_on_input,
                                                                  int interleaved, int act_mode, float act_limit, float act_alpha,
-                                                                 float act_shift) {
+                                                                 float act_shift, int E) {
     PDL_ENTER();
     h_rows = pdl_fresh(h_rows); expert_of = pdl_fresh(expert_of); weight_of = pdl_fresh(weight_of);
     extern __shared__ float x[];               // [h]
     const int p = blockIdx.x;
     const int token = p / top;
     const int e = expert_of[p];
+    if (e >= E) return;                                        // the identity: no matrix
     const float wgt = weight_on_input ? weight_of[p] : 1.0f;
     for (int i = threadIdx.x; i < h; i += ME_THREADS) x[i] = to_f32(from_f32<T>(to_f32(h_rows[(size_t)token * h + i]) * wgt));
     __syncthreads();
@@ -228,8 +265,10 @@ __global__ void __launch_bounds__(ME_THREADS) moe_gate_up_kernel(const T* __rest
 template <typename T>
 __global__ void __launch_bounds__(ME_THREADS) moe_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down,
                                                               const int* __restrict__ expert_of, const float* __restrict__ weight_of,
-                                                              float* __restrict__ y, int h, int ff, int top, int weight_on_input) {
+                                                              float* __restrict__ y, int h, int ff, int top, int weight_on_input,
+                                                              const T* __restrict__ h_rows, int E) {
     PDL_ENTER();
+    h_rows = pdl_fresh(h_rows);
     act = pdl_fresh(act); expert_of = pdl_fresh(expert_of); weight_of = pdl_fresh(weight_of); y = pdl_fresh(y);
     extern __shared__ float a[];               // [ff]
     const int token = blockIdx.x;
@@ -238,6 +277,12 @@ __global__ void __launch_bounds__(ME_THREADS) moe_down_kernel(const T* __restric
         const int p = token * top + c;
         const int e = expert_of[p];
         const float wgt = weight_on_input ? 1.0f : weight_of[p];
+        if (e >= E) {                                          // the identity: the input times the weight
+            __syncthreads();
+            for (int col = threadIdx.x; col < h; col += ME_THREADS) y[(size_t)token * h + col] += to_f32(h_rows[(size_t)token * h + col]) * weight_of[p];
+            __syncthreads();
+            continue;
+        }
         __syncthreads();
         for (int i = threadIdx.x; i < ff; i += ME_THREADS) a[i] = to_f32(act[(size_t)p * ff + i]);
         __syncthreads();
@@ -255,22 +300,22 @@ __global__ void __launch_bounds__(ME_THREADS) moe_down_kernel(const T* __restric
 // which = 0: act <- the activations of every pair; which = 1: y += the chosen experts' outputs, from act.
 MB_API int mb_moe_experts_plain(const void* h_rows, int dtype, const void* w_gate_up, const void* w_down, const int* expert_of,
                                 const float* weight_of, void* act, float* y, int tokens, int h, int ff, int top, int weight_on_input,
-                                int interleaved, int which, int act_mode, float act_limit, float act_alpha, float act_shift, cudaStream_t s) {
+                                int interleaved, int which, int act_mode, float act_limit, float act_alpha, float act_shift, int E, cudaStream_t s) {
     if (tokens <= 0) return 0;
     if (h <= 0 || ff <= 0 || top <= 0 || (size_t)h * 4 > 48 * 1024 || (size_t)ff * 4 > 48 * 1024) return MB_ERR_BAD_SIZE;
     if (dtype == MB_F32) {
         if (which == 0)
             return launch_kernel(moe_gate_up_kernel<float>, tokens * top, ME_THREADS, (size_t)h * 4, s, 0, (const float*)h_rows,
-                                 (const float*)w_gate_up, expert_of, weight_of, (float*)act, h, ff, top, weight_on_input, interleaved, act_mode, act_limit, act_alpha, act_shift);
+                                 (const float*)w_gate_up, expert_of, weight_of, (float*)act, h, ff, top, weight_on_input, interleaved, act_mode, act_limit, act_alpha, act_shift, E);
         return launch_kernel(moe_down_kernel<float>, tokens, ME_THREADS, (size_t)ff * 4, s, 0, (const float*)act, (const float*)w_down,
-                             expert_of, weight_of, y, h, ff, top, weight_on_input);
+                             expert_of, weight_of, y, h, ff, top, weight_on_input, (const float*)h_rows, E);
     }
     if (dtype == MB_BF16) {
         if (which == 0)
             return launch_kernel(moe_gate_up_kernel<bf16>, tokens * top, ME_THREADS, (size_t)h * 4, s, 0, (const bf16*)h_rows,
-                                 (const bf16*)w_gate_up, expert_of, weight_of, (bf16*)act, h, ff, top, weight_on_input, interleaved, act_mode, act_limit, act_alpha, act_shift);
+                                 (const bf16*)w_gate_up, expert_of, weight_of, (bf16*)act, h, ff, top, weight_on_input, interleaved, act_mode, act_limit, act_alpha, act_shift, E);
         return launch_kernel(moe_down_kernel<bf16>, tokens, ME_THREADS, (size_t)ff * 4, s, 0, (const bf16*)act, (const bf16*)w_down,
-                             expert_of, weight_of, y, h, ff, top, weight_on_input);
+                             expert_of, weight_of, y, h, ff, top, weight_on_input, (const bf16*)h_rows, E);
     }
     return MB_ERR_BAD_DTYPE;
 }
@@ -453,15 +498,22 @@ __global__ void __launch_bounds__(128) moe_grouped_kernel(const bf16* __restrict
     }
 }
 
-// y[t][c] += sum over the token's choices, in choice order, of rows[inv[t top + choice]][c] (times the choice's weight, if given)
+// y[t][c] += sum over the token's choices, in choice order, of rows[inv[t top + choice]][c] (times the choice's weight, if given);
+// a choice numbered E or above is the identity: its row is h_rows[t] times identity_weight
 __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ inv, const float* __restrict__ weight_of,
-                                   float* __restrict__ y, int h, int top) {
+                                   float* __restrict__ y, int h, int top, const int* __restrict__ expert_of, const bf16* __restrict__ h_rows,
+                                   const float* __restrict__ identity_weight, int E) {
     PDL_ENTER();
     rows = pdl_fresh(rows); inv = pdl_fresh(inv); y = pdl_fresh(y); weight_of = pdl_fresh(weight_of);
+    expert_of = pdl_fresh(expert_of); h_rows = pdl_fresh(h_rows); identity_weight = pdl_fresh(identity_weight);
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < h; c += blockDim.x) {
         float a = y[(size_t)t * h + c];
         for (int k = 0; k < top; ++k) {
+            if (h_rows != nullptr && expert_of[t * top + k] >= E) {
+                a += identity_weight[t * top + k] * __bfloat162float(h_rows[(size_t)t * h + c]);
+                continue;
+            }
             const float v = rows[(size_t)inv[t * top + k] * h + c];
             a += weight_of != nullptr ? v * weight_of[t * top + k] : v;
         }
@@ -527,7 +579,9 @@ MB_API int mb_moe_grouped_down(const void* act, const void* w_down, const int* o
     return grouped_by_rows<1>((const bf16*)act, (const bf16*)w_down, offsets, E, h, ff, nullptr, out, dst_rows, row_scale, accumulate, 0, pairs, s);
 }
 
-MB_API int mb_moe_combine(const float* rows, const int* inv, const float* weight_of, float* y, int tokens, int h, int top, cudaStream_t s) {
+// h_rows null: no identity choices (expert_of, identity_weight and E are not read).
+MB_API int mb_moe_combine(const float* rows, const int* inv, const float* weight_of, float* y, int tokens, int h, int top, const int* expert_of,
+                          const void* h_rows, const float* identity_weight, int E, cudaStream_t s) {
     if (tokens <= 0) return 0;
-    return launch_kernel(moe_combine_kernel, tokens, 256, 0, s, 0, rows, inv, weight_of, y, h, top);
+    return launch_kernel(moe_combine_kernel, tokens, 256, 0, s, 0, rows, inv, weight_of, y, h, top, expert_of, (const bf16*)h_rows, identity_weight, E);
 }

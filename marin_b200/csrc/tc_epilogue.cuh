@@ -10,6 +10,7 @@
 #define TC_OUT_F32 1
 #define TC_OUT_F32_ACC 2
 #define TC_OUT_SWIGLU 3       // w holds gate and up rows interleaved in blocks of 16; out [T, N/2] bf16 = silu(gate) * up
+#define TC_OUT_REGLU 5        // as TC_OUT_SWIGLU with max(gate, 0) * up
 #define TC_OUT_RELU2 4        // out bf16 = max(x w^T, 0)^2: the activation of a feed-forward without a gate
 
 __device__ __forceinline__ float relu2_of(float v) { v = fmaxf(v, 0.0f); return v * v; }
@@ -61,8 +62,8 @@ __device__ __forceinline__ void store_chunk(void* out, int mode, int t_first, in
 // rows of the same intermediate indices, so lane l < 16 holds gate(i) and lane l + 16 holds up(i): one shuffle brings
 // them together and out[t, i] = g / (1 + exp(-g)) * u is written in bf16 (crates/tensor/src/silu.rs:18; the fast
 // exponential and division are accurate to a few float32 ulps, far inside the bf16 rounding of the result).  All 32
-// lanes must call this; n_base is the warp's first weight row (a multiple of 32).
-__device__ __forceinline__ void store_chunk_swiglu(void* out, int t_first, int n_base, int lane, int T, int N, const float* v) {
+// lanes must call this; n_base is the warp's first weight row (a multiple of 32).  relu: max(g, 0) * u instead.
+__device__ __forceinline__ void store_chunk_swiglu(void* out, int t_first, int n_base, int lane, int T, int N, const float* v, bool relu) {
     bf16* o = (bf16*)out;
     const int half = N >> 1;
     const int i = (n_base >> 1) + (lane & 15);
@@ -71,7 +72,7 @@ __device__ __forceinline__ void store_chunk_swiglu(void* out, int t_first, int n
         const float u = __shfl_down_sync(0xffffffffu, v[j], 16);
         const float g = v[j];
         if (lane < 16 && t_first + j < T && i < half)
-            o[(size_t)(t_first + j) * half + i] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u);
+            o[(size_t)(t_first + j) * half + i] = __float2bfloat16_rn((relu ? fmaxf(g, 0.0f) : __fdividef(g, 1.0f + __expf(-g))) * u);
     }
 }
 

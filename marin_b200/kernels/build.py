@@ -161,6 +161,8 @@ LIBRARIES: Dict[str, List[str]] = {
     "mb_moe": ["moe.cu"],
     "mb_attention_pooled": ["attention_pooled.cu"],
     "mb_ssm": ["ssm.cu"],
+    "mb_layer_norm": ["layer_norm.cu"],
+    "mb_delta_rule": ["delta_rule.cu"],
     "mb_host": ["host/cache_core.cpp", "host/scheduler.cpp", "host/sampler.cpp", "host/safetensors.cpp"],
 }
 

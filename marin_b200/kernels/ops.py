@@ -124,6 +124,26 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, pos_table: 
                                           _ptr(out), _c_int(T), _c_int(h), _c_float(scale), _stream()), "embed")
 
 
+def embed_bigram(ctx, table: torch.Tensor, pairs: torch.Tensor, last: torch.Tensor, slots: torch.Tensor, mul_before: int, mul_now: int, buckets: int,
+                 out: torch.Tensor, scale: float = 1.0) -> None:
+    """``out[t] = float32(table[id]) * scale + float32(pairs[r])``, ``r = (id before * mul_before + id * mul_now) mod buckets`` or the
+    last row, ``buckets``, for a sequence's first token.  ``last`` (int32 ``[slots, 1]``) keeps every request's latest token."""
+    ids = ctx.token_ids
+    _need_cuda(ids, table, pairs, last, out, slots)
+    T, h = out.shape
+    assert ids.dtype == torch.int32 and ids.numel() == T and table.shape[1] == h and out.dtype == torch.float32 and last.dtype == torch.int32
+    assert tuple(pairs.shape) == (buckets + 1, h) and pairs.dtype == table.dtype and last.numel() == last.shape[0]
+    single = ctx.max_query_len <= 1
+    _cost(2 * T * h * table.element_size() + _size(out) + _size(ids))
+    _check(_lib("mb_elementwise").mb_embed_bigram(
+        _ptr(ids), _ptr(table), _ptr(pairs), _code(table), _ptr(ctx.positions), _ptr(ctx.req_index), _ptr(ctx.cu_tokens), _ptr(slots), _ptr(last),
+        _ptr(out), _c_int(T), _c_int(ctx.num_requests), _c_int(h), _c_float(scale), ctypes.c_longlong(mul_before), ctypes.c_longlong(mul_now),
+        _c_int(buckets), _c_int(int(single)), _stream()), "embed, bigram")
+    if not single:
+        _check(_lib("mb_elementwise").mb_last_token(_ptr(ids), _ptr(ctx.cu_tokens), _ptr(slots), _ptr(last), _c_int(ctx.num_requests), _stream()),
+               "last token kept")
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, unit_offset: bool = False) -> None:
     _need_cuda(x, weight, out)
     rows, n = x.shape
@@ -716,15 +736,20 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
         _c_float(scale), _c_int(window), _stream()), "attention")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False) -> None:
-    """``out[t, i] = silu(g) * u``; gate and up are the two halves of a row of ``gate_up``, or (``interleaved``)
+#: activations of a gated feed-forward and, for each, the output mode of the tensor-core product that applies it in its epilogue
+GLU_ACTIVATIONS = {"silu": 0, "relu": 1}
+_GLU_MODES = {"silu": 3, "relu": 5}
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, activation: str = "silu") -> None:
+    """``out[t, i] = act(g) * u`` (``activation`` "silu" or "relu"); gate and up are the two halves of a row of ``gate_up``, or (``interleaved``)
     alternate in blocks of 16 columns."""
     _need_cuda(gate_up, out)
     T, I = out.shape
     assert gate_up.shape == (T, 2 * I) and gate_up.dtype == out.dtype and (not interleaved or I % 16 == 0)
     _cost(_size(gate_up) + _size(out), 8.0 * T * I)
     _check(_lib("mb_elementwise").mb_swiglu(_ptr(gate_up), _ptr(out), _code(out), _c_int(T), _c_int(I), _c_int(int(interleaved)),
-                                           _stream()), "swiglu")
+                                           _c_int(GLU_ACTIVATIONS[activation]), _stream()), "swiglu")
 
 
 def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
@@ -739,8 +764,8 @@ def can_fuse_swiglu(dtype, hidden: int, intermediate: int) -> bool:
     return dtype == torch.bfloat16 and intermediate % 16 == 0 and hidden % 8 == 0
 
 
-def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor, workspace=None) -> None:
-    """``out = silu(x Wg^T) * (x Wu^T)`` with ``w_interleaved = interleave_gate_up(Wg, Wu)``: on the tensor cores the
+def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor, workspace=None, activation: str = "silu") -> None:
+    """``out = act(x Wg^T) * (x Wu^T)`` (``activation`` "silu" or "relu") with ``w_interleaved = interleave_gate_up(Wg, Wu)``: on the tensor cores the
     activation is applied to the float32 accumulators in the epilogue and the ``[T, 2 I]`` intermediate never
     exists; otherwise the product and the activation run as two kernels."""
     scaled = x if isinstance(x, NormedRows) else None
@@ -756,27 +781,28 @@ def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor,
     if not fused:
         tmp = workspace.get("gate_up", (T, N), x.dtype) if workspace is not None else torch.empty(T, N, device=x.device, dtype=x.dtype)
         gemm(scaled if scaled is not None else x, w_interleaved, tmp)
-        swiglu(tmp, out, interleaved=True)
+        swiglu(tmp, out, True, activation)
         return
     s = _scratch_for(x.device)
+    mode = _GLU_MODES[activation]
     _cost(_size(w_interleaved) + _size(x) + _size(out), 2.0 * T * N * K)
     if many_tokens(T, N):
         if scaled is not None:
             _check(_lib("mb_gemm_tc").mb_gemm_tc_persistent_coupled(
-                _ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(3), _c_int(T), _c_int(N), _c_int(K), _c_int(persistent_plan(T, N)),
+                _ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(mode), _c_int(T), _c_int(N), _c_int(K), _c_int(persistent_plan(T, N)),
                 _c_int(SM_COUNT), None, _c_int(0), None, None, _ptr(scaled.sumsq), _c_int(scaled.slots), _c_int(scaled.dim),
                 _c_float(scaled.eps), _ptr(s.error), _stream()), "gemm+swiglu (tensor cores, persistent, coupled with a norm)")
             return
-        _persistent_product(x, w_interleaved, out, 3, T, N, K, s, "gemm+swiglu (tensor cores, persistent)")
+        _persistent_product(x, w_interleaved, out, mode, T, N, K, s, "gemm+swiglu (tensor cores, persistent)")
         return
     bn, _ = gemm_plan(T, N, K)
     if scaled is not None:
         _check(_lib("mb_gemm_tc").mb_gemm_tc_coupled(
-            _ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(3), _c_int(T), _c_int(N), _c_int(K), _c_int(bn), _c_int(1),
+            _ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(mode), _c_int(T), _c_int(N), _c_int(K), _c_int(bn), _c_int(1),
             None, _c_int(0), None, None, _ptr(scaled.sumsq), _c_int(scaled.slots), _c_int(scaled.dim), _c_float(scaled.eps),
             _ptr(s.error), _stream()), "gemm+swiglu (tensor cores, coupled with a norm)")
         return
-    _check(_lib("mb_gemm_tc").mb_gemm_tc_cluster(_ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(3), _c_int(T), _c_int(N), _c_int(K),
+    _check(_lib("mb_gemm_tc").mb_gemm_tc_cluster(_ptr(x), _ptr(w_interleaved), _ptr(out), _c_int(mode), _c_int(T), _c_int(N), _c_int(K),
                                                 _c_int(bn), _c_int(1), _ptr(s.error), _stream()), "gemm+swiglu (tensor cores)")
 
 
@@ -1214,15 +1240,16 @@ def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Opt
     ``[H d]`` / ``[K d]``), the rotation of the first ``rot_dim`` elements of each head (half-split pairs, or neighbours
     ``(2i, 2i + 1)`` if ``interleaved``; sines and cosines times ``rot_mag``), and the values: as they are, also left in ``v_shared`` ("leave"), or mixed with what ``v_shared`` holds,
     ``(1 - lam) v + lam v_shared`` ("mix").  Queries go to ``q_out``, keys and values into their pages."""
-    _need_cuda(rows, q_out, q_b, k_b, v_b, q_w, k_w, positions, inv_freq, slot_mapping, k_cache, v_cache, v_shared, v_lambda)
+    _need_cuda(q_out, q_b, k_b, v_b, q_w, k_w, positions, inv_freq, slot_mapping, k_cache, v_cache, v_shared, v_lambda)
     T = rows.shape[0]
+    assert rows.is_cuda and rows.stride(1) == 1             # (it may be a column block of a wider product)
     assert tuple(q_out.shape) == (T, H * d) and q_out.dtype == rows.dtype and rows.shape[1] >= ((H + K) * d + K * dv if write_kv else H * d)
     assert k_cache.dtype == rows.dtype and v_cache.dtype == rows.dtype and k_cache.shape[3] == d and v_cache.shape[3] == dv
     assert v_shared is None or (v_shared.dtype == rows.dtype and v_shared.numel() >= T * K * dv)
     page_size = k_cache.shape[2]
     _cost(2 * T * ((H + K) * d + K * dv) * rows.element_size(), 10.0 * T * (H + K) * d)
     _check(_lib("mb_attention_sink").mb_qkv_finish(
-        _ptr(rows), _c_int(rows.shape[1]), _code(rows), _ptr(q_out), _ptr(q_b), _ptr(k_b), _ptr(v_b), _c_int(NORM_MODES[norm]), _ptr(q_w),
+        _ptr(rows), _c_int(rows.stride(0)), _code(rows), _ptr(q_out), _ptr(q_b), _ptr(k_b), _ptr(v_b), _c_int(NORM_MODES[norm]), _ptr(q_w),
         _ptr(k_w), _c_float(eps), _ptr(positions), _ptr(inv_freq), _c_int(rot_dim if inv_freq is not None else 0), _c_float(rot_mag),
         _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _c_int(VALUE_MODES[value_mode]), _ptr(v_shared), _ptr(v_lambda), _c_int(T),
         _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_int(int(write_kv)), _c_int(int(interleaved)), _stream()),
@@ -1231,14 +1258,18 @@ def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Opt
 
 def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d: int, dv: int, scale: float, window: int = 0,
                    chunk: int = 0, sink: bool = True, gate: Optional[torch.Tensor] = None, plan=None,
-                   sink_logits: Optional[torch.Tensor] = None) -> None:
+                   sink_logits: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0, out_scale: float = 1.0) -> None:
     """Causal softmax attention of the step's tokens over the paged cache.  A position sees the keys before it (its own
     included), of them only the last ``window`` (0: all) and only those of its own chunk of ``chunk`` positions (0: no
     chunks).  ``sink``: ``exp(sink_logits[head])`` is added to the softmax's denominator (float32 ``[H]``, not scaled; None: a
     score of 0, so one is added).  ``gate`` (activation dtype, a view ``[T, H dv]`` whose rows may be strided): the result is
     multiplied by ``sigmoid(gate)``.  ``v_cache`` may be ``k_cache`` itself: the values are then the first ``dv`` elements
-    of the key rows (a latent that keys and values share)."""
-    _need_cuda(q, k_cache, v_cache, out, block_table, sink_logits)
+    of the key rows (a latent that keys and values share).  ``keep_first``: the sequence's first positions are seen however
+    old they are.  ``softcap`` > 0: scores become ``softcap tanh(s / softcap)`` (the sink's does not).  The result is multiplied
+    by ``out_scale``; ``out`` may be a column block of a wider buffer."""
+    _need_cuda(q, k_cache, v_cache, block_table, sink_logits)
+    assert out.is_cuda and out.stride(1) == 1
+    variant = keep_first > 0 or softcap > 0.0 or out_scale != 1.0 or out.stride(0) != H * dv
     T = q.shape[0]
     page_size = k_cache.shape[2]
     values_in_keys = v_cache.data_ptr() == k_cache.data_ptr()
@@ -1255,7 +1286,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     size = q.element_size()
     per_row = H * (d + (3 if gate is not None else 2) * dv) * size
     key_bytes = (d if values_in_keys else K * (d + dv)) * size      # what one cached position holds for this layer
-    if use_fast_sink_attention and fast_sink_attention_supported(q.dtype, H, K, d, dv, values_in_keys) and page_size & (page_size - 1) == 0:
+    if not variant and use_fast_sink_attention and fast_sink_attention_supported(q.dtype, H, K, d, dv, values_in_keys) and page_size & (page_size - 1) == 0:
         kv_heads = K
         if values_in_keys:
             # one kv head that every query head reads: a CTA takes as many query heads as the kernels group, and `K` counts
@@ -1308,7 +1339,8 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     _check(_lib("mb_attention_sink").mb_attention_sink(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _code(q), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(ctx.req_index),
         _ptr(ctx.positions), _c_int(T), _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_float(scale), _c_int(window),
-        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), _stream()), "attention (sink)")
+        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), _c_int(keep_first),
+        _c_float(softcap), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink)")
 
 
 #: bf16 sink attention goes to the tensor-core kernels where the head layout allows (False: always the plain kernel)
@@ -1384,7 +1416,7 @@ class SinkDecodePlan:
 
 
 def sink_decode_plan(dtype, requests: int, H: int, K: int, d: int, dv: int, span: int, window: int, chunk: int,
-                     values_in_keys: bool = False):
+                     values_in_keys: bool = False, keep_first: int = 0):
     """The number of chunks whose CTAs finish soonest: the CTAs of all requests, kv heads and chunks run in waves of as many as
     the device holds at a time, and a wave lasts as long as one CTA's walk over its chunk, so the cost of ``c`` chunks is
     ``waves(c) * (blocks per chunk + a CTA's start and end)``; among equals, the fewest chunks (the merge reads them all).  A
@@ -1402,6 +1434,8 @@ def sink_decode_plan(dtype, requests: int, H: int, K: int, d: int, dv: int, span
     if chunk > 0:
         seen = min(seen, chunk)
     longest = seen + 63                                # the first chunk starts on a block border at or before the first seen key
+    if keep_first > 0:
+        longest += -(-keep_first // 64) * 64           # blocks of kept first positions come before the window's
     split = _sink_split(max(1, requests * K), longest, max(1, SINK_DECODE_CTAS_PER_SM * SM_COUNT))
     return SinkDecodePlan(split, max(1, -(-longest // split)))
 
@@ -1470,18 +1504,23 @@ SCORE_MODES = {"sigmoid": 0, "softmax": 1}
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, experts_out: torch.Tensor, weights_out: torch.Tensor, score: str = "sigmoid",
-              renormalize: bool = False, bias: Optional[torch.Tensor] = None) -> None:
+              renormalize: bool = False, bias: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None, groups: int = 1,
+              keep_groups: int = 1, factor: float = 1.0) -> None:
     """Router logits ``x router^T (+ bias)`` in float32, scores by ``score``, the ``top`` best experts per token (``top`` = the outputs'
-    second size) in order of decreasing score, the lower expert among equals; their scores are the weights."""
-    _need_cuda(x, router, experts_out, weights_out)
+    second size) in order of decreasing score, the lower expert among equals; their scores are the weights.
+    ``correction`` (float32 ``[E]``) is added to the scores for the choice only; with ``groups`` equal groups of neighbours only those of
+    the ``keep_groups`` groups with the largest choice score can be chosen; the weights are multiplied by ``factor``."""
+    _need_cuda(x, router, experts_out, weights_out, correction)
     T, h = x.shape
     E, top = router.shape[0], experts_out.shape[1]
     assert router.dtype == torch.float32 and router.shape[1] == h and experts_out.dtype == torch.int32 and weights_out.dtype == torch.float32
     assert tuple(experts_out.shape) == (T, top) and tuple(weights_out.shape) == (T, top)
     assert bias is None or (bias.is_cuda and bias.dtype == torch.float32 and bias.numel() == E)
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
     _cost(_size(x) + _size(router) + _size(experts_out) * 2, 2.0 * T * E * h)
     _check(_lib("mb_moe").mb_moe_route(_ptr(x), _code(x), _ptr(router), _ptr(bias), _ptr(experts_out), _ptr(weights_out), _c_int(T), _c_int(h), _c_int(E),
-                                      _c_int(top), _c_int(SCORE_MODES[score]), _c_int(int(renormalize)), _stream()), "router")
+                                      _c_int(top), _c_int(SCORE_MODES[score]), _c_int(int(renormalize)), _ptr(correction), _c_int(groups),
+                                      _c_int(keep_groups), _c_float(factor), _stream()), "router")
 
 
 def moe_table_route(token_ids: torch.Tensor, table: torch.Tensor, E: int, experts_out: torch.Tensor, weights_out: torch.Tensor) -> None:
@@ -1525,7 +1564,8 @@ def moe_experts_plain(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Te
     """``y[t] += sum_c down_e( silu(gate_e x) * (up_e x) )`` over token ``t``'s chosen experts ``e`` in choice order, ``x = w h[t]``
     where the weight goes on the input, else the result times ``w``.  Any sizes, both dtypes.  ``interleaved``: an expert's
     gate and up rows alternate in blocks of 16 (``interleave_gate_up``) instead of gate rows first.  ``activation`` "relu2":
-    experts without a gate, ``down_e( relu(up_e x)^2 )``, ``w_gate_up`` then holds the up matrices ``[E, ff, h]`` alone."""
+    experts without a gate, ``down_e( relu(up_e x)^2 )``, ``w_gate_up`` then holds the up matrices ``[E, ff, h]`` alone.  A choice
+    numbered ``E`` or above stands for the identity: ``w h[t]``."""
     _need_cuda(x, w_gate_up, w_down, experts, weights, act, y)
     T, h = x.shape
     top = experts.shape[1]
@@ -1544,7 +1584,7 @@ def moe_experts_plain(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Te
         _check(_lib("mb_moe").mb_moe_experts_plain(_ptr(x), _code(x), _ptr(w_gate_up), _ptr(w_down), _ptr(experts), _ptr(weights), _ptr(act),
                                                   _ptr(y), _c_int(T), _c_int(h), _c_int(ff), _c_int(top), _c_int(int(weight_on_input)),
                                                   _c_int(int(interleaved)), _c_int(which), _c_int(EXPERT_ACTIVATIONS[activation]), _c_float(limit),
-                                                  _c_float(alpha), _c_float(shift), _stream()), what)
+                                                  _c_float(alpha), _c_float(shift), _c_int(w_down.shape[0]), _stream()), what)
 
 
 #: bf16 experts go to the grouped tensor-core kernels where the sizes allow (False: always the plain kernels)
@@ -1578,8 +1618,10 @@ def _expert_streams(device, n: int):
 
 
 def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, experts: torch.Tensor, weights: torch.Tensor,
-                y: torch.Tensor, weight_on_input: bool, workspace, interleaved: bool = False, activation: str = "swiglu", form=None) -> None:
-    """The chosen experts' outputs added into ``y`` (float32 ``[T, h]``); see ``moe_experts_plain``.  bf16 with sizes in steps
+                y: torch.Tensor, weight_on_input: bool, workspace, interleaved: bool = False, activation: str = "swiglu", form=None,
+                identity: int = 0) -> None:
+    """The chosen experts' outputs added into ``y`` (float32 ``[T, h]``); see ``moe_experts_plain``.  Choices may also name ``identity``
+    numbers behind the experts': the grouped products never see their pairs, the sum over a token's choices adds them.  bf16 with sizes in steps
     of 64: the pairs are sorted by expert on the device and their inputs gathered in that order; then either two grouped
     products over all experts (few pairs: single-token steps, captured or not: nothing is read back), or, with many pairs
     per expert, the dense tensor-core products expert by expert over the sorted rows (the counts are read back once)."""
@@ -1595,14 +1637,18 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     limit, alpha, shift = _glu_form(activation, form)
     assert tuple(w_gate_up.shape) == (E, (2 if gated else 1) * ff, h) and w_gate_up.dtype == w_down.dtype == x.dtype and tuple(y.shape) == (T, h)
     assert y.dtype == torch.float32 and experts.dtype == torch.int32 and weights.dtype == torch.float32
-    ints = workspace.get("moe_ints", (E + 1 + 3 * pairs,), torch.int32)
-    offsets, order, inv, token_sorted = ints[:E + 1], ints[E + 1:E + 1 + pairs], ints[E + 1 + pairs:E + 1 + 2 * pairs], ints[E + 1 + 2 * pairs:]
+    ends = E + identity + 1
+    ints = workspace.get("moe_ints", (ends + 3 * pairs,), torch.int32)
+    offsets, order, inv, token_sorted = ints[:ends], ints[ends:ends + pairs], ints[ends + pairs:ends + 2 * pairs], ints[ends + 2 * pairs:]
+    if identity and weight_on_input:
+        raise KernelError("experts: identity choices go with weights on the output")
     weight_sorted = workspace.get("moe_weight_sorted", (pairs,), torch.float32)
     xs = workspace.get("moe_xs", (pairs, h), x.dtype)
     size = x.element_size()
     lib = _lib("mb_moe")
     touched = min(pairs, E)
-    moe_group(experts, E, offsets, order)
+    moe_group(experts, E + identity, offsets, order)
+    same = (_ptr(experts), _ptr(x), _ptr(weights), _c_int(E)) if identity else (_ptr(None), _ptr(None), _ptr(None), _c_int(E))
     _cost(2 * pairs * h * size)
     _check(lib.mb_moe_gather(_ptr(x), _ptr(order), _ptr(weights), _ptr(xs), _ptr(token_sorted), _ptr(weight_sorted), _ptr(inv), _c_int(pairs),
                              _c_int(h), _c_int(top), _c_int(int(weight_on_input)), _stream()), "experts' inputs gathered")
@@ -1652,7 +1698,7 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
                 current.wait_event(done)
         _cost(_size(rows) + 2 * _size(y))
         _check(lib.mb_moe_combine(_ptr(rows), _ptr(inv), _ptr(None if weight_on_input else weights), _ptr(y), _c_int(T), _c_int(h),
-                                  _c_int(top), _stream()), "experts' outputs added")
+                                  _c_int(top), *same, _stream()), "experts' outputs added")
         return
     _cost(touched * (2 if gated else 1) * ff * h * size + pairs * (h + ff) * size, (4.0 if gated else 2.0) * pairs * ff * h)
     _check(lib.mb_moe_grouped_gate_up(_ptr(xs), _ptr(w_gate_up), _ptr(offsets), _ptr(act), _c_int(pairs), _c_int(h), _c_int(ff), _c_int(E),
@@ -1661,7 +1707,7 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
            "experts, gate|up, SwiGLU (grouped, tensor cores)" if gated else "experts, up, relu squared (grouped, tensor cores)")
     scale = None if weight_on_input else weight_sorted
     _cost(touched * ff * h * size + pairs * ff * size + 2 * pairs * h * 4, 2.0 * pairs * ff * h)
-    if top == 1:           # every pair has a row of y to itself: the product adds into it
+    if top == 1 and not identity:           # every pair has a row of y to itself: the product adds into it
         _check(lib.mb_moe_grouped_down(_ptr(act), _ptr(w_down), _ptr(offsets), _ptr(y), _ptr(token_sorted), _ptr(scale), _c_int(1),
                                        _c_int(pairs), _c_int(h), _c_int(ff), _c_int(E), _stream()), "experts, down (grouped, tensor cores)")
         return
@@ -1669,7 +1715,7 @@ def moe_experts(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     _check(lib.mb_moe_grouped_down(_ptr(act), _ptr(w_down), _ptr(offsets), _ptr(rows), _ptr(None), _ptr(scale), _c_int(0),
                                    _c_int(pairs), _c_int(h), _c_int(ff), _c_int(E), _stream()), "experts, down (grouped, tensor cores)")
     _cost(_size(rows) + 2 * _size(y))
-    _check(lib.mb_moe_combine(_ptr(rows), _ptr(inv), _ptr(None), _ptr(y), _c_int(T), _c_int(h), _c_int(top), _stream()), "experts' outputs added")
+    _check(lib.mb_moe_combine(_ptr(rows), _ptr(inv), _ptr(None), _ptr(y), _c_int(T), _c_int(h), _c_int(top), *same, _stream()), "experts' outputs added")
 
 
 # ---- attention over a window and pooled blocks before it (csrc/attention_pooled.cu) ------------------------------------------------
@@ -1914,3 +1960,146 @@ def rmsnorm_cols(rows: torch.Tensor, col: int, weight: torch.Tensor, eps: float,
     _cost(2 * T * n * rows.element_size(), 4.0 * T * n)
     _check(_lib("mb_activations").mb_rmsnorm_cols(_ptr(rows), _c_int(rows.stride(0)), _c_int(col), _code(rows), _ptr(weight), _c_float(eps), _ptr(out),
                                                  _c_int(T), _c_int(n), _stream()), "rmsnorm of a column block")
+
+
+# ---- layer norm, and the end of a sublayer whose output is normed (csrc/layer_norm.cu) ------------------------------------------------
+NORM_KINDS = {"layer": 0, "rms": 1}
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out: torch.Tensor) -> None:
+    """``out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight (+ bias)`` over the rows of a float32 matrix."""
+    _need_cuda(x, weight, bias, out)
+    rows, n = x.shape
+    assert x.dtype == torch.float32 and weight.dtype == torch.float32 and weight.numel() == n and tuple(out.shape) == (rows, n)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == n)
+    _cost(_size(x) + _size(out), 6.0 * rows * n)
+    _check(_lib("mb_layer_norm").mb_layer_norm(_ptr(x), _ptr(weight), _ptr(bias), _ptr(None), _ptr(None), _ptr(out), _c_int(_code(out)), _c_int(rows),
+                                              _c_int(n), _c_float(eps), _c_int(0), _stream()), "layer norm")
+
+
+def norm_into(y: torch.Tensor, kind: str, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, scale: Optional[torch.Tensor],
+              hidden: torch.Tensor, rows: Optional[torch.Tensor]) -> None:
+    """The end of a sublayer: ``hidden += norm(y) * scale`` (``kind`` "layer" or "rms"; ``scale`` a vector or None), ``y <- 0`` for the next
+    sublayer to add into, and (``rows`` given) the new rows of the stream in that tensor's dtype.  ``y``, ``hidden`` float32."""
+    _need_cuda(y, weight, bias, scale, hidden, rows)
+    T, n = y.shape
+    assert y.dtype == hidden.dtype == torch.float32 and tuple(hidden.shape) == (T, n) and weight.numel() == n
+    assert all(v is None or (v.dtype == torch.float32 and v.numel() == n) for v in (weight, bias, scale))
+    assert rows is None or tuple(rows.shape) == (T, n)
+    _cost(2 * _size(y) + 2 * _size(hidden) + (_size(rows) if rows is not None else 0), 9.0 * T * n)
+    _check(_lib("mb_layer_norm").mb_layer_norm(_ptr(y), _ptr(weight), _ptr(bias), _ptr(scale), _ptr(hidden), _ptr(rows),
+                                              _c_int(_code(rows) if rows is not None else F32), _c_int(T), _c_int(n), _c_float(eps),
+                                              _c_int(NORM_KINDS[kind]), _stream()), "norm into the stream")
+
+
+def stream_rows(hidden: torch.Tensor, rows: Optional[torch.Tensor], y: torch.Tensor) -> None:
+    """Where no sublayer has run yet: the stream's rows in bfloat16 (``rows`` given) and ``y <- 0`` for the first one to add into."""
+    _need_cuda(hidden, rows, y)
+    assert hidden.dtype == y.dtype == torch.float32 and hidden.numel() == y.numel()
+    assert rows is None or (rows.dtype == torch.bfloat16 and rows.numel() == hidden.numel())
+    _cost(_size(y) + (_size(hidden) + _size(rows) if rows is not None else 0))
+    _check(_lib("mb_layer_norm").mb_stream_rows(_ptr(hidden), _ptr(rows), _ptr(y), _c_size_t(hidden.numel()), _stream()), "stream rows")
+
+
+# ---- the gated delta rule (csrc/delta_rule.cu) ------------------------------------------------------------------------------------------
+DELTA_GATES = {"sigmoid": 0, "silu": 1}
+
+
+def _columns(t: torch.Tensor, T: int, n: int, dtype) -> int:
+    """The row stride of a column block ``[T, n]`` of a product."""
+    assert t.is_cuda and t.dtype == dtype and tuple(t.shape) == (T, n) and t.stride(1) == 1, (tuple(t.shape), T, n)
+    return t.stride(0)
+
+
+def delta_conv(qkv: torch.Tensor, weight: torch.Tensor, ring: torch.Tensor, ctx, slots: torch.Tensor, out: torch.Tensor, first_req: int = 0,
+               first_token: int = 0) -> None:
+    """A causal convolution over time per channel, then silu, of the step's tokens from ``first_token`` on (the tokens of the requests from
+    ``first_req`` on); ``weight`` float32 ``[channels, taps]``, its last column on the current token.  ``ring`` (float32 ``[slots, taps,
+    channels]``) keeps every request's latest inputs, that of position ``p`` in row ``p mod taps``, and is brought up to date."""
+    _need_cuda(weight, ring, out, slots)
+    T, channels = out.shape
+    taps = weight.shape[1]
+    stride = _columns(qkv, T, channels, out.dtype)
+    assert weight.dtype == torch.float32 and weight.shape[0] == channels and ring.dtype == torch.float32 and tuple(ring.shape[1:]) == (taps, channels)
+    lib = _lib("mb_delta_rule")
+    _cost(2 * (T - first_token) * channels * out.element_size(), 2.0 * (T - first_token) * channels * taps)
+    _check(lib.mb_delta_conv(_c_void_p(qkv.data_ptr()), _c_int(stride), _code(out), _ptr(weight), _ptr(ring), _ptr(ctx.positions), _ptr(ctx.req_index),
+                             _ptr(ctx.cu_tokens), _ptr(slots), _ptr(out), _c_int(first_token), _c_int(T), _c_int(channels), _c_int(taps), _stream()),
+           "short convolution")
+    if taps > 1:
+        _cost((ctx.num_requests - first_req) * (taps - 1) * channels * (4 + out.element_size()))
+        _check(lib.mb_delta_ring(_c_void_p(qkv.data_ptr()), _c_int(stride), _code(out), _ptr(ring), _ptr(ctx.positions), _ptr(ctx.cu_tokens), _ptr(slots),
+                                 _c_int(first_req), _c_int(ctx.num_requests), _c_int(channels), _c_int(taps), _stream()), "convolution's inputs kept")
+
+
+class DeltaInputs:
+    """What a gated delta rule takes besides q, k and v, as the projections left it: ``beta`` ``[T, H]``, ``decay`` ``[T, H]`` or (one per key
+    channel) ``[T, H d]``, ``gate`` ``[T, H dv]`` (column blocks of a product, activation dtype); float32 vectors ``rate`` ``[H]`` (A_log) and
+    ``dt_bias`` (as many as decays)."""
+    __slots__ = ("beta", "decay", "gate", "rate", "dt_bias")
+
+    def __init__(self, beta, decay, gate, rate, dt_bias):
+        self.beta, self.decay, self.gate, self.rate, self.dt_bias = beta, decay, gate, rate, dt_bias
+
+
+def _delta_args(inp: DeltaInputs, T: int, H: int, d: int, dtype):
+    per_channel = inp.decay.shape[1] != H
+    assert inp.rate.numel() == H and inp.dt_bias.numel() == (H * d if per_channel else H) and inp.rate.dtype == inp.dt_bias.dtype == torch.float32
+    return (_c_void_p(inp.beta.data_ptr()), _c_int(_columns(inp.beta, T, H, dtype)), _c_void_p(inp.decay.data_ptr()),
+            _c_int(_columns(inp.decay, T, H * d if per_channel else H, dtype)), _c_int(int(per_channel)), _ptr(inp.rate), _ptr(inp.dt_bias))
+
+
+def delta_scan(qkv: torch.Tensor, inp: DeltaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, o: torch.Tensor, H: int, G: int, d: int, dv: int,
+               first_req: int = 0) -> None:
+    """The recurrence token by token over the requests from ``first_req`` on: ``qkv`` after the convolution, ``state`` float32 ``[slots, H, d,
+    dv]``, ``o`` float32 ``[T, H dv]``.  Any size, both dtypes."""
+    _need_cuda(qkv, state, o, slots)
+    T = qkv.shape[0]
+    assert qkv.shape[1] == 2 * G * d + H * dv and tuple(state.shape[1:]) == (H, d, dv) and state.dtype == o.dtype == torch.float32 and tuple(o.shape) == (T, H * dv)
+    R = ctx.num_requests - first_req
+    _cost(_size(qkv) + _size(o) + 2.0 * R * H * d * dv * 4, 6.0 * T * H * d * dv)
+    _check(_lib("mb_delta_rule").mb_delta_scan(_ptr(qkv), _code(qkv), *_delta_args(inp, T, H, d, qkv.dtype), _ptr(state), _ptr(ctx.cu_tokens), _ptr(slots),
+                                              _ptr(o), _c_int(first_req), _c_int(ctx.num_requests), _c_int(H), _c_int(G), _c_int(d), _c_int(dv), _stream()),
+           "delta rule (scan)")
+
+
+def delta_norm(o: torch.Tensor, gate_rows: torch.Tensor, gate: str, weight: torch.Tensor, eps: float, factor: float, out: torch.Tensor, H: int, dv: int,
+               first_token: int = 0) -> None:
+    """``out = o / rms(o per head) * weight * gate(gate_rows) * factor`` for the tokens from ``first_token`` on; ``out`` may be a column block."""
+    _need_cuda(o, weight)
+    T = o.shape[0]
+    assert o.dtype == torch.float32 and tuple(o.shape) == (T, H * dv) and weight.numel() == dv and weight.dtype == torch.float32
+    _cost((T - first_token) * H * dv * (4 + 2 * out.element_size()), 8.0 * (T - first_token) * H * dv)
+    _check(_lib("mb_delta_rule").mb_delta_norm(_ptr(o), _c_void_p(gate_rows.data_ptr()), _c_int(_columns(gate_rows, T, H * dv, out.dtype)),
+                                              _c_int(DELTA_GATES[gate]), _code(out), _ptr(weight), _c_float(eps), _c_float(factor),
+                                              _c_void_p(out.data_ptr()), _c_int(_columns(out, T, H * dv, out.dtype)), _c_int(first_token), _c_int(T),
+                                              _c_int(H), _c_int(dv), _stream()), "delta rule, norm and gate")
+
+
+#: single tokens of a delta rule run in one kernel where a head's state fits a block's registers (False: as portions do)
+use_delta_single = True
+
+
+def delta_single_supported(d: int, dv: int) -> bool:
+    return 1 <= d <= 256 and 4 <= dv <= 256 and dv % 4 == 0 and (dv // 4) * (16 if d > 128 else 8) <= 512
+
+
+def delta_single(qkv: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, inp: DeltaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, gate: str,
+                 norm_w: torch.Tensor, eps: float, factor: float, out: torch.Tensor, requests: int, H: int, G: int, d: int, dv: int) -> None:
+    """Convolution, recurrence, norm and gate of the first ``requests`` requests, which bring one token each (token r is request r's), in one
+    kernel; ``qkv`` as the projection left it, ``out`` a column block ``[T, H dv]``."""
+    _need_cuda(conv_w, ring, state, norm_w, slots)
+    T = qkv.shape[0]
+    channels, taps = 2 * G * d + H * dv, conv_w.shape[1]
+    dtype = qkv.dtype
+    _cost(requests * (2.0 * H * d * dv * 4 + channels * (2 * dtype.itemsize + taps * 4)), 6.0 * requests * H * d * dv)
+    _check(_lib("mb_delta_rule").mb_delta_single(
+        _c_void_p(qkv.data_ptr()), _c_int(_columns(qkv, T, channels, dtype)), _code(qkv), _ptr(conv_w), _ptr(ring), _c_int(taps),
+        *_delta_args(inp, T, H, d, dtype), _ptr(state), _ptr(ctx.positions), _ptr(ctx.seq_lens), _ptr(slots), _c_void_p(inp.gate.data_ptr()),
+        _c_int(_columns(inp.gate, T, H * dv, dtype)), _c_int(DELTA_GATES[gate]), _ptr(norm_w), _c_float(eps), _c_float(factor),
+        _c_void_p(out.data_ptr()), _c_int(_columns(out, T, H * dv, dtype)), _c_int(requests), _c_int(H), _c_int(G), _c_int(d), _c_int(dv), _stream()),
+        "delta rule (single tokens)")
+
+
+def delta_rule_jobs(dtype, d: int, dv: int) -> dict:
+    return library_jobs("mb_delta_rule")

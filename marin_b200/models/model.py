@@ -36,12 +36,17 @@ class Model:
         return specs
 
     def cache_needs(self) -> List[object]:
-        """What each schedule entry keeps between steps (None for entries that read another's cache)."""
+        """What each schedule entry keeps between steps (None for entries that read another's cache); behind them, where the
+        embedding keeps a state, the embedding's need."""
         needs = []
         for entry in self.spec.schedule:
             need = self.blocks[entry.layer].mixer.cache_need()
             needs.append(need if entry.cache_of is None else None)
-        return needs
+        own = self._embedding_need()
+        return needs if own is None else needs + [own]
+
+    def _embedding_need(self):
+        return self.embedding.cache_need() if hasattr(self.embedding, "cache_need") else None
 
     # ---- what the code around the model asks of it: every answer is the sum of the parts' own answers ----------------
     def parts(self) -> List[object]:
@@ -80,7 +85,7 @@ class Model:
                 return sum(of(n) for n in need)
             return need.bytes_read(context, dtype)
 
-        return sum(of(self.blocks[entry.layer].mixer.cache_need()) for entry in self.spec.schedule)
+        return sum(of(self.blocks[entry.layer].mixer.cache_need()) for entry in self.spec.schedule) + of(self._embedding_need())
 
     def kernel_jobs(self, dtype: torch.dtype) -> Dict[str, tuple]:
         """``{library: (sources, defines)}`` of the kernels specialised for this model's parts."""
@@ -123,10 +128,13 @@ class Model:
         T = ctx.num_tokens
         S = self.spec.streams
         ops.stage_name = "embedding"
+        extra = {}
+        if self._embedding_need() is not None:
+            extra = {"ctx": ctx, "cache": caches.view(len(self.spec.schedule), ctx)}
         if S > 0:
             # several copies of the residual stream, all equal to the embedding's output at first
             hidden = ws.get("hidden", (S, T, self.spec.hidden_size), torch.float32)
-            self.embedding.forward(ctx.token_ids, hidden[0], ctx.positions)
+            self.embedding.forward(ctx.token_ids, hidden[0], ctx.positions, **extra)
             ops.hc_spread(hidden)
             seen, observe = observe, None
             if seen is not None:
@@ -136,7 +144,7 @@ class Model:
                     seen(i, total)
         else:
             hidden = ws.get("hidden", (T, self.spec.hidden_size), torch.float32)
-            self.embedding.forward(ctx.token_ids, hidden, ctx.positions)
+            self.embedding.forward(ctx.token_ids, hidden, ctx.positions, **extra)
         if observe is not None:
             observe(0, hidden)
         carried = None            # the next block's first norm, if the block before could carry it on its last product

@@ -193,3 +193,89 @@ class HyperConnectionBlock(Part):
             return normed
         ops.hc_step(hidden, y, write=write)
         return None
+
+
+@register_block("postnorm")
+class PostNormBlock(Part):
+    """``x <- x + s1 * norm1(mixer(x)); x <- x + s2 * norm2(feedforward(x))``: the norms are on the sublayers' outputs, the sublayers
+    read the residual stream itself (in the activation dtype).  ``s1``, ``s2``: a learned vector per sublayer (layer scale: Touvron et al.,
+    "Going deeper with Image Transformers"), named by ``block_params["layer_scale"]`` inside the prefix; absent: not scaled.  The norm is an RMS
+    or layer norm part.
+
+    The sublayers *add* into a float32 buffer ``y`` that the step before left zeroed, exactly as they add into the stream of a pre-norm
+    block; one kernel then norms ``y``, scales it, adds it to the stream, zeroes ``y`` and leaves the stream's new rows in the activation
+    dtype for the sublayer behind it, across the border to the next block too when that is a block of this kind (``chains_norm``)."""
+
+    def __init__(self, spec: LayerSpec):
+        names = spec.names
+        norm_cls = lookup("norm", spec.norm.kind)
+        self.norm1 = norm_cls(name=f"{spec.prefix}.{names['norm1']}", **spec.norm.params)
+        self.mixer = lookup("mixer", spec.mixer.kind)(name=f"{spec.prefix}.{names['mixer']}", **spec.mixer.params)
+        self.norm2 = self.feedforward = None
+        if spec.feedforward is not None:
+            self.norm2 = norm_cls(name=f"{spec.prefix}.{names['norm2']}", **spec.norm.params)
+            self.feedforward = lookup("feedforward", spec.feedforward.kind)(
+                name=f"{spec.prefix}.{names['feedforward']}", **spec.feedforward.params)
+        for norm in (self.norm1, self.norm2):
+            if norm is not None and (not hasattr(norm, "weight") or getattr(norm, "unit_offset", False)):
+                raise ValueError("postnorm: the norm rides on the stream's update and has to be an RMS norm or a layer norm")
+        scales = spec.block_params.get("layer_scale")
+        self.hidden = int(spec.norm.params["dim"])
+        self.scale_names = [f"{spec.prefix}.{s}" for s in scales][: 2 if self.feedforward is not None else 1] if scales else []
+        self.scales: List[torch.Tensor] = []
+
+    def parts(self) -> List[Part]:
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.feedforward) if p is not None]
+
+    def _own_specs(self) -> List[TensorSpec]:
+        return [TensorSpec(n, (self.hidden,), "norm") for n in self.scale_names]
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for p in self.parts() for s in p.tensor_specs()] + self._own_specs()
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        for p in self.parts():
+            p.load(tensors, rt)
+        self.scales = [rt.f32(tensors.pop(n)) for n in self.scale_names]
+        self.rt = rt
+
+    def weight_bytes(self, dtype) -> int:
+        return sum(p.weight_bytes(dtype) for p in self.parts()) + sum(spec_bytes(s, dtype) for s in self._own_specs())
+
+    def bytes_read(self, tokens: int, dtype) -> int:
+        return sum(p.bytes_read(tokens, dtype) for p in self.parts()) + sum(spec_bytes(s, dtype) for s in self._own_specs())
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return sum(p.flops(tokens, pairs) for p in self.parts())
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        jobs: Dict[str, tuple] = dict(ops.library_jobs("mb_layer_norm"))
+        for p in self.parts():
+            jobs.update(p.kernel_jobs(dtype))
+        return jobs
+
+    chains_norm = True
+
+    def _join(self, index: int, y: torch.Tensor, hidden: torch.Tensor, rows) -> None:
+        norm = self.norm1 if index == 0 else self.norm2
+        ops.stage_name = "norm into the stream"
+        ops.norm_into(y, getattr(norm, "kind", "rms"), norm.weight, getattr(norm, "bias", None), norm.eps,
+                      self.scales[index] if self.scales else None, hidden, rows)
+
+    def forward(self, hidden: torch.Tensor, ctx, cache, x_in=None, next_block=None):
+        ws = ctx.workspace
+        wide = self.rt.dtype == torch.float32                  # the stream's own rows serve as they are
+        rows = hidden if wide else ws.get("stream_rows", tuple(hidden.shape), self.rt.dtype)
+        y = ws.get("sublayer_out", tuple(hidden.shape), torch.float32)
+        if x_in is None:                                       # (a block of this kind leaves rows and a zeroed y behind)
+            ops.stage_name = "stream rows"
+            ops.stream_rows(hidden, None if wide else rows, y)
+        self.mixer.forward(rows, ctx, cache, y)
+        goes_on = isinstance(next_block, PostNormBlock)
+        if self.feedforward is not None:
+            self._join(0, y, hidden, None if wide else rows)
+            self.feedforward.forward(rows, ctx, y)
+            self._join(1, y, hidden, rows if goes_on and not wide else None)
+        else:
+            self._join(0, y, hidden, rows if goes_on and not wide else None)
+        return rows if goes_on else None

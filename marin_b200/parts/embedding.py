@@ -7,6 +7,7 @@ import torch
 
 from ..kernels import ops
 from .base import Part, Runtime, element_size
+from .mixer import StateNeed
 from .registry import register_embedding, register_head
 from .spec import TensorSpec
 
@@ -16,10 +17,15 @@ class TokenEmbedding(Part):
     """``hidden[t] = float32(table[ids[t]])`` — no scaling (crates/model/src/qwen3/model.rs:133-153).  With ``positions``
     (a number of rows) a learned position table is added as it is: ``+ float32(pos_table[p])`` for the token at position
     ``p`` of its sequence.  ``tensor`` / ``position_tensor`` name the tensors where they are not ``<name>.weight``.  ``scale``
-    multiplies the table's rows (in float32, as they enter the residual stream); a head tied to the table reads it unscaled."""
+    multiplies the table's rows (in float32, as they enter the residual stream); a head tied to the table reads it unscaled.
+
+    ``bigram`` (``buckets``, ``mul_prev``, ``mul_cur``): a row of a second table (tensor ``bigram_tensor``, ``[buckets + 1, hidden]``) is added,
+    ``(id before * mul_prev + id * mul_cur) mod buckets``, or row ``buckets`` for a sequence's first token.  The token before a step's first
+    one is part of the request's state (``cache_need``)."""
 
     def __init__(self, vocab: int, hidden: int, name: str, tensor: Optional[str] = None, positions: int = 0,
-                 position_tensor: Optional[str] = None, scale: float = 1.0):
+                 position_tensor: Optional[str] = None, scale: float = 1.0, bigram: Optional[Dict[str, int]] = None,
+                 bigram_tensor: Optional[str] = None):
         self.vocab, self.hidden, self.name = int(vocab), int(hidden), name
         self.scale = float(scale)
         self.tensor = tensor or f"{name}.weight"
@@ -27,23 +33,42 @@ class TokenEmbedding(Part):
         self.position_tensor = position_tensor or f"{name}.positions.weight"
         self.table: Optional[torch.Tensor] = None
         self.pos_table: Optional[torch.Tensor] = None
+        self.bigram = None
+        if bigram is not None:
+            self.bigram = {k: int(bigram[k]) for k in ("buckets", "mul_prev", "mul_cur")}
+            if self.bigram["buckets"] <= 0 or self.positions:
+                raise ValueError("a bigram embedding needs at least one bucket, and does not go with a position table")
+        self.bigram_tensor = bigram_tensor or f"{name}.bigram.weight"
+        self.pairs: Optional[torch.Tensor] = None
+
+    def cache_need(self):
+        """A request's latest token, where the next one's embedding depends on it."""
+        return StateNeed((1,), torch.int32) if self.bigram is not None else None
 
     def tensor_specs(self) -> List[TensorSpec]:
         specs = [TensorSpec(self.tensor, (self.vocab, self.hidden), "table")]
         if self.positions:
             specs.append(TensorSpec(self.position_tensor, (self.positions, self.hidden), "table"))
+        if self.bigram is not None:
+            specs.append(TensorSpec(self.bigram_tensor, (self.bigram["buckets"] + 1, self.hidden), "table"))
         return specs
 
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.table = rt.matrix(tensors.pop(self.tensor))
         if self.positions:
             self.pos_table = rt.matrix(tensors.pop(self.position_tensor))
+        if self.bigram is not None:
+            self.pairs = rt.matrix(tensors.pop(self.bigram_tensor))
 
     def bytes_read(self, tokens: int, dtype: torch.dtype) -> int:
         # only the rows asked for leave memory
-        return tokens * self.hidden * element_size(dtype) * (2 if self.positions else 1)
+        return tokens * self.hidden * element_size(dtype) * (2 if self.positions or self.bigram is not None else 1)
 
-    def forward(self, ids: torch.Tensor, out: torch.Tensor, positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+    def forward(self, ids: torch.Tensor, out: torch.Tensor, positions: Optional[torch.Tensor] = None, ctx=None, cache=None) -> torch.Tensor:
+        if self.bigram is not None:
+            b = self.bigram
+            ops.embed_bigram(ctx, self.table, self.pairs, cache.state, cache.slots, b["mul_prev"], b["mul_cur"], b["buckets"], out, self.scale)
+            return out
         if self.positions:
             if positions is None:
                 raise ValueError("an embedding with a position table needs the tokens' positions")

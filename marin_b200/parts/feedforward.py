@@ -31,23 +31,22 @@ class FeedForward(Part):
 @register_feedforward("swiglu")
 class SwiGLU(FeedForward):
     """``down( g / (1 + exp(-g)) * u )`` with ``g = x W_gate^T`` and ``u = x W_up^T``, no bias
-    (crates/model/src/qwen3/mlp.rs:22-37, crates/tensor/src/silu.rs:18)."""
+    (crates/model/src/qwen3/mlp.rs:22-37, crates/tensor/src/silu.rs:18).  ``activation`` "relu": ``down( max(g, 0) * u )``."""
 
-    def __init__(self, hidden: int, intermediate: int, name: str):
-        self.hidden, self.intermediate, self.name = int(hidden), int(intermediate), name
+    def __init__(self, hidden: int, intermediate: int, name: str, activation: str = "silu",
+                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight")):
+        self.hidden, self.intermediate, self.name, self.activation = int(hidden), int(intermediate), name, activation
+        if activation not in ops.GLU_ACTIVATIONS:
+            raise ValueError(f"swiglu: unknown activation {activation!r}")
+        self.gate_name, self.up_name, self.down_name = (f"{name}.{n}" for n in names)
         self.w_gate_up = self.w_down = None
 
     def tensor_specs(self) -> List[TensorSpec]:
-        n, h, i = self.name, self.hidden, self.intermediate
-        return [
-            TensorSpec(f"{n}.gate_proj.weight", (i, h)),
-            TensorSpec(f"{n}.up_proj.weight", (i, h)),
-            TensorSpec(f"{n}.down_proj.weight", (h, i)),
-        ]
+        h, i = self.hidden, self.intermediate
+        return [TensorSpec(self.gate_name, (i, h)), TensorSpec(self.up_name, (i, h)), TensorSpec(self.down_name, (h, i))]
 
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
-        n = self.name
-        gate, up = tensors.pop(f"{n}.gate_proj.weight"), tensors.pop(f"{n}.up_proj.weight")
+        gate, up = tensors.pop(self.gate_name), tensors.pop(self.up_name)
         # One matrix for both projections.  Where the tensor-core kernel can apply the activation in its epilogue
         # the rows are interleaved in blocks of 16 (gate, up, gate, ...) so that a gate value and its up value
         # meet in one warp; otherwise gate rows come first, then up rows.
@@ -56,7 +55,7 @@ class SwiGLU(FeedForward):
             self.w_gate_up = rt.matrix(ops.interleave_gate_up(gate, up))
         else:
             self.w_gate_up = rt.matrix(torch.cat([gate, up], dim=0))
-        self.w_down = rt.matrix(tensors.pop(f"{n}.down_proj.weight"))
+        self.w_down = rt.matrix(tensors.pop(self.down_name))
 
     couples_norm = True
 
@@ -64,13 +63,13 @@ class SwiGLU(FeedForward):
         T = x.shape[0]
         ws = ctx.workspace
         act = ws.get("ffn_act", (T, self.intermediate), x.dtype)
-        ops.stage_name = "gate|up, SwiGLU"
+        ops.stage_name = "gate|up, SwiGLU" if self.activation == "silu" else f"gate|up, {self.activation}"
         if self.fused:
-            ops.gemm_swiglu(x, self.w_gate_up, act, ws)
+            ops.gemm_swiglu(x, self.w_gate_up, act, ws, self.activation)
         else:
             gate_up = ws.get("gate_up", (T, 2 * self.intermediate), x.dtype)
             ops.gemm(x, self.w_gate_up, gate_up)
-            ops.swiglu(gate_up, act)
+            ops.swiglu(gate_up, act, activation=self.activation)
         ops.stage_name = "down"
         return ops.gemm(act, self.w_down, residual, accumulate=True, then_norm=then_norm)
 
@@ -218,12 +217,15 @@ class RoutedExperts(FeedForward):
     reads, ``expert(w h)``, so it passes through the activation; "output": ``w expert(h)``.  Experts have no biases;
     ``activation`` "swiglu": ``down( silu(gate x) * (up x) )``; "relu2": no gate, ``down( relu(up x)^2 )``.
     ``shared_intermediate``: one more expert of that width (same form, tensors ``shared.*``) that every token uses with
-    weight 1.  Nothing is read back to the host: routing, grouping and the experts' products are kernels over device arrays,
+    weight 1.  ``correction``: a learned vector added to the scores for the choice only (the weights stay without); ``groups`` /
+    ``keep_groups``: the router's outputs form equal groups of neighbours and only those of the best groups (by their largest
+    choice score) can be chosen; ``identity``: the router has so many outputs behind the experts' that stand for the identity (the
+    input itself times the weight); ``weight_scale`` multiplies the weights.  Nothing is read back to the host: routing, grouping and the experts' products are kernels over device arrays,
     so single-token steps can be captured in graphs.
     ``names``: the router's (or table's) tensor and the pattern of an expert's tensors inside ``name`` (``{e}`` the expert's
     number)."""
 
-    NAMES = {"router": "router.weight", "router_bias": "router.bias", "table": "table", "gate": "experts.{e}.gate_proj.weight",
+    NAMES = {"router": "router.weight", "router_bias": "router.bias", "correction": "router.correction", "table": "table", "gate": "experts.{e}.gate_proj.weight",
              "up": "experts.{e}.up_proj.weight", "down": "experts.{e}.down_proj.weight", "shared_gate": "shared.gate", "shared_up": "shared.up",
              "shared_down": "shared.down", "shared_scale": "shared.scale"}
 
@@ -231,10 +233,20 @@ class RoutedExperts(FeedForward):
                  renormalize: bool = False, weight_on: str = "input", names=None, router: str = "learned", vocab: int = 0,
                  activation: str = "swiglu", shared_intermediate: Optional[int] = None, router_bias: bool = False,
                  act_limit: float = 0.0, act_alpha: float = 1.0, act_shift: float = 0.0, shared_limit: Optional[float] = None,
-                 shared_scaled: bool = False):
+                 shared_scaled: bool = False, correction: bool = False, groups: int = 1, keep_groups: int = 1, identity: int = 0,
+                 weight_scale: float = 1.0):
         self.hidden, self.intermediate, self.experts, self.top, self.name = int(hidden), int(intermediate), int(experts), int(top), name
-        if not 1 <= self.top <= self.experts:
-            raise ValueError(f"routed_experts: top {top} of {experts} experts")
+        self.correction, self.groups, self.keep_groups = bool(correction), int(groups), int(keep_groups)
+        self.identity, self.weight_scale = int(identity), float(weight_scale)
+        self.outputs = self.experts + self.identity             # of the router
+        if self.groups < 1 or self.outputs % self.groups != 0 or not 1 <= self.keep_groups <= self.groups:
+            raise ValueError(f"routed_experts: {self.outputs} outputs do not form {groups} equal groups of which {keep_groups} are kept")
+        if not 1 <= self.top <= self.outputs // self.groups * self.keep_groups:
+            raise ValueError(f"routed_experts: top {top} of {self.outputs // self.groups * self.keep_groups} that can be chosen")
+        if (self.correction or self.identity or self.groups > 1) and router != "learned":
+            raise ValueError("routed_experts: corrections, groups and identity outputs go with a learned router")
+        if self.identity and weight_on != "output":
+            raise ValueError("routed_experts: identity outputs go with weights on the output")
         if score not in ops.SCORE_MODES or weight_on not in ("input", "output"):
             raise ValueError(f"routed_experts: score {score!r} / weight_on {weight_on!r}")
         if router not in ("learned", "table") or activation not in ops.EXPERT_ACTIVATIONS:
@@ -257,7 +269,10 @@ class RoutedExperts(FeedForward):
                                         self.form[1], self.form[2], shared_scaled,
                                         tuple(self.names[k] for k in ("shared_gate", "shared_up", "shared_down", "shared_scale")))
             elif self.gated:
-                self.shared = SwiGLU(hidden, int(shared_intermediate), f"{name}.shared")
+                shared_names = tuple(self.names[k] for k in ("shared_gate", "shared_up", "shared_down"))
+                # (the default names of a shared expert are those of a feed-forward of its own inside ``shared``)
+                own = {} if shared_names == ("shared.gate", "shared.up", "shared.down") and "shared_gate" not in (names or {}) else {"names": shared_names}
+                self.shared = SwiGLU(hidden, int(shared_intermediate), name if own else f"{name}.shared", **own)
             else:
                 self.shared = ActMLP(hidden, int(shared_intermediate), name, activation,
                                      names=(self.names["shared_up"], self.names["shared_down"]))
@@ -275,9 +290,11 @@ class RoutedExperts(FeedForward):
         if self.routing == "table":
             specs.append(TensorSpec(self._n("table"), (self.vocab, self.top), "int_table", limit=self.experts))
         else:
-            specs.append(TensorSpec(self._n("router"), (self.experts, h), "bias"))
+            specs.append(TensorSpec(self._n("router"), (self.outputs, h), "bias"))
             if self.router_bias:
-                specs.append(TensorSpec(self._n("router_bias"), (self.experts,), "bias"))
+                specs.append(TensorSpec(self._n("router_bias"), (self.outputs,), "bias"))
+            if self.correction:
+                specs.append(TensorSpec(self._n("correction"), (self.outputs,), "bias"))
         if self.shared is not None:
             specs += self.shared.tensor_specs()
         return specs
@@ -304,6 +321,7 @@ class RoutedExperts(FeedForward):
             self.router = rt.f32(tensors.pop(self._n("router")))
             if self.router_bias:
                 self.router_b = rt.f32(tensors.pop(self._n("router_bias")))
+            self.correction_b = rt.f32(tensors.pop(self._n("correction"))) if self.correction else None
         if self.shared is not None:
             self.shared.load(tensors, rt)
         self.rt = rt
@@ -311,12 +329,12 @@ class RoutedExperts(FeedForward):
     def bytes_read(self, tokens: int, dtype) -> int:
         """Only the experts that some token chose are read: at most ``tokens * top`` of them."""
         per_expert = (3 if self.gated else 2) * self.hidden * self.intermediate * element_size(dtype)
-        routing = tokens * self.top * 4 if self.routing == "table" else self.experts * self.hidden * 4
+        routing = tokens * self.top * 4 if self.routing == "table" else self.outputs * self.hidden * 4
         shared = self.shared.bytes_read(tokens, dtype) if self.shared is not None else 0
         return min(self.experts, tokens * self.top) * per_expert + routing + shared
 
     def flops(self, tokens: int, pairs: int = 0) -> float:
-        routing = self.experts if self.routing == "learned" else 0
+        routing = self.outputs if self.routing == "learned" else 0
         shared = self.shared.flops(tokens, pairs) if self.shared is not None else 0.0
         return 2.0 * tokens * self.hidden * (routing + (3 if self.gated else 2) * self.top * self.intermediate) + shared
 
@@ -335,10 +353,11 @@ class RoutedExperts(FeedForward):
         if self.routing == "table":
             ops.moe_table_route(ctx.token_ids, self.table, self.experts, chosen, weights)
         else:
-            ops.moe_route(x, self.router, chosen, weights, self.score, self.renormalize, self.router_b)
+            ops.moe_route(x, self.router, chosen, weights, self.score, self.renormalize, self.router_b, self.correction_b, self.groups,
+                          self.keep_groups, self.weight_scale)
         ops.stage_name = "experts"
         ops.moe_experts(x, self.w_gate_up, self.w_down, chosen, weights, residual, self.weight_on == "input", ws, self.interleaved,
-                        self.activation, self.form)
+                        self.activation, self.form, self.identity)
         if self.shared is not None:
             self.shared.forward(x, ctx, residual)
         return None

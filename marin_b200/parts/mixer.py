@@ -46,6 +46,8 @@ class PagedKV:
     pooled: int = 0
     #: with ``pooled``: how many of the latest positions a reader looks at one by one (what lies before them, by blocks)
     pooled_window: int = 0
+    #: with ``window``: the sequence's first positions that stay visible however old they are (their pages are never given back)
+    keep_first: int = 0
 
     def __post_init__(self):
         if self.pooled and self.window is not None:
@@ -69,7 +71,7 @@ class PagedKV:
 
     def bytes_read(self, context: int, dtype: torch.dtype) -> int:
         """Bytes one decoded token reads of a sequence of ``context`` positions."""
-        kept = context if self.window is None else min(context, self.window)
+        kept = context if self.window is None else min(context, self.window + self.keep_first)
         if self.pooled and self.pooled_window:
             kept = min(context, self.pooled_window) + max(0, context - self.pooled_window) // self.pooled
         return kept * self.bytes_per_token(dtype)
@@ -352,6 +354,10 @@ class SinkAttention(Mixer):
     learned ``lam`` (``first_of_mix`` says which a layer is; the first one's ``lam`` tensor is expected and unused).
     ``gate``: the heads' outputs are multiplied by ``sigmoid(x W_g^T)`` before the output projection.  One fused product
     makes q | k | v | g.
+
+    ``keep_first`` (with ``window``): the sequence's first positions are seen however old they are, at their true positions; their
+    pages are never given back.  ``softcap``: scores become ``softcap tanh(s / softcap)``, the sink's does not.  ``out_scale``: the
+    result times a number (applied to the heads' outputs, the output projection being linear).
     """
 
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "g": "g_proj.weight",
@@ -361,7 +367,8 @@ class SinkAttention(Mixer):
     def __init__(self, hidden: int, heads: int, kv_heads: int, head_dim: int, name: str, position: PartSpec,
                  v_head_dim: Optional[int] = None, scale: Optional[float] = None, bias: bool = False, qk_norm: Optional[str] = "head",
                  norm_eps: float = 1e-6, window: Optional[int] = None, chunk: Optional[int] = None, sink: bool = True,
-                 value_mix: Optional[str] = None, first_of_mix: bool = False, gate: bool = False, names=None):
+                 value_mix: Optional[str] = None, first_of_mix: bool = False, gate: bool = False, names=None, keep_first: int = 0,
+                 softcap: Optional[float] = None, out_scale: float = 1.0):
         self.hidden, self.heads, self.kv_heads, self.head_dim = int(hidden), int(heads), int(kv_heads), int(head_dim)
         if self.heads % self.kv_heads != 0:
             raise ValueError(f"{heads} heads cannot share {kv_heads} kv heads evenly")
@@ -372,6 +379,8 @@ class SinkAttention(Mixer):
         self.scale = float(scale) if scale is not None else 1.0 / math.sqrt(self.head_dim)
         self.window = int(window) if window else None
         self.chunk = int(chunk) if chunk else None
+        self.keep_first = int(keep_first) if self.window else 0
+        self.softcap, self.out_scale = float(softcap) if softcap else None, float(out_scale)
         self.sink, self.gate = bool(sink), bool(gate)
         self.learned_sink = sink == "learned"
         self.sink_logits = None
@@ -388,7 +397,7 @@ class SinkAttention(Mixer):
     def cache_need(self):
         # (a chunked mask never looks behind its chunk's start, but pages are not given back there: the keys a window
         # has passed are dropped by the cache manager, a chunk's are only skipped)
-        return PagedKV(self.kv_heads, self.head_dim, self.window, self.v_head_dim)
+        return PagedKV(self.kv_heads, self.head_dim, self.window, self.v_head_dim, keep_first=self.keep_first)
 
     def tensor_specs(self) -> List[TensorSpec]:
         h = self.hidden
@@ -428,7 +437,7 @@ class SinkAttention(Mixer):
         self.rt = rt
 
     def flops(self, tokens: int, pairs: int = 0) -> float:
-        w = self.window
+        w = self.window + self.keep_first if self.window else 0
         if w and tokens > w and pairs == tokens * (tokens + 1) // 2:
             pairs = w * (w + 1) // 2 + (tokens - w) * w          # one prompt from its first position: the window's pairs
         elif w:
@@ -439,11 +448,11 @@ class SinkAttention(Mixer):
         return ops.sink_attention_jobs(dtype, self.heads, self.kv_heads, self.head_dim, self.v_head_dim)
 
     def decode_plan_key(self):
-        return ("sink_attention", self.heads, self.kv_heads, self.head_dim, self.v_head_dim, self.chunk, self.window)
+        return ("sink_attention", self.heads, self.kv_heads, self.head_dim, self.v_head_dim, self.chunk, self.window, self.keep_first)
 
     def decode_plan(self, requests: int, span: int, rt: Runtime):
         return ops.sink_decode_plan(rt.dtype, requests, self.heads, self.kv_heads, self.head_dim, self.v_head_dim, span,
-                                    self.window or 0, self.chunk or 0)
+                                    self.window or 0, self.chunk or 0, keep_first=self.keep_first)
 
     def forward(self, x, ctx, cache, residual: torch.Tensor):
         T = x.shape[0]
@@ -473,7 +482,8 @@ class SinkAttention(Mixer):
         plans = ctx.decode_plans
         ops.attention_sink(q, cache.k, cache.v, out, ctx, cache.block_table, self.heads, self.kv_heads, self.head_dim, self.v_head_dim,
                            self.scale, self.window or 0, self.chunk or 0, self.sink, gate,
-                           plans.get(self.decode_plan_key()) if plans else None, self.sink_logits)
+                           plans.get(self.decode_plan_key()) if plans else None, self.sink_logits, self.keep_first, self.softcap or 0.0,
+                           self.out_scale)
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
         return None
@@ -805,3 +815,68 @@ class ShiftedMixer(Mixer):
         ops.shift_mix(x, last.state, ctx, last.slots, self.mu, shifted)
         ops.keep_last_row(x, last.state, ctx, last.slots)
         return self.inner.forward(shifted[0], ctx, inner_cache, residual)
+
+
+@register_mixer("parallel_mixers")
+class ParallelMixers(Mixer):
+    """Several mixers side by side on the same rows: ``sum_i scale_i mixer_i(x)``.  ``inner`` gives the mixers by name (their tensors lie in
+    ``<name>.<inner name>``), ``scales`` their weights; an inner mixer takes its weight as its parameter ``out_scale``.  What each keeps between
+    steps is kept side by side: ``cache_need`` answers the tuple of their needs, the view is the tuple of their views."""
+
+    def __init__(self, hidden: int, inner: Dict[str, PartSpec], name: str, scales: Optional[Dict[str, float]] = None):
+        self.hidden, self.name = int(hidden), name
+        scales = scales or {}
+        self.inner = [lookup("mixer", spec.kind)(name=f"{name}.{key}", out_scale=float(scales.get(key, 1.0)), **spec.params) for key, spec in inner.items()]
+        self.capturable = all(getattr(m, "capturable", True) for m in self.inner)
+        windows = {getattr(m, "window", None) for m in self.inner} - {None}
+        self.window = windows.pop() if len(windows) == 1 else None
+
+    def cache_need(self):
+        return tuple(m.cache_need() for m in self.inner)
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for m in self.inner for s in m.tensor_specs()]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        for m in self.inner:
+            m.load(tensors, rt)
+        self.rt = rt
+
+    def bytes_read(self, tokens: int, dtype) -> int:
+        return sum(m.bytes_read(tokens, dtype) for m in self.inner)
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return sum(m.flops(tokens, pairs) for m in self.inner)
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        jobs: Dict[str, tuple] = {}
+        for m in self.inner:
+            jobs.update(m.kernel_jobs(dtype))
+        return jobs
+
+    def workspace_per_token(self, dtype) -> int:
+        return sum(m.workspace_per_token(dtype) for m in self.inner if hasattr(m, "workspace_per_token"))
+
+    def decode_plan_key(self):
+        keys = tuple(m.decode_plan_key() for m in self.inner)
+        return ("parallel_mixers", keys) if any(k is not None for k in keys) else None
+
+    def decode_plan(self, requests: int, span: int, rt: Runtime):
+        """The inner mixers' plans by their own keys."""
+        plans = {}
+        for m in self.inner:
+            key = m.decode_plan_key()
+            plan = m.decode_plan(requests, span, rt) if key is not None else None
+            if plan is not None:
+                plans[key] = plan
+        return plans or None
+
+    def forward(self, x, ctx, cache, residual: torch.Tensor):
+        own = ctx.decode_plans.get(self.decode_plan_key()) if ctx.decode_plans else None
+        outer = ctx.decode_plans
+        if own:
+            ctx.decode_plans = dict(outer, **own)
+        for m, view in zip(self.inner, cache):
+            m.forward(x, ctx, view, residual)
+        ctx.decode_plans = outer
+        return None

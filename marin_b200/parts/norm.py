@@ -69,3 +69,31 @@ class DynamicTanh(Part):
         """``x`` float32 ``[rows, dim]`` → ``out`` (float32 or bfloat16) ``[rows, dim]``."""
         ops.dynamic_tanh(x, self.weight, self.bias, self.alpha, out)
         return out
+
+
+@register_norm("layernorm")
+class LayerNorm(Part):
+    """``y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b`` over the last axis, sums in float32.  ``names`` gives the tensors' names
+    inside ``name`` (weight, offset; "" names the tensor ``name`` itself); ``bias=False`` leaves the offset out."""
+
+    kind = "layer"
+
+    def __init__(self, dim: int, eps: float, name: str, bias: bool = True, names=("weight", "bias")):
+        self.dim, self.eps, self.name, self.has_bias = int(dim), float(eps), name, bool(bias)
+        self.weight_name, self.bias_name = (f"{name}.{part}" if part else name for part in names)
+        self.weight = self.bias = None
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [TensorSpec(self.weight_name, (self.dim,), "norm")] + ([TensorSpec(self.bias_name, (self.dim,), "bias")] if self.has_bias else [])
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.weight = rt.f32(tensors.pop(self.weight_name))
+        self.bias = rt.f32(tensors.pop(self.bias_name)) if self.has_bias else None
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        return ops.library_jobs("mb_layer_norm")
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """``x`` float32 ``[rows, dim]`` → ``out`` (float32 or bfloat16) ``[rows, dim]``."""
+        ops.layer_norm(x, self.weight, self.bias, self.eps, out)
+        return out

@@ -256,3 +256,142 @@ class Mamba2(Mixer):
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
         return None
+
+
+@register_mixer("delta_rule")
+class DeltaRule(Mixer):
+    """A gated delta rule (Yang, Kautz, Hatamizadeh, "Gated Delta Networks: Improving Mamba2 with Delta Rule").
+
+    ``q = W_q x``, ``k = W_k x`` (``kv_heads`` x ``dim``), ``v = W_v x`` (``heads`` x ``vdim``; head ``h`` uses q/k head ``h // (heads /
+    kv_heads)``), each through a causal convolution per channel of ``taps`` taps (weight ``[channels, taps]``, the last column on the current
+    token) and silu; q and k divided by ``sqrt(sum of squares + 1e-6)`` per head, q also times ``dim^(-1/2)``.  Per head, with ``beta = sigmoid(W_b x)``:
+    ``S <- g S``, ``u = beta (v - S^T k)``, ``S <- S + k u^T``, ``o = S^T q`` (``S`` ``dim`` x ``vdim``).
+
+    ``decay`` "head": ``g = exp(-exp(A_log_h) softplus(W_a x + dt_bias))``, one per head; "channel": one per head and key channel (it multiplies
+    that channel's row of ``S``), its argument out of two matrices, ``W_a2 (W_a1 x) + dt_bias`` with ``decay_rank`` numbers between.  Each head's ``o`` is
+    divided by its root mean square over ``vdim`` (``norm_eps`` under the root), times a weight ``[vdim]``, times ``gate`` ("silu" or "sigmoid") of ``W_g
+    x`` or, with ``gate_rank``, of ``W_g2 (W_g1 x)``; then ``out_scale`` and ``W_o`` into the residual.
+
+    A request's state is the matrices of all heads (float32) and the convolution's latest inputs (a ring of ``taps`` rows): two needs."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "b": "b", "a": "a", "a1": "a1", "a2": "a2", "dt_bias": "dt_bias", "rate": "A_log", "g": "g", "g1": "g1",
+             "g2": "g2", "norm": "norm", "o": "o", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}
+
+    def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, name: str, decay: str = "head",
+                 decay_rank: Optional[int] = None, gate: str = "silu", gate_rank: Optional[int] = None, norm_eps: float = 1e-6, names=None,
+                 out_scale: float = 1.0):
+        self.hidden, self.heads, self.kv_heads, self.dim, self.vdim, self.taps = (int(v) for v in (hidden, heads, kv_heads, dim, vdim, taps))
+        self.name, self.decay, self.gate = name, decay, gate
+        self.decay_rank, self.gate_rank = int(decay_rank) if decay_rank else None, int(gate_rank) if gate_rank else None
+        self.norm_eps, self.out_scale = float(norm_eps), float(out_scale)
+        if self.heads % self.kv_heads != 0:
+            raise ValueError(f"delta_rule: {heads} heads cannot share {kv_heads} q/k heads evenly")
+        if decay not in ("head", "channel") or gate not in ops.DELTA_GATES or (decay == "channel") != (self.decay_rank is not None):
+            raise ValueError(f"delta_rule: decay {decay!r} (rank {decay_rank}) / gate {gate!r}")
+        if self.dim > 256 or self.taps > 64:
+            raise ValueError("delta_rule: key heads above 256 or more than 64 taps are not supported")
+        self.names = dict(self.NAMES, **(names or {}))
+        self.qk, self.hv = self.kv_heads * self.dim, self.heads * self.vdim
+        self.channels = 2 * self.qk + self.hv
+        self.decays = self.heads * self.dim if decay == "channel" else self.heads
+        self.w_in = self.w_low = self.w_high = self.w_o = None
+
+    def _n(self, key: str) -> str:
+        return f"{self.name}.{self.names[key]}"
+
+    def cache_need(self):
+        return (StateNeed((self.heads, self.dim, self.vdim), torch.float32), StateNeed((self.taps, self.channels), torch.float32))
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        h, hv, n = self.hidden, self.hv, self.decays
+        specs = []
+        for p, rows in (("q", self.qk), ("k", self.qk), ("v", hv)):
+            specs += [TensorSpec(self._n(p), (rows, h)), TensorSpec(self._n(f"{p}_conv"), (rows, self.taps), "bias", 1.0 / self.taps)]
+        specs += [TensorSpec(self._n("b"), (self.heads, h)), TensorSpec(self._n("rate"), (self.heads,), "bias"),
+                  TensorSpec(self._n("norm"), (self.vdim,), "norm"), TensorSpec(self._n("dt_bias"), (n,), "bias"), TensorSpec(self._n("o"), (h, hv))]
+        for low, high, whole, rank, rows in (("a1", "a2", "a", self.decay_rank, n), ("g1", "g2", "g", self.gate_rank, hv)):
+            specs += [TensorSpec(self._n(low), (rank, h)), TensorSpec(self._n(high), (rows, rank))] if rank else [TensorSpec(self._n(whole), (rows, h))]
+        return specs
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        # One product of the layer's input: q | k | v, then whatever gates and decays come straight from it, then beta (blocks padded to
+        # multiples of 8 columns, so that every kernel can take them by 16-byte loads).  Small products of two matrices: their first
+        # matrices are one product, their second ones a block-diagonal one over its result.
+        blocks: Dict[str, torch.Tensor] = {"qkv": torch.cat([tensors.pop(self._n(p)) for p in "qkv"], dim=0)}
+        low: Dict[str, tuple] = {}
+        for first, second, whole, rank in (("g1", "g2", "g", self.gate_rank), ("a1", "a2", "a", self.decay_rank)):
+            if rank:
+                low[whole] = (tensors.pop(self._n(first)), tensors.pop(self._n(second)))
+            else:
+                blocks[whole] = tensors.pop(self._n(whole))
+        blocks["b"] = tensors.pop(self._n("b"))
+        self.cols, at, rows = {}, 0, []
+        for key, w in blocks.items():
+            self.cols[key] = (at, w.shape[0])
+            pad = -w.shape[0] % 8
+            rows += [w] + ([torch.zeros(pad, w.shape[1], dtype=w.dtype, device=w.device)] if pad else [])
+            at += w.shape[0] + pad
+        self.w_in = rt.matrix(torch.cat(rows, dim=0))
+        self.high_cols = {}
+        if low:
+            ranks = [-(-first.shape[0] // 8) * 8 for first, _ in low.values()]
+            first_all = torch.zeros(sum(ranks), self.hidden, dtype=next(iter(low.values()))[0].dtype)
+            second_all = torch.zeros(sum(second.shape[0] for _, second in low.values()), sum(ranks), dtype=first_all.dtype)
+            r = c = 0
+            for (whole, (first, second)), width in zip(low.items(), ranks):
+                first_all[r:r + first.shape[0]] = first.cpu()
+                second_all[c:c + second.shape[0], r:r + first.shape[0]] = second.cpu()
+                self.high_cols[whole] = (c, second.shape[0])
+                r, c = r + width, c + second.shape[0]
+            self.w_low, self.w_high = rt.matrix(first_all), rt.matrix(second_all)
+        self.conv_w = rt.f32(torch.cat([tensors.pop(self._n(f"{p}_conv")).to(torch.float32) for p in "qkv"], dim=0))
+        self.rate, self.dt_bias, self.norm_w = (rt.f32(tensors.pop(self._n(k))) for k in ("rate", "dt_bias", "norm"))
+        self.w_o = rt.matrix(tensors.pop(self._n("o")))
+        self.rt = rt
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return super().flops(tokens, pairs) + tokens * (8.0 * self.heads * self.dim * self.vdim + 2.0 * self.channels * self.taps)
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        return ops.delta_rule_jobs(dtype, self.dim, self.vdim)
+
+    def forward(self, x, ctx, cache, residual: torch.Tensor):
+        T = x.shape[0]
+        ws = ctx.workspace
+        H, G, d, dv = self.heads, self.kv_heads, self.dim, self.vdim
+        matrices, ring = cache
+        ops.stage_name = "q|k|v|b"
+        rows = ws.get("delta_rows", (T, self.w_in.shape[0]), x.dtype)
+        ops.gemm(x, self.w_in, rows)
+        high = None
+        if self.w_low is not None:
+            ops.stage_name = "decay, gate"
+            small = ws.get("delta_low", (T, self.w_low.shape[0]), x.dtype)
+            ops.gemm(x, self.w_low, small)
+            high = ws.get("delta_high", (T, self.w_high.shape[0]), x.dtype)
+            ops.gemm(small, self.w_high, high)
+
+        def block(key):
+            src, (at, n) = (high, self.high_cols[key]) if key in self.high_cols else (rows, self.cols[key])
+            return src[:, at:at + n]
+
+        inputs = ops.DeltaInputs(block("b"), block("a"), block("g"), self.rate, self.dt_bias)
+        qkv = block("qkv")
+        out = ws.get("delta_out", (T, self.hv), x.dtype)
+        ops.stage_name = "delta rule"
+        single = ctx.num_decode if ops.use_delta_single and ops.delta_single_supported(d, dv) else 0
+        if single:                                             # requests with one token each come first in the batch
+            ops.delta_single(qkv, self.conv_w, ring.state, inputs, matrices.state, ctx, matrices.slots, self.gate, self.norm_w, self.norm_eps,
+                             self.out_scale, out, single, H, G, d, dv)
+        if ctx.num_requests > single:
+            ops.stage_name = "convolution"
+            conv = ws.get("delta_conv", (T, self.channels), x.dtype)
+            ops.delta_conv(qkv, self.conv_w, ring.state, ctx, ring.slots, conv, single, single)
+            ops.stage_name = "delta rule"
+            o = ws.get("delta_o", (T, self.hv), torch.float32)
+            ops.delta_scan(conv, inputs, matrices.state, ctx, matrices.slots, o, H, G, d, dv, single)
+            ops.stage_name = "norm, gate"
+            ops.delta_norm(o, inputs.gate, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, H, dv, single)
+        ops.stage_name = "o"
+        ops.gemm(out, self.w_o, residual, accumulate=True)
+        return None
