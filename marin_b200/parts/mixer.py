@@ -875,7 +875,7 @@ class ParallelMixers(Mixer):
         own = ctx.decode_plans.get(self.decode_plan_key()) if ctx.decode_plans else None
         outer = ctx.decode_plans
         if own:
-            ctx.decode_plans = dict(outer, **own)
+            ctx.decode_plans = {**outer, **own}
         for m, view in zip(self.inner, cache):
             m.forward(x, ctx, view, residual)
         ctx.decode_plans = outer
