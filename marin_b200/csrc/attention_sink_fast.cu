@@ -1,12 +1,15 @@
 // bf16 softmax attention with a sink, a chunked mask or a window, value heads of their own width and an output gate, on the
 // tensor cores (mma.sync), compiled for one head layout:
 //   -DHEAD_DIM (keys and queries), -DV_DIM (values), -DGROUP (query heads per kv head); both sizes multiples of 16 up to 128.
-// A position i sees the keys j <= i with j >= lo(i) = max(i - window + 1 (window > 0), floor(i / chunk) chunk (chunk > 0), 0).
+// A position i sees the keys j <= i with j >= lo(i) = max(i - window + 1 (window > 0), floor(i / chunk) chunk (chunk > 0), 0) and the
+// sequence's first `keep` positions.  Scores may be capped, s <- cap tanh(s / cap); the sink's score is not.  The result is multiplied
+// by `out_scale`; output rows are `out_stride` elements apart.
 //   p_j = exp(s_j) / (sink + sum_j exp(s_j)), s_j = q_i . k_j * scale, sink = exp(b_h) (a key without a value whose score b_h is
 //   0 or a learned number per query head, not scaled) or 0;
 //   out_i = (sum_j p_j v_j) * sigmoid(gate_i) where a gate is given.
 // Scores, maxima and sums are float32 (in the exp2 domain); the weights are rounded to bf16 for the product with V.
-// Prompt portions: 64 queries x 64-key blocks per CTA, only the blocks between lo(first query) and the last query.
+// Prompt portions: 64 queries x 64-key blocks per CTA, only the blocks between lo(first query) and the last query and those of the
+// kept first positions before them.
 // Single tokens: the visible keys of a sequence split over CTAs, partial (max, sum, accumulator) merged by a second kernel
 // in chunk order, which also adds the sink and applies the gate.
 // K pages [page][kv_head][offset][HEAD_DIM], V pages [page][kv_head][offset][V_DIM].
@@ -55,18 +58,30 @@ __device__ __forceinline__ float ex2_approx(float x) {
 }
 __device__ __forceinline__ float sigmoid_of(float s) { return __fdividef(1.0f, 1.0f + ex2_approx(s * -LOG2E)); }
 
+// A score in log2 units, capped where cap > 0: tanh(x) = 1 - 2 / (1 + e^(2x)) from the fast exponential, whose absolute error of a
+// few 1e-7 times the cap stays far below the rounding of the score's own operands.
+__device__ __forceinline__ float score_log2(float dot, float scale, float cap, float inv_cap) {
+    const float s = dot * scale;
+    if (cap > 0.0f) return cap * LOG2E * (1.0f - __fdividef(2.0f, 1.0f + ex2_approx(s * inv_cap * (2.0f * LOG2E))));
+    return s * LOG2E;
+}
+
+// Blocks of kept first positions that lie wholly before block `first_block` (those from it on are walked anyway).
+__device__ __forceinline__ int kept_blocks(int keep, int first_block) { return min((keep + 63) / 64, first_block); }
+
 __device__ __forceinline__ int first_seen(int pos, int window, int chunk) {
     int lo = window > 0 ? max(0, pos - window + 1) : 0;
     if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
     return lo;
 }
 
-// The rows of one 64-key block of K and V (cp.async); keys outside [k_first, k_last] are zero (their pages may not exist).
+// The rows of one 64-key block of K and V (cp.async); keys outside [k_first, k_last] that are not kept first positions are zero
+// (their pages may not exist).
 // Two threads a row (128 threads, 64 rows), each taking every other 16-byte piece: the page look-up and the row's address
 // are worked out once a thread and block, and the copies that follow differ by constants.  (With one piece a thread and
 // turn, index arithmetic and look-ups were most of the kernel's instructions: 800 a warp and block, against 36 MMAs.)
 __device__ __forceinline__ void load_kv_block(bf16* dst_k, bf16* dst_v, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
-                                              const int* __restrict__ table, int K, int kh, int page_shift, int key0, int k_first, int k_last) {
+                                              const int* __restrict__ table, int K, int kh, int page_shift, int key0, int k_first, int k_last, int keep) {
 #ifdef V_IN_K
     constexpr int CK = D / 8, CV = 0;
 #else
@@ -76,7 +91,7 @@ __device__ __forceinline__ void load_kv_block(bf16* dst_k, bf16* dst_v, const bf
     const int key = key0 + row;
     bf16* dk = dst_k + row * LDK;
     bf16* dv = dst_v + row * LDV;
-    if (key <= k_last && key >= k_first) {
+    if (key <= k_last && (key >= k_first || key < keep)) {
         const int page_mask = (1 << page_shift) - 1;
 #ifdef V_IN_K
         const size_t slot = ((size_t)table[key >> page_shift] << page_shift) + (size_t)(key & page_mask);       // one kv head
@@ -108,7 +123,7 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache, bf16* __restrict__ out,
     const int* __restrict__ block_table, int max_pages, const int* __restrict__ cu_tokens, const int* __restrict__ seq_lens,
     int first_req, int K, int page_shift, float scale, int window, int chunk, int sink, const float* __restrict__ sink_logit,
-    const bf16* __restrict__ gate, int gate_stride) {
+    const bf16* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride) {
     PDL_ENTER_EARLY();
     q = pdl_fresh(q); k_cache = pdl_fresh(k_cache); v_cache = pdl_fresh(v_cache); gate = pdl_fresh(gate);
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -121,16 +136,17 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
 #endif
     const int H = K * GROUP;
     const int r = first_req + blockIdx.z, h = blockIdx.y, qt = gridDim.x - 1 - blockIdx.x;   // long tiles first
-    const int tok0 = cu_tokens[r], n = cu_tokens[r + 1] - tok0;
-    if (qt * BM >= n) return;
-    const int len = seq_lens[r], pos0 = len - n;
-    const int rows = min(BM, n - qt * BM);
+    const int tok0 = cu_tokens[r], count = cu_tokens[r + 1] - tok0;
+    if (qt * BM >= count) return;
+    const int len = seq_lens[r], pos0 = len - count;
+    const int rows = min(BM, count - qt * BM);
     const int q_first = pos0 + qt * BM, q_last = q_first + rows - 1;
     const int kh = h / GROUP;
     const int* table = block_table + (size_t)r * max_pages;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int k_first = first_seen(q_first, window, chunk);       // lo() never decreases with the position
     const int kb_first = k_first / BN, kb_last = q_last / BN;
+    const int kept = kept_blocks(keep, kb_first), blocks = kept + kb_last - kb_first + 1;      // block number n: n, or kb_first + n - kept
     {
         constexpr int CHUNKS = D / 8;
         for (int idx = threadIdx.x; idx < BM * CHUNKS; idx += 128) {
@@ -139,7 +155,7 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
             if (row < rows) cp_async16(d, q + ((size_t)(tok0 + qt * BM + row) * H + h) * D + c * 8);
             else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
         }
-        load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, kb_first * BN, k_first, q_last);
+        load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, kept > 0 ? 0 : kb_first * BN, k_first, q_last, keep);
         cp_async_commit();
     }
     cp_async_wait<0>();
@@ -151,17 +167,17 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
     const int row0 = warp * 16 + (lane >> 2);                 // this thread's rows: row0 and row0 + 8
     const int qp[2] = {q_first + row0, q_first + row0 + 8};
     const int lo[2] = {first_seen(qp[0], window, chunk), first_seen(qp[1], window, chunk)};
-    const float sl2 = scale * LOG2E;
+    const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
     // running maximum (log2 units) and this thread's share of the running sum, per row; the sink is a score (0 or the head's
     // learned number, not scaled) and a 1 in the sum
     float m_run[2], l_run[2];
     m_run[0] = m_run[1] = sink ? (sink_logit != nullptr ? sink_logit[h] * LOG2E : 0.0f) : -INFINITY;
     l_run[0] = l_run[1] = (sink && (lane & 3) == 0) ? 1.0f : 0.0f;
 
-    for (int kb = kb_first; kb <= kb_last; ++kb) {
-        const int key0 = kb * BN;
-        if (kb > kb_first) {                                   // the barrier at the end of the last block freed the buffers
-            load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, key0, k_first, q_last);
+    for (int n = 0; n < blocks; ++n) {
+        const int key0 = (n < kept ? n : kb_first + n - kept) * BN;
+        if (n > 0) {                                   // the barrier at the end of the last block freed the buffers
+            load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, key0, k_first, q_last, keep);
             cp_async_commit();
             cp_async_wait<0>();
             __syncthreads();
@@ -191,8 +207,8 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int rr = e >> 1, kj = key + (e & 1);
-                const float v = s[j][e] * sl2;
-                s[j][e] = (interior || (kj <= qp[rr] && kj >= lo[rr])) ? v : -INFINITY;
+                const float v = score_log2(s[j][e], scale, softcap, inv_cap);
+                s[j][e] = (interior || (kj <= qp[rr] && (kj >= lo[rr] || kj < keep))) ? v : -INFINITY;
                 mx[rr] = fmaxf(mx[rr], s[j][e]);
             }
         }
@@ -246,9 +262,9 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         const int row = row0 + 8 * rr;
         if (row < rows) {
-            const float inv = 1.0f / l;
+            const float inv = out_scale / l;
             const size_t t = (size_t)(tok0 + qt * BM + row);
-            bf16* dst = out + (t * H + h) * DV;
+            bf16* dst = out + t * out_stride + (size_t)h * DV;
             const bf16* grow = gate != nullptr ? gate + t * gate_stride + (size_t)h * DV : nullptr;
 #pragma unroll
             for (int i = 0; i < DV / 8; ++i) {
@@ -265,7 +281,8 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
 }
 
 // ---- single tokens: the visible keys of a sequence split over CTAs -------------------------------------------------------
-// CTA (chunk, kv head, request): keys [start + chunk * split, + split) where start = lo(pos) rounded down to a block of 64; the
+// CTA (chunk, kv head, request): a chunk is `split` consecutive keys of the list "blocks of kept first positions that lie before the
+// window's, then the keys from start on", start = lo(pos) rounded down to a block of 64; the
 // GROUP query heads of the kv head are rows 0..GROUP-1 of a 16-row tile (a thread holds row g of the tile's upper half and,
 // with more than 8 heads, row g + 8 of the lower: two running maxima and sums); warp w takes keys 16 w .. 16 w + 15 of every
 // block with a running (max, sum) of its own.  The four warps are merged in shared memory in warp order and written as the chunk's
@@ -287,7 +304,7 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
 __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache, float* __restrict__ part_acc,
     float* __restrict__ part_ml, const int* __restrict__ block_table, int max_pages, const int* __restrict__ seq_lens, int K,
-    int page_shift, float scale, int window, int chunk_size, int split) {
+    int page_shift, float scale, int window, int chunk_size, int split, int keep, float softcap) {
     PDL_ENTER();
     q = pdl_fresh(q); k_cache = pdl_fresh(k_cache); v_cache = pdl_fresh(v_cache);
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -299,8 +316,9 @@ __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
     const int len = seq_lens[r], pos = len - 1;
     if (len <= 0) return;
     const int lo = first_seen(pos, window, chunk_size);
-    const int c_begin = (lo / BN) * BN + chunk * split, c_end = min(len, c_begin + split);
-    if (c_begin >= len) return;
+    const int kept = kept_blocks(keep, lo / BN) * BN, behind = (lo / BN) * BN - kept;   // key number v of the list: v, or v + behind
+    const int c_begin = chunk * split, c_end = min(len - behind, c_begin + split);
+    if (c_begin >= len - behind) return;
     const int* table = block_table + (size_t)r * max_pages;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     {
@@ -317,21 +335,22 @@ __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f; }
     const int g = lane >> 2;                                   // this thread's row of the tile: a query head if g < GROUP
-    const float sl2 = scale * LOG2E;
+    const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
     float m_run = -INFINITY, l_run = 0.0f;
     float m_low = -INFINITY, l_low = 0.0f;                    // row g + 8 (used with more than 8 heads)
 #ifdef V_IN_K
-    load_kv_block(sK0, sK0, k_cache, v_cache, table, K, kh, page_shift, c_begin, lo, pos);
+    load_kv_block(sK0, sK0, k_cache, v_cache, table, K, kh, page_shift, c_begin < kept ? c_begin : c_begin + behind, lo, pos, keep);
     cp_async_commit();
     int stage = 0;
 #endif
-    for (int key0 = c_begin; key0 < c_end; key0 += BN) {
+    for (int v0 = c_begin; v0 < c_end; v0 += BN) {
+        const int key0 = v0 < kept ? v0 : v0 + behind;
 #ifdef V_IN_K
         bf16* sK = sK0 + stage * DEC_STAGE_ELEMS;
         bf16* sV = sK;
-        if (key0 + BN < c_end) {                               // the next block, into the buffer the last block's products have left
+        if (v0 + BN < c_end) {                               // the next block, into the buffer the last block's products have left
             bf16* next = sK0 + (stage ^ 1) * DEC_STAGE_ELEMS;
-            load_kv_block(next, next, k_cache, v_cache, table, K, kh, page_shift, key0 + BN, lo, pos);
+            load_kv_block(next, next, k_cache, v_cache, table, K, kh, page_shift, v0 + BN < kept ? v0 + BN : v0 + BN + behind, lo, pos, keep);
         }
         cp_async_commit();
         cp_async_wait<1>();                                    // all but the newest group: this block (and the queries) are here
@@ -339,7 +358,7 @@ __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
 #else
         bf16* sK = sK0;
         bf16* sV = sK + BN * LDK;
-        load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, key0, lo, pos);
+        load_kv_block(sK, sV, k_cache, v_cache, table, K, kh, page_shift, key0, lo, pos, keep);
         cp_async_commit();
         cp_async_wait<0>();
 #endif
@@ -361,11 +380,11 @@ __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
 #pragma unroll
             for (int e = 0; e < 2; ++e) {                      // elements 2 and 3 belong to rows 8..15
                 const int key = key0 + warp * 16 + j * 8 + 2 * (lane & 3) + e;
-                const bool seen = key <= pos && key >= lo;
-                s[j][e] = seen ? s[j][e] * sl2 : -INFINITY;
+                const bool seen = key <= pos && (key >= lo || key < keep);
+                s[j][e] = seen ? score_log2(s[j][e], scale, softcap, inv_cap) : -INFINITY;
                 mx = fmaxf(mx, s[j][e]);
                 if (DEC_LOWER) {
-                    s[j][2 + e] = seen ? s[j][2 + e] * sl2 : -INFINITY;
+                    s[j][2 + e] = seen ? score_log2(s[j][2 + e], scale, softcap, inv_cap) : -INFINITY;
                     mx_low = fmaxf(mx_low, s[j][2 + e]);
                 }
             }
@@ -472,7 +491,7 @@ __global__ void __launch_bounds__(128, 4) attn_sink_decode_kernel(
 __global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_kernel(
     const float* __restrict__ part_acc, const float* __restrict__ part_ml, const int* __restrict__ seq_lens, int split, int window,
     int chunk_size, int sink, const float* __restrict__ sink_logit, int R, int H, const bf16* __restrict__ gate, int gate_stride,
-    bf16* __restrict__ out) {
+    bf16* __restrict__ out, int keep, float out_scale, int out_stride) {
     PDL_ENTER();
     part_acc = pdl_fresh(part_acc); part_ml = pdl_fresh(part_ml); gate = pdl_fresh(gate);
     __shared__ float wgt[MG_MAX_CHUNKS], scratch[32];
@@ -480,8 +499,9 @@ __global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_kernel(
     const int len = seq_lens[r];
     if (len <= 0) return;
     const int pos = len - 1;
-    const int start = (first_seen(pos, window, chunk_size) / BN) * BN;
-    const int chunks = min((len - start + split - 1) / split, MG_MAX_CHUNKS);
+    const int first_block = first_seen(pos, window, chunk_size) / BN;
+    const int behind = (first_block - kept_blocks(keep, first_block)) * BN;
+    const int chunks = min((len - behind + split - 1) / split, MG_MAX_CHUNKS);
     const float s0 = sink_logit != nullptr ? sink_logit[h] * LOG2E : 0.0f;        // the sink's score in log2 units
     float mx = sink ? s0 : -INFINITY;
     for (int c = threadIdx.x; c < chunks; c += MG_THREADS) {
@@ -498,7 +518,7 @@ __global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_kernel(
         part = fmaf(part_ml[(((size_t)c * R + r) * H + h) * 2 + 1], f, part);
     }
     const float total = block_sum(part, scratch) + (sink ? exp2f(s0 - M) : 0.0f);       // (its barriers publish wgt)
-    const float inv = 1.0f / total;
+    const float inv = out_scale / total;
     for (int i = threadIdx.x; i < DV; i += MG_THREADS) {
         float a = 0.0f;
         int c = 0;
@@ -512,7 +532,7 @@ __global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_kernel(
         for (; c < chunks; ++c) a = fmaf(part_acc[(((size_t)c * R + r) * H + h) * DV + i], wgt[c], a);
         a *= inv;
         if (gate != nullptr) a *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)r * gate_stride + (size_t)h * DV + i])));
-        out[((size_t)r * H + h) * DV + i] = __float2bfloat16_rn(a);
+        out[(size_t)r * out_stride + (size_t)h * DV + i] = __float2bfloat16_rn(a);
     }
 }
 
@@ -529,36 +549,37 @@ MB_API int mb_attn_sink_layout(int* d, int* dv, int* group) { *d = D; *dv = DV; 
 // chunks * split covers the most keys a token sees plus one block.
 MB_API int mb_attn_sink_decode(const void* q, const void* k_cache, const void* v_cache, float* part_acc, float* part_ml,
                                const int* block_table, int max_pages, const int* seq_lens, int requests, int K, int page_size,
-                               float scale, int window, int chunk, int split, int chunks, cudaStream_t s) {
+                               float scale, int window, int chunk, int split, int chunks, int keep, float softcap, cudaStream_t s) {
     if (requests <= 0) return 0;
     const int shift = page_shift_of(page_size);
-    if (shift < 0 || split <= 0 || split % BN != 0 || chunks <= 0 || chunks > MG_MAX_CHUNKS || window < 0 || chunk < 0) return MB_ERR_BAD_SIZE;
+    if (shift < 0 || split <= 0 || split % BN != 0 || chunks <= 0 || chunks > MG_MAX_CHUNKS || window < 0 || chunk < 0 || keep < 0) return MB_ERR_BAD_SIZE;
     cudaFuncSetAttribute(attn_sink_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, DEC_SMEM);
     return launch_kernel(attn_sink_decode_kernel, dim3(chunks, K, requests), 128, DEC_SMEM, s, 0, (const bf16*)q, (const bf16*)k_cache,
-                         (const bf16*)v_cache, part_acc, part_ml, block_table, max_pages, seq_lens, K, shift, scale, window, chunk, split);
+                         (const bf16*)v_cache, part_acc, part_ml, block_table, max_pages, seq_lens, K, shift, scale, window, chunk, split, keep, softcap);
 }
 
 // The parts of every request merged in chunk order, with the sink and the gate: out bf16 [requests][K * GROUP][V_DIM].
 MB_API int mb_attn_sink_merge(const float* part_acc, const float* part_ml, void* out, const int* seq_lens, int requests, int K, int window,
-                              int chunk, int sink, const void* gate, int gate_stride, int split, const float* sink_logit, cudaStream_t s) {
+                              int chunk, int sink, const void* gate, int gate_stride, int split, const float* sink_logit, int keep, float out_scale,
+                              int out_stride, cudaStream_t s) {
     if (requests <= 0) return 0;
-    if (split <= 0) return MB_ERR_BAD_SIZE;
+    if (split <= 0 || keep < 0 || out_stride < K * GROUP * DV) return MB_ERR_BAD_SIZE;
     return launch_kernel(attn_sink_merge_kernel, requests * K * GROUP, MG_THREADS, 0, s, 0, (const float*)part_acc,
                          (const float*)part_ml, seq_lens, split, window, chunk, sink, sink_logit, requests, K * GROUP, (const bf16*)gate, gate_stride,
-                         (bf16*)out);
+                         (bf16*)out, keep, out_scale, out_stride);
 }
 
 // Prompt portions: requests first_req .. first_req + count - 1 of the step.
 MB_API int mb_attn_sink_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                 int max_pages, const int* cu_tokens, const int* seq_lens, int first_req, int count, int max_query_len,
                                 int K, int page_size, float scale, int window, int chunk, int sink, const void* gate, int gate_stride,
-                                const float* sink_logit, cudaStream_t s) {
+                                const float* sink_logit, int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
     if (count <= 0 || max_query_len <= 0) return 0;
     const int shift = page_shift_of(page_size);
-    if (shift < 0 || window < 0 || chunk < 0) return MB_ERR_BAD_SIZE;
+    if (shift < 0 || window < 0 || chunk < 0 || keep < 0 || out_stride < K * GROUP * DV || out_stride % 2 != 0) return MB_ERR_BAD_SIZE;
     cudaFuncSetAttribute(attn_sink_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
     dim3 grid((max_query_len + BM - 1) / BM, K * GROUP, count);
     return launch_kernel(attn_sink_prefill_kernel, grid, 128, PF_SMEM, s, 0, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
                          (bf16*)out, block_table, max_pages, cu_tokens, seq_lens, first_req, K, shift, scale, window, chunk, sink, sink_logit,
-                         (const bf16*)gate, gate_stride);
+                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
 }

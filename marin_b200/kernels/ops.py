@@ -1269,7 +1269,8 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     by ``out_scale``; ``out`` may be a column block of a wider buffer."""
     _need_cuda(q, k_cache, v_cache, block_table, sink_logits)
     assert out.is_cuda and out.stride(1) == 1
-    variant = keep_first > 0 or softcap > 0.0 or out_scale != 1.0 or out.stride(0) != H * dv
+    more = (_c_int(keep_first), _c_float(softcap), _c_float(out_scale), _c_int(out.stride(0)))
+    variant = keep_first > 0 or softcap > 0.0 or out_scale != 1.0 or out.stride(0) != H * dv        # (not in the tcgen05 kernel)
     T = q.shape[0]
     page_size = k_cache.shape[2]
     values_in_keys = v_cache.data_ptr() == k_cache.data_ptr()
@@ -1286,7 +1287,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     size = q.element_size()
     per_row = H * (d + (3 if gate is not None else 2) * dv) * size
     key_bytes = (d if values_in_keys else K * (d + dv)) * size      # what one cached position holds for this layer
-    if not variant and use_fast_sink_attention and fast_sink_attention_supported(q.dtype, H, K, d, dv, values_in_keys) and page_size & (page_size - 1) == 0:
+    if use_fast_sink_attention and fast_sink_attention_supported(q.dtype, H, K, d, dv, values_in_keys) and page_size & (page_size - 1) == 0:
         kv_heads = K
         if values_in_keys:
             # one kv head that every query head reads: a CTA takes as many query heads as the kernels group, and `K` counts
@@ -1297,7 +1298,8 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
         nd = ctx.num_decode
         if nd > 0:
             if plan is None:
-                plan = sink_decode_plan(q.dtype, nd, H, 1 if values_in_keys else K, d, dv, ctx.max_seq_len, window, chunk, values_in_keys)
+                plan = sink_decode_plan(q.dtype, nd, H, 1 if values_in_keys else K, d, dv, ctx.max_seq_len, window, chunk, values_in_keys,
+                                        keep_first)
             acc = ctx.workspace.get("sink_parts", (plan.chunks, nd, H, dv), torch.float32)
             ml = ctx.workspace.get("sink_part_sums", (plan.chunks, nd, H, 2), torch.float32)
             if launch_log is not None:
@@ -1305,16 +1307,16 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
                 _pending_cost["rows"], _pending_cost["window"] = "decode", window
             _check(lib.mb_attn_sink_decode(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(acc), _ptr(ml), _ptr(block_table),
                                            _c_int(max_pages), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(page_size), _c_float(scale),
-                                           _c_int(window), _c_int(chunk), _c_int(plan.split), _c_int(plan.chunks), _stream()),
+                                           _c_int(window), _c_int(chunk), _c_int(plan.split), _c_int(plan.chunks), _c_int(keep_first), _c_float(softcap), _stream()),
                    "attention (sink, decode)")
             _cost(_size(acc) + nd * H * dv * size * (2 if gate is not None else 1))
             _check(lib.mb_attn_sink_merge(_ptr(acc), _ptr(ml), _ptr(out), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(window),
                                           _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _c_int(plan.split), _ptr(sink_logits),
-                                          _stream()), "attention (sink, parts merged)")
+                                          _c_int(keep_first), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink, parts merged)")
         if ctx.num_requests > nd and launch_log is not None:
             _cost((T - nd) * per_row, 0.0, key_bytes, 2.0 * H * (d + dv))
             _pending_cost["rows"], _pending_cost["window"] = "prefill", window
-        if (ctx.num_requests > nd and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
+        if (ctx.num_requests > nd and not variant and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
                 and (gate is None or (gate.data_ptr() % 16 == 0 and gate_stride % 8 == 0))):
             # heads of 64 or 128 with values as wide: the tcgen05 kernel that plain causal attention uses takes the chunked
             # mask, the sink and the gate as parameters; over a shared latent one CTA per query head reads the one kv head's rows
@@ -1330,7 +1332,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
             _check(lib.mb_attn_sink_prefill(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
                                             _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
                                             _c_int(ctx.max_query_len), _c_int(K), _c_int(page_size), _c_float(scale), _c_int(window),
-                                            _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _ptr(sink_logits), _stream()),
+                                            _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _ptr(sink_logits), *more, _stream()),
                    "attention (sink, prefill)")
         return
     if launch_log is not None:
@@ -1339,8 +1341,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     _check(_lib("mb_attention_sink").mb_attention_sink(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _code(q), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(ctx.req_index),
         _ptr(ctx.positions), _c_int(T), _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_float(scale), _c_int(window),
-        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), _c_int(keep_first),
-        _c_float(softcap), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink)")
+        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), *more, _stream()), "attention (sink)")
 
 
 #: bf16 sink attention goes to the tensor-core kernels where the head layout allows (False: always the plain kernel)
