@@ -2102,5 +2102,59 @@ def delta_single(qkv: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, in
         "delta rule (single tokens)")
 
 
+#: prompt portions of a bf16 delta rule run 64 tokens at a time on the tensor cores where the head layout allows (False: token by token)
+use_chunked_delta_rule = True
+#: the longest portion of a step must have more tokens than this for it: a chunk costs the same however few of its tokens are there
+DELTA_CHUNKED_FROM = 8
+
+
+def delta_chunked_supported(dtype, d: int, dv: int) -> bool:
+    return dtype == torch.bfloat16 and d % 16 == 0 and 16 <= d <= 128 and dv % 16 == 0
+
+
+def _delta_slice(dv: int) -> int:
+    """Value channels a CTA of the walk takes (its columns of the state are independent of the others)."""
+    return 32 if dv % 32 == 0 else 16
+
+
+def _delta_chunked_job(d: int, dv: int) -> tuple:
+    return (["delta_rule_chunked.cu"], [f"QK_DIM={d}", f"V_SLICE={_delta_slice(dv)}"])
+
+
+def delta_chunk_bytes(d: int, dv: int) -> int:
+    """Scratch memory of a chunk of 64 tokens and a head between the two kernels of the chunked form."""
+    return (6 * 64 * d + 2 * 64 * 64) * 2 + (64 * dv + d) * 4
+
+
+def delta_chunked(qkv: torch.Tensor, inp: DeltaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, o: torch.Tensor, H: int, G: int, d: int, dv: int,
+                  first_req: int = 0, first_token: int = 0) -> None:
+    """The same recurrence as ``delta_scan``, 64 tokens at a time on the tensor cores: what does not depend on the state for all chunks and
+    heads side by side, then the chunks of a request in order (the state and every float32 factor split into two bf16 numbers where they
+    are operands)."""
+    _need_cuda(qkv, state, o, slots)
+    T = qkv.shape[0]
+    assert qkv.dtype == torch.bfloat16 and qkv.shape[1] == 2 * G * d + H * dv and tuple(state.shape[1:]) == (H, d, dv)
+    assert state.dtype == o.dtype == torch.float32 and tuple(o.shape) == (T, H * dv)
+    R, rows = ctx.num_requests - first_req, T - first_token
+    chunks = rows // 64 + R                               # at most: room for a partial chunk per request
+    planes = ctx.workspace.get("delta_planes", (chunks * H, 6 * 64 * d + 2 * 64 * 64), torch.bfloat16)
+    floats = ctx.workspace.get("delta_floats", (chunks * H, 64 * dv + d), torch.float32)
+    lib = build.load(f"mb_delta_rule_chunked_d{d}_v{_delta_slice(dv)}", *_delta_chunked_job(d, dv))
+    scratch = float(rows) / 64 * H * delta_chunk_bytes(d, dv)
+    for which, what in ((0, "delta rule (chunks prepared)"), (1, "delta rule (chunks walked)")):
+        if which == 0:
+            _cost(rows * qkv.shape[1] * 2 + scratch, rows * H * 64.0 * (2 * d + d + dv))
+        else:
+            _cost(scratch + rows * H * dv * 4 + 2.0 * R * H * d * dv * 4, rows * H * dv * (6.0 * d + 64.0))
+        _check(lib.mb_delta_chunked(_ptr(qkv), *_delta_args(inp, T, H, d, qkv.dtype), _ptr(state), _ptr(ctx.cu_tokens), _ptr(slots), _ptr(o),
+                                    _ptr(planes), _ptr(floats), _c_int(first_req), _c_int(ctx.num_requests), _c_int(ctx.max_query_len), _c_int(H),
+                                    _c_int(G), _c_int(dv), _c_int(which), _stream()), what)
+
+
 def delta_rule_jobs(dtype, d: int, dv: int) -> dict:
-    return library_jobs("mb_delta_rule")
+    """The kernels a delta rule of this head layout runs: any size token by token, single tokens and, where the layout allows, the
+    chunked tensor-core kernels for prompt portions."""
+    jobs = library_jobs("mb_delta_rule")
+    if use_chunked_delta_rule and delta_chunked_supported(dtype, d, dv):
+        jobs[f"mb_delta_rule_chunked_d{d}_v{_delta_slice(dv)}"] = _delta_chunked_job(d, dv)
+    return jobs

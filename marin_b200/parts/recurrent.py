@@ -12,7 +12,7 @@ from typing import Dict, List, Optional, Sequence
 import torch
 
 from ..kernels import ops
-from .base import Runtime
+from .base import Runtime, element_size
 from .mixer import Mixer, StateNeed
 from .registry import register_mixer
 from .spec import TensorSpec
@@ -355,6 +355,12 @@ class DeltaRule(Mixer):
     def kernel_jobs(self, dtype) -> Dict[str, tuple]:
         return ops.delta_rule_jobs(dtype, self.dim, self.vdim)
 
+    def workspace_per_token(self, dtype) -> int:
+        """Bytes a step keeps per token beside the products' rows: the convolution's output, the heads' sums and, in chunks of 64 tokens,
+        what the two chunked kernels hand over."""
+        chunked = self.heads * ops.delta_chunk_bytes(self.dim, self.vdim) // 64 if ops.delta_chunked_supported(dtype, self.dim, self.vdim) else 0
+        return self.channels * element_size(dtype) + 4 * self.hv + chunked
+
     def forward(self, x, ctx, cache, residual: torch.Tensor):
         T = x.shape[0]
         ws = ctx.workspace
@@ -389,7 +395,11 @@ class DeltaRule(Mixer):
             ops.delta_conv(qkv, self.conv_w, ring.state, ctx, ring.slots, conv, single, single)
             ops.stage_name = "delta rule"
             o = ws.get("delta_o", (T, self.hv), torch.float32)
-            ops.delta_scan(conv, inputs, matrices.state, ctx, matrices.slots, o, H, G, d, dv, single)
+            if (ops.use_chunked_delta_rule and ops.delta_chunked_supported(x.dtype, d, dv) and self.channels % 8 == 0
+                    and ctx.max_query_len > ops.DELTA_CHUNKED_FROM):
+                ops.delta_chunked(conv, inputs, matrices.state, ctx, matrices.slots, o, H, G, d, dv, single, single)
+            else:
+                ops.delta_scan(conv, inputs, matrices.state, ctx, matrices.slots, o, H, G, d, dv, single)
             ops.stage_name = "norm, gate"
             ops.delta_norm(o, inputs.gate, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, H, dv, single)
         ops.stage_name = "o"
