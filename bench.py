@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, with their fractions of roofline.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers N] [--impl ours|reference]
-    python bench.py --arch lakulix|fegarax|nirotar|vogunex [--model 4b|8b|14b] [--layers 12] [--batch 8] [--profile]
+    python bench.py --arch lakulix|fegarax|nirotar|vogunex|pununex [--model 4b|8b|14b] [--layers 12] [--batch 8] [--profile]
 
 The default run has the layer sizes of the Qwen3-4B layout with random bfloat16 weights, a batch of 8
 sequences and a context of 4096 positions (the last timed step reaches it).  A "step" is one decode
@@ -399,6 +399,31 @@ def vogunex_layout(raw: dict, layers: int) -> dict:
             "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": kinds[i % 4][2]} for i in range(layers)]}
 
 
+PUNUNEX_LAYERS = ("in turn: attention with the layout's heads (a window of 1,024 positions and the first 4 kept, no rotation, scores capped, a learned "
+                  "sink) beside a gated delta rule (heads of 128 x 128 filling the width, four taps, a decay per key channel and a sigmoid gate, each "
+                  "out of two matrices of rank 128) with a dense relu-gated feed-forward of the layout's width; a gated delta rule alone (as many "
+                  "heads, a decay per head, a silu gate) with experts; the parallel layer with experts; the delta rule with experts.  8 gated experts of "
+                  "3/8 of the layout's feed-forward width in 2 groups of which both are kept, no identity outputs (every token activates as many "
+                  "weights as in the other designs), 2 chosen, and a shared expert of a quarter of it")
+
+
+def pununex_layout(raw: dict, layers: int) -> dict:
+    """A Pununex configuration at a Qwen3 layout's sizes: the same width, vocabulary and attention heads; feed-forwards that
+    activate as many weights per token as the layout's dense gated one."""
+    head, heads, width, ff = raw["head_dim"], raw["num_attention_heads"], raw["hidden_size"], raw["intermediate_size"]
+    attention = {"heads": heads, "kv_heads": raw["num_key_value_heads"], "dim": head, "vdim": head, "scale": head ** -0.5, "softcap": 50.0,
+                 "mask": {"size": 1024, "keep_first": 4}}
+    delta = {"heads": width // 128, "kv_heads": width // 128, "dim": 128, "vdim": 128, "conv": 4}
+    parallel = {"left": attention, "right": dict(delta, decay_rank=128, gate_rank=128), "left_scale": 0.6, "right_scale": 0.4}
+    expert = ff * 3 // 8 // 64 * 64
+    moe = {"kind": "moe", "expert": {"ff": expert}, "router": {"experts": 8, "top": 2, "identity": 0, "scale": 1.0, "groups": {"count": 2, "keep": 2}},
+           "shared": {"ff": (ff - 2 * expert) // 64 * 64}}
+    kinds = [("parallel", parallel, {"kind": "dense", "ff": ff}), ("delta", delta, moe), ("parallel", parallel, moe), ("delta", delta, moe)]
+    return {"architecture": "Pununex", "vocab": raw["vocab_size"], "width": width, "norm": {"eps": 1e-6}, "max_positions": 2 * CONTEXT,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}},
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": kinds[i % 4][2]} for i in range(layers)]}
+
+
 def arch_mode(args, pk, arch: str) -> int:
     """Decode and prompt throughput of another architecture at a Qwen3 layout's sizes, and of that Qwen3 layout at the same
     depth, with their fractions of roofline: one JSON line.  With --profile: the architecture's stage tables."""
@@ -407,7 +432,7 @@ def arch_mode(args, pk, arch: str) -> int:
     import torch
 
     from marin_b200 import Engine
-    from marin_b200.config import FegaraxConfig, LakulixConfig, NirotarConfig, Qwen3Config, VogunexConfig
+    from marin_b200.config import FegaraxConfig, LakulixConfig, NirotarConfig, PununexConfig, Qwen3Config, VogunexConfig
 
     layers = args.layers or 12
     raw = dict(LAYOUTS[args.model], num_hidden_layers=layers)
@@ -415,8 +440,11 @@ def arch_mode(args, pk, arch: str) -> int:
     title = arch.capitalize()
     # the model it is measured beside: the Qwen3 layout, or for Nirotar the engine's closest model, Fegarax at that layout's sizes
     # (for Vogunex: Nirotar, whose windowed and latent attention and experts with a shared one are the nearest kernels)
-    beside = "fegarax" if arch == "nirotar" else "nirotar" if arch == "vogunex" else "qwen3"
-    if arch == "vogunex":
+    # (for Pununex: Vogunex, which keeps recurrent states beside a window of keys and has experts with a shared one)
+    beside = {"nirotar": "fegarax", "vogunex": "nirotar", "pununex": "vogunex"}.get(arch, "qwen3")
+    if arch == "pununex":
+        other = PununexConfig.from_dict(pununex_layout(raw, layers))
+    elif arch == "vogunex":
         other = VogunexConfig.from_dict(vogunex_layout(raw, layers))
     elif arch == "lakulix":
         other = LakulixConfig.from_dict(lakulix_layout(raw, layers))
@@ -425,7 +453,8 @@ def arch_mode(args, pk, arch: str) -> int:
     else:
         other = NirotarConfig.from_dict(nirotar_layout(raw, layers))
     arms = {arch: other, beside: FegaraxConfig.from_dict(fegarax_layout(raw, layers)) if beside == "fegarax" else
-            NirotarConfig.from_dict(nirotar_layout(raw, layers)) if beside == "nirotar" else Qwen3Config.from_dict(raw)}
+            NirotarConfig.from_dict(nirotar_layout(raw, layers)) if beside == "nirotar" else
+            VogunexConfig.from_dict(vogunex_layout(raw, layers)) if beside == "vogunex" else Qwen3Config.from_dict(raw)}
     out = {}
     for name, cfg in arms.items():
         if args.profile and name != arch:
@@ -462,13 +491,14 @@ def arch_mode(args, pk, arch: str) -> int:
         gc.collect()
         torch.cuda.empty_cache()
     print(json.dumps({
-        "metric": f"{title} beside the {'Fegarax layers at the ' if beside == 'fegarax' else 'Nirotar layers at the ' if beside == 'nirotar' else ''}Qwen3-{args.model.upper()} layout at equal width, depth and vocabulary: decode tok/s at batch {args.batch} "
+        "metric": f"{title} beside the {beside.capitalize() + ' layers at the ' if beside != 'qwen3' else ''}Qwen3-{args.model.upper()} layout at equal width, depth and vocabulary: decode tok/s at batch {args.batch} "
                   f"(context {CONTEXT}), prefill tok/s at {PREFILL_TOKENS} tokens, fractions of roofline",
         "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": warmup, "dtype": "bf16", "higher_is_better": True,
         "data": "synthetic (uniform random token ids, seeded random weights)", "peaks": pk,
         "config": {"layers": layers, "width": raw["hidden_size"], "ff": raw["intermediate_size"], "vocab": raw["vocab_size"],
                    "global_batch": args.batch, "seq_len": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "kv_block": PAGE,
                    f"{arch}_layers": FEGARAX_LAYERS if arch == "fegarax" else NIROTAR_LAYERS if arch == "nirotar" else VOGUNEX_LAYERS if arch == "vogunex" else
+                   PUNUNEX_LAYERS if arch == "pununex" else
                    "lightning (heads of 128 x 128), attention (the layout's heads), wkv (heads of 64) in turn, a dense feed-forward in each",
                    "l2": "inputs larger than L2 (weights read per step exceed 126 MB)"},
         arch: out[arch], beside: out[beside], "impl": "ours"}))
@@ -496,9 +526,9 @@ def main() -> int:
     ap.add_argument("--model", default="4b", choices=sorted(LAYOUTS), help="layer sizes: Qwen3-4B (the default), 8B or 14B layout")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length the last timed decode step reaches (default 4096)")
     ap.add_argument("--profile", action="store_true", help="print where a step's time goes, stage by stage, instead of the JSON line")
-    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "lakulix", "fegarax", "nirotar", "vogunex"],
+    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "lakulix", "fegarax", "nirotar", "vogunex", "pununex"],
                     help="qwen3: the default workload; lakulix, fegarax: that architecture at the layout's sizes beside the Qwen3 layout of "
-                         "equal size; nirotar: beside the Fegarax layers at that layout's sizes; vogunex: beside the Nirotar layers at those sizes")
+                         "equal size; nirotar: beside the Fegarax layers at that layout's sizes; vogunex: beside the Nirotar layers at those sizes; pununex: beside the Vogunex layers")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()

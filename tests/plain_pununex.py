@@ -143,7 +143,7 @@ def relu(x: torch.Tensor) -> torch.Tensor:
 def route(h: torch.Tensor, t: Dict[str, torch.Tensor], name: str, router: dict):
     """Per row: the chosen outputs of the router (real experts first, then identity experts), their weights, and how far the
     choice is from falling otherwise (the smaller of the gap between the last kept and the first dropped group and the gap
-    between the last chosen and the first passed-over output among the kept groups, in units of the scores' size)."""
+    between the last chosen and the first passed-over output among the kept groups)."""
     top, groups = router["top"], router.get("groups") or {"count": 1, "keep": 1}
     s = torch.softmax(h @ t[f"{name}.router"].T, dim=-1)
     choice = s + t[f"{name}.correction"] if f"{name}.correction" in t else s
@@ -165,7 +165,7 @@ def route(h: torch.Tensor, t: Dict[str, torch.Tensor], name: str, router: dict):
         w = s[i, picked]
         chosen.append(picked)
         weights.append(w / (w.sum() + 1e-20) * router["scale"])
-        margins.append(gap * E)
+        margins.append(gap)
     return chosen, weights, torch.tensor(margins, dtype=F)
 
 
