@@ -25,6 +25,8 @@
 // wait.  The rows read a block's 64 scores twice, each time with one load of 64 columns; keeping them in registers
 // instead takes the thread to 128 registers with spills and is slower, and two threads per row, each with half of
 // the keys, meet at a barrier every block and are slower too: 1,800 cycles.)
+// The sequence's first `keep` positions may stay visible behind a window or chunk: their blocks come before the window's in the list
+// of blocks a tile walks.  Scores may be capped, s <- cap tanh(s / cap) (an instantiation of its own: CAP); the sink's is not.
 // Two CTAs fit an SM: one's softmax overlaps the other's MMAs.  Needs pages of at least 16 positions.  Waits are
 // bounded and record a code in *error_flag.
 // The mma.sync kernel in attention_fast.cu is the fallback and the plain twin (the reference's counterpart:
@@ -213,11 +215,19 @@ __device__ __forceinline__ int first_seen(int pos, int window, int chunk) {
     return lo;
 }
 
+// A capped score: cap tanh(x) with x = dot * scale / cap.  Where every |x| of a block is at most 0.5, tanh(x) = x P(x^2) with a cubic
+// P fitted there by least squares (relative error 6e-7, which times a score of half the cap stays far below its operands' rounding);
+// else from the fast exponential.
+#define TA_CAP_SMALL 0.5f
+__device__ __forceinline__ float tanh_any(float x) { return 1.0f - __fdividef(2.0f, 1.0f + ta_exp2(x * 2.8853900817779268f)); }
+
+template <bool CAP>
 __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
     bf16* __restrict__ out, const int* __restrict__ block_table, int max_pages, const int* __restrict__ cu_tokens,
     const int* __restrict__ seq_lens, int first_req, int K, int page_shift, float scale, int window, int* __restrict__ error_flag,
-    int box_rows, int chunk, int sink, const float* __restrict__ sink_logit, const bf16* __restrict__ gate, int gate_stride) {
+    int box_rows, int chunk, int sink, const float* __restrict__ sink_logit, const bf16* __restrict__ gate, int gate_stride, int keep,
+    float softcap, float out_scale, int out_stride) {
     extern __shared__ __align__(1024) uint8_t smem[];     // the swizzled tiles need 1024-byte alignment (checked below)
     uint8_t* sQ = smem;
     uint8_t* sKV = sQ + TA_Q_BYTES;                       // [buffer][K then V][half][64 rows][128 B]
@@ -235,7 +245,6 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     volatile int* abort = (volatile int*)(tmem_slot + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     PDL_ENTER_EARLY();
-    const int H = K * GROUP;
     const int r = first_req + blockIdx.z, h = blockIdx.y, qt = gridDim.x - 1 - blockIdx.x;   // long tiles first
     const int tok0 = cu_tokens[r], n = cu_tokens[r + 1] - tok0;
     if (qt * TA_BM >= n) return;                           // nothing to do here (before any tensor memory is taken)
@@ -259,7 +268,8 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     const int k_lo = first_seen(q_first, window, chunk);   // the first key a position sees never decreases with the position
     const int kh = h / GROUP;
     const int kb_first = k_lo / TA_BN, kb_last = q_last / TA_BN;
-    const int nblk = kb_last - kb_first + 1;
+    const int kept = min((keep + TA_BN - 1) / TA_BN, kb_first);          // blocks of kept first positions before the others
+    const int nblk = kept + kb_last - kb_first + 1;
     // the page ids of this tile's keys, copied once: the issuer must not wait for global memory between two MMAs
     __shared__ int s_pages[TA_PAGE_CACHE];
     const int page_first = (kb_first * TA_BN) >> page_shift;
@@ -276,7 +286,11 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     // the many CTAs that read the same keys and values (the query tiles of a request, the heads of a group) do not
     // all ask the L2 for the same lines at the same moment.
     const int rot = (int)(((unsigned)(h * gridDim.x + qt) * 37u) % (unsigned)nblk);
-    auto block_of = [&](int i) { const int j = i + rot; return kb_first + (j >= nblk ? j - nblk : j); };
+    auto block_of = [&](int i) {
+        int j = i + rot;
+        j = j >= nblk ? j - nblk : j;
+        return j < kept ? j : kb_first + j - kept;
+    };
 
     if (warp == 5 || (warp == 6 && !TA_V_IN_K)) {
         // ---- the loader warps: warp 5 asks for Q once and then for every block of K, warp 6 for every block of V, each
@@ -295,7 +309,7 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
             if (g >= TA_BN || j >= nblk) return 0;
             const int key = block_of(j) * TA_BN + g;
             const int pg = (key >> page_shift) - page_first;
-            const int page_id = pg < TA_PAGE_CACHE ? s_pages[pg] : table[min(key >> page_shift, max_pages - 1)];
+            const int page_id = (pg >= 0 && pg < TA_PAGE_CACHE) ? s_pages[pg] : table[min(key >> page_shift, max_pages - 1)];
             return (int)((((size_t)page_id * K + kh) << page_shift) + (size_t)(key & page_mask));
         };
         auto load_block = [&](int j, int row) {
@@ -419,7 +433,10 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
         const int row_t = threadIdx.x;
         const int qp = q_first + row_t;
         const int lo_t = first_seen(qp, window, chunk);
-        const float sl2 = scale * 1.4426950408889634f;
+        // a score in log2 units is sl2 times the product, or cap_l2 tanh(to_cap times it)
+        const float to_cap = CAP ? scale / softcap : 0.0f;
+        const float sl2 = (CAP ? softcap : scale) * 1.4426950408889634f;
+        const float c2 = to_cap * to_cap, p0 = 0.999999464f * to_cap, p1 = -0.333264679f * to_cap * c2, p2_ = 0.131918818f * to_cap * c2 * c2, p3 = -0.0444444381f * to_cap * c2 * c2 * c2;
         const uint32_t lane_base = tmem_base + ((uint32_t)(warp * 32) << 16);
         // the maximum O and l are currently scaled by (log2 units); a sink is a key without a value whose score is 0 or the
         // head's learned number (not scaled): the maximum starts there and the sum at 1
@@ -438,15 +455,24 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             // two passes over the 64 scores, 32 at a time (tensor memory is cheap to read twice; registers are not):
             // the row maximum first, then the probabilities
-            const bool interior = key0 + TA_BN - 1 <= q_first && key0 >= first_seen(q_last, window, chunk);
+            const bool interior = key0 + TA_BN - 1 <= q_first && (key0 >= first_seen(q_last, window, chunk) || key0 + TA_BN <= keep);
             float mx = -INFINITY;
+            bool small = true;                                 // (CAP) every score of the block is small against the cap
             {
                 float s[64];
                 tmem_ld64(s_col, s);
+                if (CAP) {                                     // (keys that are masked below count too: no harm)
+                    float t4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+                    for (int j = 0; j < 64; j += 4) {
+                        t4[0] = fmaxf(t4[0], fabsf(s[j])); t4[1] = fmaxf(t4[1], fabsf(s[j + 1])); t4[2] = fmaxf(t4[2], fabsf(s[j + 2])); t4[3] = fmaxf(t4[3], fabsf(s[j + 3]));
+                    }
+                    small = __all_sync(0xffffffffu, fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])) * fabsf(to_cap) <= TA_CAP_SMALL);
+                }
                 if (!interior) {
 #pragma unroll
                     for (int j = 0; j < 64; ++j)
-                        if (!(key0 + j <= qp && key0 + j >= lo_t)) s[j] = -INFINITY;
+                        if (!(key0 + j <= qp && (key0 + j >= lo_t || key0 + j < keep))) s[j] = -INFINITY;
                 }
                 float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -454,6 +480,9 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
                     m4[0] = fmaxf(m4[0], s[j]); m4[1] = fmaxf(m4[1], s[j + 1]); m4[2] = fmaxf(m4[2], s[j + 2]); m4[3] = fmaxf(m4[3], s[j + 3]);
                 }
                 mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+                if (CAP) {
+                    if (mx != -INFINITY) mx = tanh_any(mx * to_cap);
+                }
             }
             // raise the scaling maximum only when the true one has moved by more than 8 (or from -inf)
             const float m_true = fmaxf(m_used, mx * sl2);
@@ -484,10 +513,22 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
             {
                 float s[64];
                 tmem_ld64(s_col, s);
+                if (CAP) {                                     // (before the mask: every product is a number)
+                    if (small) {
+#pragma unroll
+                        for (int j = 0; j < 64; ++j) {
+                            const float t = s[j] * s[j];
+                            s[j] *= fmaf(t, fmaf(t, fmaf(t, p3, p2_), p1), p0);
+                        }
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 64; ++j) s[j] = tanh_any(s[j] * to_cap);
+                    }
+                }
                 if (!interior) {
 #pragma unroll
                     for (int j = 0; j < 64; ++j)
-                        if (!(key0 + j <= qp && key0 + j >= lo_t)) s[j] = -INFINITY;
+                        if (!(key0 + j <= qp && (key0 + j >= lo_t || key0 + j < keep))) s[j] = -INFINITY;
                 }
                 float sum2[2] = {0.0f, 0.0f};
 #pragma unroll
@@ -515,8 +556,8 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
         }
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const float inv = 1.0f / l_run;
-            bf16* dst = out + ((size_t)(tok0 + qt * TA_BM + row_t) * H + h) * DV;
+            const float inv = out_scale / l_run;
+            bf16* dst = out + (size_t)(tok0 + qt * TA_BM + row_t) * out_stride + (size_t)h * DV;
             const bf16* grow = (gate != nullptr && row_t < rows) ? gate + (size_t)(tok0 + qt * TA_BM + row_t) * gate_stride + (size_t)h * DV : nullptr;
 #pragma unroll
             for (int c = 0; c < DV / 32; ++c) {
@@ -576,8 +617,9 @@ MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_
                               int max_pages, const int* cu_tokens, const int* seq_lens, int first_req, int requests,
                               int max_query_len, int tokens, int K, int page_size, long long cache_pages, float scale,
                               int window, int* error_flag, int chunk, int sink, const void* gate, int gate_stride, const float* sink_logit,
-                              cudaStream_t s) {
+                              int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
     if (requests <= 0 || max_query_len <= 0) return 0;
+    if (keep < 0 || softcap < 0.0f || out_stride < K * GROUP * DV || out_stride % 8 != 0 || ((uintptr_t)out & 15)) return MB_ERR_BAD_SIZE;
     if (chunk < 0 || (gate != nullptr && (((uintptr_t)gate & 15) || gate_stride % 8 != 0))) return MB_ERR_BAD_SIZE;
     int page_shift = -1;
     for (int b = 4; b < 16; ++b)
@@ -586,7 +628,8 @@ MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_
     if (((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15)) return MB_ERR_BAD_SIZE;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM);
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, TA_SMEM);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -600,6 +643,7 @@ MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_
     rc = TA_V_IN_K ? map_2d(&mv, k_cache, cache_rows, D, box_rows) : map_2d(&mv, v_cache, cache_rows, DV, box_rows);
     if (rc) return rc;
     dim3 grid((max_query_len + TA_BM - 1) / TA_BM, K * GROUP, requests);
-    return launch_kernel(attn_prefill_tc_kernel, grid, 256, TA_SMEM, s, 0, mq, mk, mv, (bf16*)out, block_table, max_pages, cu_tokens,
-                         seq_lens, first_req, K, page_shift, scale, window, error_flag, box_rows, chunk, sink, sink_logit, (const bf16*)gate, gate_stride);
+    return launch_kernel(softcap > 0.0f ? attn_prefill_tc_kernel<true> : attn_prefill_tc_kernel<false>, grid, 256, TA_SMEM, s, 0, mq, mk, mv, (bf16*)out,
+                         block_table, max_pages, cu_tokens, seq_lens, first_req, K, page_shift, scale, window, error_flag, box_rows, chunk, sink, sink_logit,
+                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
 }

@@ -43,6 +43,72 @@ __global__ void delta_conv_kernel(const T* __restrict__ in, int in_stride, const
     out[(size_t)t * channels + c] = from_f32<T>(silu_f(sum));
 }
 
+// The same for bf16 channels in multiples of 8: a thread owns 8 channels of CONV_RUN consecutive tokens, keeps the last TAPS - 1
+// inputs in registers and reads every row once (16-byte loads).  At a request's first token the window is filled from its ring.
+#define CONV_RUN 8
+
+__device__ __forceinline__ void unpack8(const uint4& raw, float* x) {
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h2[i]); x[2 * i] = f.x; x[2 * i + 1] = f.y; }
+}
+
+template <int TAPS>
+__global__ void __launch_bounds__(128) delta_conv_run_kernel(
+    const bf16* __restrict__ in, int in_stride, const float* __restrict__ w, const float* __restrict__ ring, const int* __restrict__ positions,
+    const int* __restrict__ req_index, const int* __restrict__ cu_tokens, const int* __restrict__ slots, bf16* __restrict__ out, int first_token,
+    int tokens, int channels) {
+    PDL_ENTER();
+    in = pdl_fresh(in); ring = pdl_fresh(ring);
+    const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+    if (c0 >= channels) return;
+    const int t0 = first_token + blockIdx.x * CONV_RUN, t1 = min(tokens, t0 + CONV_RUN);
+    float wt[8][TAPS], past[TAPS > 1 ? TAPS - 1 : 1][8];       // past[b]: the input b + 1 tokens back
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c0 + e) * TAPS + j];
+    for (int t = t0; t < t1; ++t) {
+        const int req = req_index[t], first = cu_tokens[req];
+        if (TAPS > 1 && (t == t0 || t == first)) {             // fill the window: from this step's rows, the ring, or nothing
+            const int pos = positions[t];
+            const float* kept = ring + (size_t)slots[req] * TAPS * channels + c0;
+#pragma unroll
+            for (int b = 0; b < TAPS - 1; ++b) {
+                if (t - b - 1 >= first) unpack8(*reinterpret_cast<const uint4*>(in + (size_t)(t - b - 1) * in_stride + c0), past[b]);
+                else {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) past[b][e] = pos - b - 1 >= 0 ? kept[(size_t)((pos - b - 1) % TAPS) * channels + e] : 0.0f;
+                }
+            }
+        }
+        float now[8];
+        unpack8(*reinterpret_cast<const uint4*>(in + (size_t)t * in_stride + c0), now);
+        uint4 packed;
+        __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+        float y[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            float sum = 0.0f;                                  // (the oldest first, as the plain kernel adds)
+#pragma unroll
+            for (int b = TAPS - 2; b >= 0; --b) sum = fmaf(wt[e][TAPS - 2 - b], past[b][e], sum);
+            sum = fmaf(wt[e][TAPS - 1], now[e], sum);
+            y[e] = __fdividef(sum, 1.0f + __expf(-sum));       // (a few float32 ulps, far inside the rounding to bf16)
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) p2[i] = __floats2bfloat162_rn(y[2 * i], y[2 * i + 1]);
+        *reinterpret_cast<uint4*>(out + (size_t)t * channels + c0) = packed;
+#pragma unroll
+        for (int b = TAPS - 2; b > 0; --b)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) past[b][e] = past[b - 1][e];
+        if (TAPS > 1) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) past[0][e] = now[e];
+        }
+    }
+}
+
 // The ring after the step: the inputs of a request's last taps - 1 tokens (or as many as it brought).
 template <typename T>
 __global__ void delta_ring_kernel(const T* __restrict__ in, int in_stride, float* __restrict__ ring, const int* __restrict__ positions,
@@ -65,6 +131,15 @@ MB_API int mb_delta_conv(const void* in, int in_stride, int dtype, const float* 
     if (dtype == MB_F32)
         return launch_kernel(delta_conv_kernel<float>, grid, 128, 0, s, 0, (const float*)in, in_stride, w, ring, positions, req_index, cu_tokens,
                              slots, (float*)out, first_token, channels, taps);
+    if (dtype == MB_BF16 && taps <= 4 && channels % 8 == 0 && in_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+        dim3 runs((tokens - first_token + CONV_RUN - 1) / CONV_RUN, (channels / 8 + 127) / 128);
+#define CONV_CASE(N)                                                                                                                              \
+    if (taps == N)                                                                                                                                \
+        return launch_kernel(delta_conv_run_kernel<N>, runs, 128, 0, s, 0, (const bf16*)in, in_stride, w, ring, positions, req_index, cu_tokens, slots, \
+                             (bf16*)out, first_token, tokens, channels);
+        CONV_CASE(1) CONV_CASE(2) CONV_CASE(3) CONV_CASE(4)
+#undef CONV_CASE
+    }
     if (dtype == MB_BF16)
         return launch_kernel(delta_conv_kernel<bf16>, grid, 128, 0, s, 0, (const bf16*)in, in_stride, w, ring, positions, req_index, cu_tokens,
                              slots, (bf16*)out, first_token, channels, taps);
@@ -221,7 +296,7 @@ MB_API int mb_delta_scan(const void* qkv, int dtype, const void* b_rows, int b_s
 // out = o / rms_head(o) * weight[vdim] * gate(g) * factor; gate 0: sigmoid, 1: silu.  g: [tokens][g_stride].
 template <typename T>
 __global__ void delta_norm_kernel(const float* __restrict__ o, const T* __restrict__ g, int g_stride, int gate, const float* __restrict__ w, float eps,
-                                  float factor, T* __restrict__ out, int out_stride, int first_token, int pairs, int H, int dv) {
+                                  float factor, T* __restrict__ out, int out_stride, int first_token, int pairs, int H, int dv, int vec) {
     PDL_ENTER();
     o = pdl_fresh(o); g = pdl_fresh(g);
     const int p = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -229,10 +304,43 @@ __global__ void delta_norm_kernel(const float* __restrict__ o, const T* __restri
     const int t = first_token + p / H, head = p % H;
     const float* row = o + ((size_t)t * H + head) * dv;
     float ss = 0.0f;
-    for (int i = lane; i < dv; i += 32) { const float v = row[i]; ss = fmaf(v, v, ss); }
-    const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
     const T* gr = g + (size_t)t * g_stride + (size_t)head * dv;
     T* dst = out + (size_t)t * out_stride + (size_t)head * dv;
+    if (sizeof(T) == 2 && vec) {                               // four elements a lane and turn, at most 256 of a head
+        float4 v[2], z[2];
+        const int turns = (dv + 127) / 128;
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int i = u * 128 + lane * 4;
+            v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+            z[u] = v[u];
+            if (u < turns && i < dv) {
+                v[u] = *reinterpret_cast<const float4*>(row + i);
+                const uint2 raw = *reinterpret_cast<const uint2*>(gr + i);
+                const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+                z[u] = make_float4(a.x, a.y, b.x, b.y);
+            }
+            ss += (v[u].x * v[u].x + v[u].y * v[u].y) + (v[u].z * v[u].z + v[u].w * v[u].w);
+        }
+        const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int i = u * 128 + lane * 4;
+            if (u >= turns || i >= dv) continue;
+            const float4 ww = *reinterpret_cast<const float4*>(w + i);
+            float4 s4 = make_float4(__fdividef(1.0f, 1.0f + __expf(-z[u].x)), __fdividef(1.0f, 1.0f + __expf(-z[u].y)), __fdividef(1.0f, 1.0f + __expf(-z[u].z)),
+                                    __fdividef(1.0f, 1.0f + __expf(-z[u].w)));
+            if (gate == 1) { s4.x *= z[u].x; s4.y *= z[u].y; s4.z *= z[u].z; s4.w *= z[u].w; }
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[u].x * f * ww.x * s4.x, v[u].y * f * ww.y * s4.y), hi = __floats2bfloat162_rn(v[u].z * f * ww.z * s4.z, v[u].w * f * ww.w * s4.w);
+            uint2 packed;
+            packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+            packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+            *reinterpret_cast<uint2*>(dst + i) = packed;
+        }
+        return;
+    }
+    for (int i = lane; i < dv; i += 32) { const float v = row[i]; ss = fmaf(v, v, ss); }
+    const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
     for (int i = lane; i < dv; i += 32) {
         const float z = to_f32(gr[i]);
         dst[i] = from_f32<T>(row[i] * f * w[i] * (gate == 0 ? sigmoid_f(z) : silu_f(z)));
@@ -244,12 +352,13 @@ MB_API int mb_delta_norm(const float* o, const void* g, int g_stride, int gate, 
     if (tokens <= first_token) return 0;
     if (H <= 0 || dv <= 0 || gate < 0 || gate > 1 || first_token < 0 || out_stride < H * dv) return MB_ERR_BAD_SIZE;
     const int pairs = (tokens - first_token) * H, blocks = (pairs + 7) / 8;
+    const int vec = dv % 4 == 0 && dv <= 256 && g_stride % 4 == 0 && out_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)w) & 15) == 0 && (((uintptr_t)g | (uintptr_t)out) & 7) == 0;
     if (dtype == MB_F32)
         return launch_kernel(delta_norm_kernel<float>, blocks, 256, 0, s, 0, o, (const float*)g, g_stride, gate, w, eps, factor, (float*)out, out_stride,
-                             first_token, pairs, H, dv);
+                             first_token, pairs, H, dv, vec);
     if (dtype == MB_BF16)
         return launch_kernel(delta_norm_kernel<bf16>, blocks, 256, 0, s, 0, o, (const bf16*)g, g_stride, gate, w, eps, factor, (bf16*)out, out_stride,
-                             first_token, pairs, H, dv);
+                             first_token, pairs, H, dv, vec);
     return MB_ERR_BAD_DTYPE;
 }
 
@@ -274,7 +383,7 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
     float* gs = ks + d4;                       // [d]
     float* vs = gs + d4;                       // [dv]
     float* sums = vs + dv;                     // [PARTS][dv]
-    __shared__ float scratch[32];
+    __shared__ float scratch[32], scratch2[32];
     const int head = blockIdx.x, r = blockIdx.y;
     if (seq_lens[r] <= 0) return;              // a row that pads a captured batch
     const int groups = dv >> 2, threads = blockDim.x;
@@ -288,31 +397,72 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
         const int n = part + PARTS * j;
         s[j] = (owner && n < d) ? S[(size_t)n * groups] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    const float rate_raw = rate_log[head], beta_raw = to_f32(b_rows[(size_t)r * b_stride + head]);
+    float decay_raw = 0.0f, decay_bias = 0.0f, gate_raw = 0.0f, norm_raw = 0.0f;         // asked for early, used late
+    if (threadIdx.x < d) {
+        const int at = per_channel ? head * d + threadIdx.x : head;
+        decay_raw = to_f32(a_rows[(size_t)r * a_stride + at]);
+        decay_bias = dt_bias[at];
+    }
+    if (threadIdx.x < dv) {
+        gate_raw = to_f32(g[(size_t)r * g_stride + (size_t)head * dv + threadIdx.x]);
+        norm_raw = norm_w[threadIdx.x];
+    }
     // the convolution of this head's q, k and v channels
     const int share = H / G, kh = head / share, channels = 2 * G * d + H * dv;
     float* kept = ring + (size_t)slot * taps * channels;
     const T* row = in + (size_t)r * in_stride;
+    const int pos_row = pos % taps;
     float qq = 0.0f, kk = 0.0f;
     for (int i = threadIdx.x; i < 2 * d + dv; i += threads) {
         const int c = i < d ? kh * d + i : i < 2 * d ? G * d + kh * d + (i - d) : 2 * G * d + head * dv + (i - 2 * d);
         const float now = to_f32(row[c]);
         float sum = 0.0f;
-        for (int back = min(taps - 1, pos); back > 0; --back)
-            sum = fmaf(conv_w[(size_t)c * taps + taps - 1 - back], kept[(size_t)((pos - back) % taps) * channels + c], sum);
+        const int most = min(taps - 1, pos);
+        if (taps <= 4) {                       // all loads in flight at once
+            float x[3], y[3];
+#pragma unroll
+            for (int back = 3; back > 0; --back) {
+                x[back - 1] = y[back - 1] = 0.0f;
+                if (back <= most) {
+                    int at = pos_row - back;
+                    at = at < 0 ? at + taps : at;
+                    x[back - 1] = kept[(size_t)at * channels + c];
+                    y[back - 1] = conv_w[(size_t)c * taps + taps - 1 - back];
+                }
+            }
+#pragma unroll
+            for (int back = 3; back > 0; --back) sum = fmaf(y[back - 1], x[back - 1], sum);
+        } else {
+            for (int back = most; back > 0; --back)
+                sum = fmaf(conv_w[(size_t)c * taps + taps - 1 - back], kept[(size_t)((pos - back) % taps) * channels + c], sum);
+        }
         sum = silu_f(fmaf(conv_w[(size_t)c * taps + taps - 1], now, sum));
-        if (taps > 1 && (i >= 2 * d || head == kh * share)) kept[(size_t)(pos % taps) * channels + c] = now;
+        if (taps > 1 && (i >= 2 * d || head == kh * share)) kept[(size_t)pos_row * channels + c] = now;
         sum = to_f32(from_f32<T>(sum));        // as the convolution of many tokens leaves it
         if (i < d) { qs[i] = sum; qq = fmaf(sum, sum, qq); }
         else if (i < 2 * d) { ks[i - d] = sum; kk = fmaf(sum, sum, kk); }
         else vs[i - 2 * d] = sum;
     }
-    const float rate = expf(rate_log[head]);
-    for (int i = threadIdx.x; i < d; i += threads)
-        gs[i] = per_channel ? expf(-rate * softplus_f(to_f32(a_rows[(size_t)r * a_stride + (size_t)head * d + i]) + dt_bias[head * d + i]))
-                            : expf(-rate * softplus_f(to_f32(a_rows[(size_t)r * a_stride + head]) + dt_bias[head]));
-    const float beta = sigmoid_f(to_f32(b_rows[(size_t)r * b_stride + head]));
-    qq = block_sum(qq, scratch);
-    kk = block_sum(kk, scratch);               // (their barriers publish qs, ks, gs and vs)
+    const float rate = expf(rate_raw);
+    for (int i = threadIdx.x; i < d; i += threads) {
+        if (i >= threads) {
+            const int at = per_channel ? head * d + i : head;
+            decay_raw = to_f32(a_rows[(size_t)r * a_stride + at]);
+            decay_bias = dt_bias[at];
+        }
+        gs[i] = expf(-rate * softplus_f(decay_raw + decay_bias));
+    }
+    const float beta = sigmoid_f(beta_raw);
+    qq = warp_sum(qq);
+    kk = warp_sum(kk);
+    if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = qq; scratch2[threadIdx.x >> 5] = kk; }
+    __syncthreads();                           // (publishes qs, ks, gs and vs too)
+    {
+        const int lane = threadIdx.x & 31, warps = (threads + 31) >> 5;
+        qq = warp_sum(lane < warps ? scratch[lane] : 0.0f);
+        kk = warp_sum(lane < warps ? scratch2[lane] : 0.0f);
+    }
     const float fq = 1.0f / (sqrtf((float)d) * sqrtf(qq + UNIT_EPS)), fk = 1.0f / sqrtf(kk + UNIT_EPS);
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
@@ -362,8 +512,9 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
     ss = block_sum(ss, scratch);
     const float f = factor / sqrtf(ss / (float)dv + eps);
     for (int i = threadIdx.x; i < dv; i += threads) {
-        const float z = to_f32(g[(size_t)r * g_stride + (size_t)head * dv + i]);
-        out[(size_t)r * out_stride + (size_t)head * dv + i] = from_f32<T>(vs[i] * f * norm_w[i] * (gate == 0 ? sigmoid_f(z) : silu_f(z)));
+        const float z = i < threads ? gate_raw : to_f32(g[(size_t)r * g_stride + (size_t)head * dv + i]);
+        const float wn = i < threads ? norm_raw : norm_w[i];
+        out[(size_t)r * out_stride + (size_t)head * dv + i] = from_f32<T>(vs[i] * f * wn * (gate == 0 ? sigmoid_f(z) : silu_f(z)));
     }
 }
 

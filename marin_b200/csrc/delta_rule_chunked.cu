@@ -12,8 +12,8 @@
 // and slice of value channels) then walks the chunks in order: U = U0 - W S0, O, S.
 //
 // Exactness.  Every exponent that is taken is of a non-positive number: with one decay per channel a block of 16 rows is worked out
-// against a reference between it and the earlier rows (exp(G_i - R) exp(R - G_j), both at most 1), and the 16 x 16 blocks on the diagonal
-// pair by pair.  Decays, sums, unit vectors, A, the substitution and the state are float32; where a float32 number has to be an
+// against a reference between it and the earlier rows (exp(G_i - R) exp(R - G_j), both at most 1), the lower half of a block's diagonal
+// square against one in its middle, and the 8 x 8 squares left on the diagonal pair by pair.  Decays, sums, unit vectors, A, the substitution and the state are float32; where a float32 number has to be an
 // operand of a product it is split into two bf16 numbers (value = hi + lo) and the three larger products are taken, so that about 16
 // bits of it enter.
 #define MB_LIB "delta_rule_chunked"
@@ -70,11 +70,11 @@ __device__ __forceinline__ int first_chunk(const int* cu_tokens, int first_req, 
 #define LDR (DQ + 2)                  // raw q and k rows in shared memory (bf16): rows fall into different banks
 #define LDG (DQ + 1)
 #define LDL (CH + 4)
-#define PREP_SMEM(CHANNEL) (2 * CH * LDR * 2 + ((CHANNEL) ? CH * LDG : CH) * 4 + 2 * CH * LDL * 4 + 3 * CH * 4 + 16)
-#define PREP_THREADS 128
+#define PREP_SMEM(CHANNEL) (2 * CH * LDR * 2 + ((CHANNEL) ? CH * LDG : CH) * 4 + CH * LDL * 4 + 4 * CH * 4 + 16)
+#define PREP_THREADS 256
 
 template <bool CHANNEL>
-__global__ void __launch_bounds__(PREP_THREADS) prepare_kernel(
+__global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
     const bf16* __restrict__ qkv, const bf16* __restrict__ b_rows, int b_stride, const bf16* __restrict__ a_rows, int a_stride,
     const float* __restrict__ rate_log, const float* __restrict__ dt_bias, const int* __restrict__ cu_tokens, int first_req,
     bf16* __restrict__ planes, float* __restrict__ floats, int H, int G, int dv) {
@@ -84,11 +84,11 @@ __global__ void __launch_bounds__(PREP_THREADS) prepare_kernel(
     bf16* sq = reinterpret_cast<bf16*>(smem_raw);              // [CH][LDR]
     bf16* sk = sq + CH * LDR;
     float* sL = reinterpret_cast<float*>(sk + CH * LDR);       // [CH][LDL] beta_i A_ij
-    float* sP = sL + CH * LDL;                                 // [CH][LDL]
-    float* sG = sP + CH * LDL;                                 // [CH][LDG], or [CH] with one decay per head (log2 units)
+    float* sG = sL + CH * LDL;                                 // [CH][LDG], or [CH] with one decay per head (log2 units)
     float* s_beta = sG + (CHANNEL ? CH * LDG : CH);
     float* s_fq = s_beta + CH;
     float* s_fk = s_fq + CH;
+    float* s_qk = s_fk + CH;                                   // q_i . k_i as they are
     const int req = first_req + blockIdx.z, head = blockIdx.y;
     const int tok0 = cu_tokens[req] + blockIdx.x * CH;
     const int rows = min(CH, cu_tokens[req + 1] - tok0);
@@ -131,130 +131,162 @@ __global__ void __launch_bounds__(PREP_THREADS) prepare_kernel(
         for (int i = 0; i < CH; ++i) { run += sG[i]; sG[i] = run; }
     }
     for (int row = warp; row < CH; row += PREP_THREADS / 32) {
-        float qq = 0.0f, kk = 0.0f;
+        float qq = 0.0f, kk = 0.0f, qk = 0.0f;
         for (int c = lane; c < DQ; c += 32) {
             const float x = __bfloat162float(sq[row * LDR + c]), y = __bfloat162float(sk[row * LDR + c]);
             qq = fmaf(x, x, qq);
             kk = fmaf(y, y, kk);
+            qk = fmaf(x, y, qk);
         }
         qq = warp_sum(qq);
         kk = warp_sum(kk);
+        qk = warp_sum(qk);
         if (lane == 0) {
             s_fq[row] = 1.0f / (sqrtf((float)DQ) * sqrtf(qq + UNIT_EPS));
             s_fk[row] = 1.0f / sqrtf(kk + UNIT_EPS);
+            s_qk[row] = qk;
         }
     }
-    // (the weighted products' upper triangle stays zero)
-    for (int idx = tid; idx < CH * LDL; idx += PREP_THREADS) { sL[idx] = 0.0f; sP[idx] = 0.0f; }
+    // (the upper triangles stay zero; of P's only what lies in a diagonal block is ever read)
+    for (int idx = tid; idx < CH * LDL; idx += PREP_THREADS) sL[idx] = 0.0f;
+    bf16* ph = out + 6 * PLANE;
+    for (int idx = tid; idx < 4 * 16 * 8; idx += PREP_THREADS) {
+        const int row = (idx >> 3), at = row * CH + (row & ~15) + (idx & 7) * 2;
+        *reinterpret_cast<uint32_t*>(ph + at) = 0u;
+        *reinterpret_cast<uint32_t*>(ph + PPLANE + at) = 0u;
+    }
     __syncthreads();
-    // ---- A and P: warp w makes the rows 16 w .. 16 w + 15
+    // ---- A and P: two warps make the rows 16 I .. 16 I + 15, each eight columns of every block of sixteen
     {
-        const int i0 = warp * 16 + g, i1 = i0 + 8;
-        float accA[4][2][4], accP[4][2][4];
+        const int I = warp >> 1, half = warp & 1;
+        const int i0 = I * 16 + g, i1 = i0 + 8;
+        float accA[4][4], accP[4][4];                          // [block of columns]; the fourth: this block's own
 #pragma unroll
         for (int J = 0; J < 4; ++J)
 #pragma unroll
-            for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) { accA[J][nt][e] = 0.0f; accP[J][nt][e] = 0.0f; }
+            for (int e = 0; e < 4; ++e) { accA[J][e] = 0.0f; accP[J][e] = 0.0f; }
+        // a reference for the rows of this block against earlier ones: the sum at the last row before it; for its rows 8 .. 15 against
+        // its rows 0 .. 7 (worked out by the first of the two warps): the sum at its row 7
+        const float* ref = sG + (I > 0 ? I * 16 - 1 : 0) * LDG;
+        const float* mid = sG + (I * 16 + 7) * LDG;
 #pragma unroll 1
         for (int kk = 0; kk < DQ / 16; ++kk) {
             uint32_t rk[4], rq[4];                             // raw bf16 pairs: rows i0, i1 at channels c, c + 8
+            const int c = kk * 16 + t2;
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const int row = (u & 1) ? i1 : i0, c = kk * 16 + t2 + (u >> 1) * 8;
-                rk[u] = *reinterpret_cast<const uint32_t*>(sk + row * LDR + c);
-                rq[u] = *reinterpret_cast<const uint32_t*>(sq + row * LDR + c);
+                const int row = (u & 1) ? i1 : i0;
+                rk[u] = *reinterpret_cast<const uint32_t*>(sk + row * LDR + c + (u >> 1) * 8);
+                rq[u] = *reinterpret_cast<const uint32_t*>(sq + row * LDR + c + (u >> 1) * 8);
             }
             if (!CHANNEL) {
 #pragma unroll
                 for (int J = 0; J < 4; ++J) {
-                    if (J > warp) continue;
-#pragma unroll
-                    for (int nt = 0; nt < 2; ++nt) {
-                        const bf16* row = sk + (J * 16 + nt * 8 + g) * LDR + kk * 16 + t2;
-                        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(row), b1 = *reinterpret_cast<const uint32_t*>(row + 8);
-                        mma_bf16_16816(accA[J][nt], rk, b0, b1);
-                        mma_bf16_16816(accP[J][nt], rq, b0, b1);
-                    }
+                    const int jb = J < 3 ? J : I;
+                    if (J < 3 && J >= I) continue;
+                    const bf16* row = sk + (jb * 16 + half * 8 + g) * LDR + c;
+                    const uint32_t b0 = *reinterpret_cast<const uint32_t*>(row), b1 = *reinterpret_cast<const uint32_t*>(row + 8);
+                    mma_bf16_16816(accA[J], rk, b0, b1);
+                    mma_bf16_16816(accP[J], rq, b0, b1);
                 }
-            } else if (warp > 0) {
-                // the reference: the sum at the last row before this warp's block
-                const float* ref = sG + (warp * 16 - 1) * LDG;
+            } else {
                 uint32_t kh_[4], kl_[4], qh_[4], ql_[4];
-                float r[4];
+                if (I > 0) {
+                    const float r[4] = {ref[c], ref[c + 1], ref[c + 8], ref[c + 9]};
 #pragma unroll
-                for (int u = 0; u < 4; ++u) r[u] = ref[kk * 16 + t2 + (u >> 1) * 8 + (u & 1)];
+                    for (int u = 0; u < 4; ++u) {
+                        const float* gi = sG + ((u & 1) ? i1 : i0) * LDG + c + (u >> 1) * 8;
+                        const float e0 = ex2_approx(gi[0] - r[(u >> 1) * 2]), e1 = ex2_approx(gi[1] - r[(u >> 1) * 2 + 1]);
+                        const float2 k2 = bf2(rk[u]), q2 = bf2(rq[u]);
+                        split_bf16(k2.x * e0, k2.y * e1, kh_[u], kl_[u]);
+                        split_bf16(q2.x * e0, q2.y * e1, qh_[u], ql_[u]);
+                    }
 #pragma unroll
-                for (int u = 0; u < 4; ++u) {
-                    const int row = (u & 1) ? i1 : i0, c = kk * 16 + t2 + (u >> 1) * 8;
-                    const float e0 = ex2_approx(sG[row * LDG + c] - r[(u >> 1) * 2]), e1 = ex2_approx(sG[row * LDG + c + 1] - r[(u >> 1) * 2 + 1]);
-                    const float2 k2 = bf2(rk[u]), q2 = bf2(rq[u]);
-                    split_bf16(k2.x * e0, k2.y * e1, kh_[u], kl_[u]);
-                    split_bf16(q2.x * e0, q2.y * e1, qh_[u], ql_[u]);
-                }
-#pragma unroll
-                for (int J = 0; J < 3; ++J) {
-                    if (J >= warp) continue;
-#pragma unroll
-                    for (int nt = 0; nt < 2; ++nt) {
-                        const int j = J * 16 + nt * 8 + g, c = kk * 16 + t2;
+                    for (int J = 0; J < 3; ++J) {
+                        if (J >= I) continue;
+                        const int j = J * 16 + half * 8 + g;
                         const float* gj = sG + j * LDG + c;
                         const float2 x = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c)), y = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c + 8));
                         uint32_t bh0, bl0, bh1, bl1;
                         split_bf16(x.x * ex2_approx(r[0] - gj[0]), x.y * ex2_approx(r[1] - gj[1]), bh0, bl0);
                         split_bf16(y.x * ex2_approx(r[2] - gj[8]), y.y * ex2_approx(r[3] - gj[9]), bh1, bl1);
-                        mma3(accA[J][nt], kh_, kl_, bh0, bh1, bl0, bl1);
-                        mma3(accP[J][nt], qh_, ql_, bh0, bh1, bl0, bl1);
+                        mma3(accA[J], kh_, kl_, bh0, bh1, bl0, bl1);
+                        mma3(accP[J], qh_, ql_, bh0, bh1, bl0, bl1);
                     }
+                }
+                if (half == 0) {                               // rows 8 .. 15 of the block (the operands of rows 0 .. 7 are zero)
+                    const float r[4] = {mid[c], mid[c + 1], mid[c + 8], mid[c + 9]};
+                    kh_[0] = kh_[2] = kl_[0] = kl_[2] = qh_[0] = qh_[2] = ql_[0] = ql_[2] = 0u;
+#pragma unroll
+                    for (int u = 1; u < 4; u += 2) {
+                        const float* gi = sG + i1 * LDG + c + (u >> 1) * 8;
+                        const float e0 = ex2_approx(gi[0] - r[(u >> 1) * 2]), e1 = ex2_approx(gi[1] - r[(u >> 1) * 2 + 1]);
+                        const float2 k2 = bf2(rk[u]), q2 = bf2(rq[u]);
+                        split_bf16(k2.x * e0, k2.y * e1, kh_[u], kl_[u]);
+                        split_bf16(q2.x * e0, q2.y * e1, qh_[u], ql_[u]);
+                    }
+                    const float* gj = sG + i0 * LDG + c;      // token g of the block: the same index as row i0
+                    const float2 x = bf2(rk[0]), y = bf2(rk[2]);
+                    uint32_t bh0, bl0, bh1, bl1;
+                    split_bf16(x.x * ex2_approx(r[0] - gj[0]), x.y * ex2_approx(r[1] - gj[1]), bh0, bl0);
+                    split_bf16(y.x * ex2_approx(r[2] - gj[8]), y.y * ex2_approx(r[3] - gj[9]), bh1, bl1);
+                    mma3(accA[3], kh_, kl_, bh0, bh1, bl0, bl1);
+                    mma3(accP[3], qh_, ql_, bh0, bh1, bl0, bl1);
                 }
             }
         }
 #pragma unroll
         for (int J = 0; J < 4; ++J) {
-            if (J > warp || (CHANNEL && J == warp)) continue;
+            const int jb = J < 3 ? J : I;
+            if ((J < 3 && J >= I) || (CHANNEL && J == 3 && half == 1)) continue;
+            const int j = jb * 16 + half * 8 + t2;
 #pragma unroll
-            for (int nt = 0; nt < 2; ++nt)
+            for (int rr = 0; rr < 2; ++rr) {
+                if (CHANNEL && J == 3 && rr == 0) continue;    // rows 0 .. 7 of the block's own square: pair by pair below
+                const int i = rr ? i1 : i0;
+                float a[2], b[2];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int i = (e >> 1) ? i1 : i0, j = J * 16 + nt * 8 + t2 + (e & 1);
-                    if (j > i) continue;
-                    const float w = CHANNEL ? 1.0f : ex2_approx(sG[i] - sG[j]);
-                    if (j < i) sL[i * LDL + j] = s_beta[i] * s_fk[i] * s_fk[j] * accA[J][nt][e] * w;
-                    sP[i * LDL + j] = s_fq[i] * s_fk[j] * accP[J][nt][e] * w;
+                for (int e = 0; e < 2; ++e) {
+                    const float w = CHANNEL ? 1.0f : j + e <= i ? ex2_approx(sG[i] - sG[j + e]) : 0.0f;
+                    a[e] = s_beta[i] * s_fk[i] * s_fk[j + e] * accA[J][rr * 2 + e] * w;
+                    b[e] = s_fq[i] * s_fk[j + e] * accP[J][rr * 2 + e] * w;
+                    if (j + e < i) sL[i * LDL + j + e] = a[e];
                 }
-        }
-        if (CHANNEL) {                                         // the block on the diagonal, a pair of rows per lane
-            for (int p = lane; p < 136; p += 32) {
-                int ii = (int)((sqrtf(8.0f * (float)p + 1.0f) - 1.0f) * 0.5f);
-                if ((ii + 1) * (ii + 2) / 2 <= p) ++ii;
-                if (ii * (ii + 1) / 2 > p) --ii;
-                const int i = warp * 16 + ii, j = warp * 16 + p - ii * (ii + 1) / 2;
-                float a = 0.0f, b = 0.0f;
-#pragma unroll 4
-                for (int c = 0; c < DQ; c += 2) {
-                    const float2 ki = bf2(*reinterpret_cast<const uint32_t*>(sk + i * LDR + c)), kj = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c));
-                    const float2 qi = bf2(*reinterpret_cast<const uint32_t*>(sq + i * LDR + c));
-                    const float x = kj.x * ex2_approx(sG[i * LDG + c] - sG[j * LDG + c]), y = kj.y * ex2_approx(sG[i * LDG + c + 1] - sG[j * LDG + c + 1]);
-                    a = fmaf(ki.x, x, a); a = fmaf(ki.y, y, a);
-                    b = fmaf(qi.x, x, b); b = fmaf(qi.y, y, b);
-                }
-                if (j < i) sL[i * LDL + j] = s_beta[i] * s_fk[i] * s_fk[j] * a;
-                sP[i * LDL + j] = s_fq[i] * s_fk[j] * b;
+                uint32_t hi, lo;                               // (a weight of zero where j > i)
+                split_bf16(b[0], b[1], hi, lo);
+                *reinterpret_cast<uint32_t*>(ph + i * CH + j) = hi;
+                *reinterpret_cast<uint32_t*>(ph + PPLANE + i * CH + j) = lo;
             }
+        }
+        if (CHANNEL && lane < 28) {                            // the 8 x 8 square on the diagonal that is this warp's, a pair of rows per lane
+            int ii = 1;
+            while ((ii + 1) * ii / 2 <= lane) ++ii;
+            const int i = warp * 8 + ii, j = warp * 8 + lane - ii * (ii - 1) / 2;
+            float a = 0.0f, b = 0.0f;
+#pragma unroll 4
+            for (int c = 0; c < DQ; c += 2) {
+                const float2 ki = bf2(*reinterpret_cast<const uint32_t*>(sk + i * LDR + c)), kj = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c));
+                const float2 qi = bf2(*reinterpret_cast<const uint32_t*>(sq + i * LDR + c));
+                const float x = kj.x * ex2_approx(sG[i * LDG + c] - sG[j * LDG + c]), y = kj.y * ex2_approx(sG[i * LDG + c + 1] - sG[j * LDG + c + 1]);
+                a = fmaf(ki.x, x, a); a = fmaf(ki.y, y, a);
+                b = fmaf(qi.x, x, b); b = fmaf(qi.y, y, b);
+            }
+            sL[i * LDL + j] = s_beta[i] * s_fk[i] * s_fk[j] * a;
+            b *= s_fq[i] * s_fk[j];
+            const bf16 hi = __float2bfloat16_rn(b);
+            ph[i * CH + j] = hi;
+            ph[PPLANE + i * CH + j] = __float2bfloat16_rn(b - __bfloat162float(hi));
+        }
+        if (CHANNEL && tid < CH) {                             // P_ii = q_i . k_i
+            const float b = s_qk[tid] * s_fq[tid] * s_fk[tid];
+            const bf16 hi = __float2bfloat16_rn(b);
+            ph[tid * CH + tid] = hi;
+            ph[PPLANE + tid * CH + tid] = __float2bfloat16_rn(b - __bfloat162float(hi));
         }
     }
     __syncthreads();
-    // ---- P, Q+, K exp(G_63 - G), exp(G_63)
+    // ---- Q+, K exp(G_63 - G), exp(G_63)
     {
-        bf16* ph = out + 6 * PLANE;
-        for (int idx = tid; idx < CH * CH / 2; idx += PREP_THREADS) {
-            const int i = idx / (CH / 2), j = (idx % (CH / 2)) * 2;
-            uint32_t hi, lo;
-            split_bf16(sP[i * LDL + j], sP[i * LDL + j + 1], hi, lo);
-            *reinterpret_cast<uint32_t*>(ph + i * CH + j) = hi;
-            *reinterpret_cast<uint32_t*>(ph + PPLANE + i * CH + j) = lo;
-        }
         for (int idx = tid; idx < CH * DQ / 2; idx += PREP_THREADS) {
             const int i = idx / (DQ / 2), c = (idx % (DQ / 2)) * 2;
             const float g0 = CHANNEL ? sG[i * LDG + c] : sG[i], g1 = CHANNEL ? sG[i * LDG + c + 1] : g0;

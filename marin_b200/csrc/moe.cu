@@ -338,6 +338,9 @@ MB_API int mb_moe_experts_plain(const void* h_rows, int dtype, const void* w_gat
 #define G_STAGES_OF(MODE) ((MODE) == 0 ? 4 : 6)
 #define G_NB_OF(MODE) ((MODE) == 0 ? 2 : 1)
 
+// A row per blockIdx.x; with few rows their columns are spread over blockIdx.y too, so that every load of a row is in flight at once.
+static inline dim3 spread(int rows, int h, int threads) { return dim3(rows, rows >= 512 ? 1 : (h + threads - 1) / threads); }
+
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ h_rows, const int* __restrict__ order, const float* __restrict__ weight_of,
                                   T* __restrict__ xs, int* __restrict__ token_sorted, float* __restrict__ weight_sorted,
@@ -348,9 +351,10 @@ __global__ void moe_gather_kernel(const T* __restrict__ h_rows, const int* __res
     const int p = order[i];
     const int token = p / top;
     const float w = weight_of[p];
-    if (threadIdx.x == 0) { token_sorted[i] = token; weight_sorted[i] = w; inv[p] = i; }
+    if (threadIdx.x == 0 && blockIdx.y == 0) { token_sorted[i] = token; weight_sorted[i] = w; inv[p] = i; }
     const float f = weight_on_input ? w : 1.0f;
-    for (int c = threadIdx.x; c < h; c += blockDim.x) xs[(size_t)i * h + c] = from_f32<T>(to_f32(h_rows[(size_t)token * h + c]) * f);
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < h; c += gridDim.y * blockDim.x)
+        xs[(size_t)i * h + c] = from_f32<T>(to_f32(h_rows[(size_t)token * h + c]) * f);
 }
 
 // MODE 0: W [E][2 N][K] (gate rows, then up rows), result silu(gate) * up as bf16 [rows][N].
@@ -507,7 +511,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, const int* __
     rows = pdl_fresh(rows); inv = pdl_fresh(inv); y = pdl_fresh(y); weight_of = pdl_fresh(weight_of);
     expert_of = pdl_fresh(expert_of); h_rows = pdl_fresh(h_rows); identity_weight = pdl_fresh(identity_weight);
     const int t = blockIdx.x;
-    for (int c = threadIdx.x; c < h; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < h; c += gridDim.y * blockDim.x) {
         float a = y[(size_t)t * h + c];
         for (int k = 0; k < top; ++k) {
             if (h_rows != nullptr && expert_of[t * top + k] >= E) {
@@ -555,7 +559,7 @@ static int grouped_by_rows(const bf16* A, const bf16* W, const int* offsets, int
 MB_API int mb_moe_gather(const void* h_rows, const int* order, const float* weight_of, void* xs, int* token_sorted, float* weight_sorted,
                          int* inv, int pairs, int h, int top, int weight_on_input, cudaStream_t s) {
     if (pairs <= 0) return 0;
-    return launch_kernel(moe_gather_kernel<bf16>, pairs, 128, 0, s, 0, (const bf16*)h_rows, order, weight_of, (bf16*)xs, token_sorted,
+    return launch_kernel(moe_gather_kernel<bf16>, spread(pairs, h, 128), 128, 0, s, 0, (const bf16*)h_rows, order, weight_of, (bf16*)xs, token_sorted,
                          weight_sorted, inv, h, top, weight_on_input);
 }
 
@@ -583,5 +587,5 @@ MB_API int mb_moe_grouped_down(const void* act, const void* w_down, const int* o
 MB_API int mb_moe_combine(const float* rows, const int* inv, const float* weight_of, float* y, int tokens, int h, int top, const int* expert_of,
                           const void* h_rows, const float* identity_weight, int E, cudaStream_t s) {
     if (tokens <= 0) return 0;
-    return launch_kernel(moe_combine_kernel, tokens, 256, 0, s, 0, rows, inv, weight_of, y, h, top, expert_of, (const bf16*)h_rows, identity_weight, E);
+    return launch_kernel(moe_combine_kernel, spread(tokens, h, 256), 256, 0, s, 0, rows, inv, weight_of, y, h, top, expert_of, (const bf16*)h_rows, identity_weight, E);
 }

@@ -720,7 +720,8 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
                                          _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
                                          _c_int(ctx.max_query_len), _c_int(T), _c_int(K), _c_int(page_size),
                                          ctypes.c_longlong(k_cache.shape[0]), _c_float(scale), _c_int(window),
-                                         _ptr(_scratch_for(q.device).error), _c_int(0), _c_int(0), _ptr(None), _c_int(0), _ptr(None), _stream()),
+                                         _ptr(_scratch_for(q.device).error), _c_int(0), _c_int(0), _ptr(None), _c_int(0), _ptr(None),
+                                         _c_int(0), _c_float(0.0), _c_float(1.0), _c_int(H * d), _stream()),
                    "attention (prefill, tensor cores)")
         elif ctx.num_requests > nd:
             _attention_cost(q, T - nd, H, K, d, "prefill")
@@ -1270,7 +1271,6 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     _need_cuda(q, k_cache, v_cache, block_table, sink_logits)
     assert out.is_cuda and out.stride(1) == 1
     more = (_c_int(keep_first), _c_float(softcap), _c_float(out_scale), _c_int(out.stride(0)))
-    variant = keep_first > 0 or softcap > 0.0 or out_scale != 1.0 or out.stride(0) != H * dv        # (not in the tcgen05 kernel)
     T = q.shape[0]
     page_size = k_cache.shape[2]
     values_in_keys = v_cache.data_ptr() == k_cache.data_ptr()
@@ -1316,10 +1316,10 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
         if ctx.num_requests > nd and launch_log is not None:
             _cost((T - nd) * per_row, 0.0, key_bytes, 2.0 * H * (d + dv))
             _pending_cost["rows"], _pending_cost["window"] = "prefill", window
-        if (ctx.num_requests > nd and not variant and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
-                and (gate is None or (gate.data_ptr() % 16 == 0 and gate_stride % 8 == 0))):
+        if (ctx.num_requests > nd and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
+                and (gate is None or (gate.data_ptr() % 16 == 0 and gate_stride % 8 == 0)) and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0):
             # heads of 64 or 128 with values as wide: the tcgen05 kernel that plain causal attention uses takes the chunked
-            # mask, the sink and the gate as parameters; over a shared latent one CTA per query head reads the one kv head's rows
+            # mask, the kept positions, the cap, the sink and the gate as parameters; over a shared latent one CTA per query head reads the one kv head's rows
             g = H // kv_heads
             tc = build.load(build.attention_tc_name(d, g, dv, values_in_keys), *build.attention_tc_job(d, g, dv, values_in_keys))
             _check(tc.mb_attn_prefill_tc(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
@@ -1327,7 +1327,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
                                          _c_int(ctx.max_query_len), _c_int(T), _c_int(kv_heads), _c_int(page_size),
                                          ctypes.c_longlong(k_cache.shape[0]), _c_float(scale), _c_int(window),
                                          _ptr(_scratch_for(q.device).error), _c_int(chunk), _c_int(int(sink)), _ptr(gate),
-                                         _c_int(gate_stride), _ptr(sink_logits), _stream()), "attention (sink, prefill, tensor cores)")
+                                         _c_int(gate_stride), _ptr(sink_logits), *more, _stream()), "attention (sink, prefill, tensor cores)")
         elif ctx.num_requests > nd:
             _check(lib.mb_attn_sink_prefill(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
                                             _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
