@@ -38,7 +38,7 @@ __global__ void delta_conv_kernel(const T* __restrict__ in, int in_stride, const
     float sum = 0.0f;
     for (int back = min(taps - 1, pos); back >= 0; --back) {
         const float v = t - back >= first ? to_f32(in[(size_t)(t - back) * in_stride + c]) : kept[(size_t)((pos - back) % taps) * channels + c];
-        sum = fmaf(w[(size_t)c * taps + taps - 1 - back], v, sum);
+        sum = fmaf(w[(size_t)(taps - 1 - back) * channels + c], v, sum);
     }
     out[(size_t)t * channels + c] = from_f32<T>(silu_f(sum));
 }
@@ -65,12 +65,21 @@ __global__ void __launch_bounds__(128) delta_conv_run_kernel(
     const int t0 = first_token + blockIdx.x * CONV_RUN, t1 = min(tokens, t0 + CONV_RUN);
     float wt[8][TAPS], past[TAPS > 1 ? TAPS - 1 : 1][8];       // past[b]: the input b + 1 tokens back
 #pragma unroll
-    for (int e = 0; e < 8; ++e)
+    for (int j = 0; j < TAPS; ++j) {
+        const float4 a = *reinterpret_cast<const float4*>(w + (size_t)j * channels + c0), b = *reinterpret_cast<const float4*>(w + (size_t)j * channels + c0 + 4);
+        wt[0][j] = a.x; wt[1][j] = a.y; wt[2][j] = a.z; wt[3][j] = a.w; wt[4][j] = b.x; wt[5][j] = b.y; wt[6][j] = b.z; wt[7][j] = b.w;
+    }
+    uint4 raw[CONV_RUN];                                       // every row of the run in flight at once
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c0 + e) * TAPS + j];
-    for (int t = t0; t < t1; ++t) {
-        const int req = req_index[t], first = cu_tokens[req];
-        if (TAPS > 1 && (t == t0 || t == first)) {             // fill the window: from this step's rows, the ring, or nothing
+    for (int u = 0; u < CONV_RUN; ++u)
+        if (t0 + u < t1) raw[u] = *reinterpret_cast<const uint4*>(in + (size_t)(t0 + u) * in_stride + c0);
+    int req = req_index[t0], first = cu_tokens[req], end = cu_tokens[req + 1];
+#pragma unroll
+    for (int u = 0; u < CONV_RUN; ++u) {
+        const int t = t0 + u;
+        if (t >= t1) break;
+        if (t == end) { req = req_index[t]; first = t; end = cu_tokens[req + 1]; }
+        if (TAPS > 1 && (u == 0 || t == first)) {              // fill the window: from this step's rows, the ring, or nothing
             const int pos = positions[t];
             const float* kept = ring + (size_t)slots[req] * TAPS * channels + c0;
 #pragma unroll
@@ -83,7 +92,7 @@ __global__ void __launch_bounds__(128) delta_conv_run_kernel(
             }
         }
         float now[8];
-        unpack8(*reinterpret_cast<const uint4*>(in + (size_t)t * in_stride + c0), now);
+        unpack8(raw[u], now);
         uint4 packed;
         __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&packed);
         float y[8];
@@ -122,7 +131,7 @@ __global__ void delta_ring_kernel(const T* __restrict__ in, int in_stride, float
     for (int t = first; t < end; ++t) kept[(size_t)(positions[t] % taps) * channels + c] = to_f32(in[(size_t)t * in_stride + c]);
 }
 
-// Tokens first_token .. tokens - 1, requests first_req .. requests - 1; out: [tokens][channels].
+// w: float32 [taps][channels], the last row meets the current token.  Tokens first_token .. tokens - 1, requests first_req .. requests - 1; out: [tokens][channels].
 MB_API int mb_delta_conv(const void* in, int in_stride, int dtype, const float* w, const float* ring, const int* positions, const int* req_index,
                          const int* cu_tokens, const int* slots, void* out, int first_token, int tokens, int channels, int taps, cudaStream_t s) {
     if (tokens <= first_token) return 0;
@@ -131,7 +140,7 @@ MB_API int mb_delta_conv(const void* in, int in_stride, int dtype, const float* 
     if (dtype == MB_F32)
         return launch_kernel(delta_conv_kernel<float>, grid, 128, 0, s, 0, (const float*)in, in_stride, w, ring, positions, req_index, cu_tokens,
                              slots, (float*)out, first_token, channels, taps);
-    if (dtype == MB_BF16 && taps <= 4 && channels % 8 == 0 && in_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+    if (dtype == MB_BF16 && taps <= 4 && channels % 8 == 0 && in_stride % 8 == 0 && (((uintptr_t)in | (uintptr_t)out | (uintptr_t)w) & 15) == 0) {
         dim3 runs((tokens - first_token + CONV_RUN - 1) / CONV_RUN, (channels / 8 + 127) / 128);
 #define CONV_CASE(N)                                                                                                                              \
     if (taps == N)                                                                                                                                \
@@ -374,8 +383,12 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
     float* __restrict__ state, const int* __restrict__ positions, const int* __restrict__ seq_lens, const int* __restrict__ slots,
     const T* __restrict__ g, int g_stride, int gate, const float* __restrict__ norm_w, float eps, float factor, T* __restrict__ out, int out_stride, int H,
     int G, int d, int dv) {
+    // The state is asked for before the wait for the kernel ahead: only this kernel (and the prompt kernels) of an earlier step wrote it,
+    // and every step has kernels in between that let nothing start before all work ahead of them is done (its embedding, the norms);
+    // slots, positions and lengths are the step's inputs, copied before its first kernel.  All else waits.
+#ifdef PDL_LAUNCH_FIRST
     PDL_ENTER();
-    in = pdl_fresh(in); b_rows = pdl_fresh(b_rows); a_rows = pdl_fresh(a_rows); g = pdl_fresh(g); ring = pdl_fresh(ring); state = pdl_fresh(state);
+#endif
     extern __shared__ float smem[];
     const int d4 = (d + 3) / 4 * 4;
     float* qs = smem;                          // [d]
@@ -397,6 +410,10 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
         const int n = part + PARTS * j;
         s[j] = (owner && n < d) ? S[(size_t)n * groups] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+#ifndef PDL_LAUNCH_FIRST
+    PDL_ENTER();
+#endif
+    in = pdl_fresh(in); b_rows = pdl_fresh(b_rows); a_rows = pdl_fresh(a_rows); g = pdl_fresh(g); ring = pdl_fresh(ring);
     const float rate_raw = rate_log[head], beta_raw = to_f32(b_rows[(size_t)r * b_stride + head]);
     float decay_raw = 0.0f, decay_bias = 0.0f, gate_raw = 0.0f, norm_raw = 0.0f;         // asked for early, used late
     if (threadIdx.x < d) {
@@ -428,16 +445,16 @@ __global__ void __launch_bounds__(512) delta_single_kernel(
                     int at = pos_row - back;
                     at = at < 0 ? at + taps : at;
                     x[back - 1] = kept[(size_t)at * channels + c];
-                    y[back - 1] = conv_w[(size_t)c * taps + taps - 1 - back];
+                    y[back - 1] = conv_w[(size_t)(taps - 1 - back) * channels + c];
                 }
             }
 #pragma unroll
             for (int back = 3; back > 0; --back) sum = fmaf(y[back - 1], x[back - 1], sum);
         } else {
             for (int back = most; back > 0; --back)
-                sum = fmaf(conv_w[(size_t)c * taps + taps - 1 - back], kept[(size_t)((pos - back) % taps) * channels + c], sum);
+                sum = fmaf(conv_w[(size_t)(taps - 1 - back) * channels + c], kept[(size_t)((pos - back) % taps) * channels + c], sum);
         }
-        sum = silu_f(fmaf(conv_w[(size_t)c * taps + taps - 1], now, sum));
+        sum = silu_f(fmaf(conv_w[(size_t)(taps - 1) * channels + c], now, sum));
         if (taps > 1 && (i >= 2 * d || head == kh * share)) kept[(size_t)pos_row * channels + c] = now;
         sum = to_f32(from_f32<T>(sum));        // as the convolution of many tokens leaves it
         if (i < d) { qs[i] = sum; qq = fmaf(sum, sum, qq); }

@@ -57,6 +57,26 @@ __device__ __forceinline__ void mma3(float* c, const uint32_t* ah, const uint32_
     mma_bf16_16816(c, ah, bl0, bl1);
 }
 
+// The same into three sums (added up at the end): three chains of products instead of one three times as long.
+struct Sums3 {
+    float hh[2][4], lh[2][4], hl[2][4];
+    __device__ __forceinline__ void clear() {
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) hh[n][e] = lh[n][e] = hl[n][e] = 0.0f;
+    }
+    __device__ __forceinline__ void add(const uint32_t* ah, const uint32_t* al, const uint32_t* bh, const uint32_t* bl) {
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            mma_bf16_16816(hh[n], ah, bh[2 * n], bh[2 * n + 1]);
+            mma_bf16_16816(lh[n], al, bh[2 * n], bh[2 * n + 1]);
+            mma_bf16_16816(hl[n], ah, bl[2 * n], bl[2 * n + 1]);
+        }
+    }
+    __device__ __forceinline__ float at(int n, int e) const { return hh[n][e] + (lh[n][e] + hl[n][e]); }
+};
+
 // What a chunk and head leaves for the walk, in bf16 planes of [64][DQ] (W, Q+, K exp(G_63 - G), each hi then lo), [64][64] (P hi, lo),
 // then float32 U0 [64][dv] and exp(G_63) [DQ].
 #define PLANE (CH * DQ)
@@ -67,17 +87,17 @@ __device__ __forceinline__ void mma3(float* c, const uint32_t* ah, const uint32_
 // Where request r's chunks start among all chunks of the step (room is left for a partial chunk per request).
 __device__ __forceinline__ int first_chunk(const int* cu_tokens, int first_req, int r) { return (cu_tokens[r] - cu_tokens[first_req]) / CH + (r - first_req); }
 
-#define LDR (DQ + 2)                  // raw q and k rows in shared memory (bf16): rows fall into different banks
-#define LDG (DQ + 1)
+#define LDR (DQ + 8)                  // raw q and k rows in shared memory (bf16) and sums (float32): eight rows of four lanes meet all banks
+#define LDG (DQ + 8)
 #define LDL (CH + 4)
-#define PREP_SMEM(CHANNEL) (2 * CH * LDR * 2 + ((CHANNEL) ? CH * LDG : CH) * 4 + CH * LDL * 4 + 4 * CH * 4 + 16)
+#define PREP_SMEM(CHANNEL, dv) (2 * CH * LDR * 2 + ((CHANNEL) ? CH * LDG : CH) * 4 + CH * LDL * 4 + 4 * CH * 4 + CH * ((dv) + 8) * 2 + 16)
 #define PREP_THREADS 256
 
 template <bool CHANNEL>
 __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
     const bf16* __restrict__ qkv, const bf16* __restrict__ b_rows, int b_stride, const bf16* __restrict__ a_rows, int a_stride,
     const float* __restrict__ rate_log, const float* __restrict__ dt_bias, const int* __restrict__ cu_tokens, int first_req,
-    bf16* __restrict__ planes, float* __restrict__ floats, int H, int G, int dv) {
+    bf16* __restrict__ planes, float* __restrict__ floats, int H, int G, int dv, int a_vec) {
     PDL_ENTER();
     qkv = pdl_fresh(qkv); b_rows = pdl_fresh(b_rows); a_rows = pdl_fresh(a_rows);
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -98,17 +118,52 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
     const size_t slot = (size_t)(first_chunk(cu_tokens, first_req, req) + blockIdx.x) * H + head;
     bf16* out = planes + slot * CHUNK_BF16;
     float* fout = floats + slot * CHUNK_F32(dv);
-    // ---- q and k as the convolution left them; rows past the request's tokens are zero
-    for (int idx = tid; idx < 2 * CH * (DQ / 8); idx += PREP_THREADS) {
-        const int which = idx / (CH * (DQ / 8)), rest = idx % (CH * (DQ / 8));
-        const int row = rest / (DQ / 8), c = rest % (DQ / 8);
-        uint4 raw = make_uint4(0, 0, 0, 0);
-        if (row < rows) raw = *reinterpret_cast<const uint4*>(qkv + (size_t)(tok0 + row) * channels + (size_t)which * G * DQ + (size_t)kh * DQ + c * 8);
-        uint32_t* dst = reinterpret_cast<uint32_t*>((which ? sk : sq) + row * LDR + c * 8);
-        dst[0] = raw.x; dst[1] = raw.y; dst[2] = raw.z; dst[3] = raw.w;
+    // ---- q, k and v as the convolution left them; rows past the request's tokens are zero
+    bf16* sv = reinterpret_cast<bf16*>(s_qk + CH);             // [CH][dv + 8]
+    {
+        const bf16* base = qkv + (size_t)tok0 * channels;
+        for (int idx = tid; idx < 2 * CH * (DQ / 8); idx += PREP_THREADS) {
+            const int which = idx / (CH * (DQ / 8)), rest = idx % (CH * (DQ / 8));
+            const int row = rest / (DQ / 8), c = rest % (DQ / 8);
+            bf16* dst = (which ? sk : sq) + row * LDR + c * 8;
+            if (row < rows) cp_async16(dst, base + (size_t)row * channels + (size_t)which * G * DQ + (size_t)kh * DQ + c * 8);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        }
+        const int per = dv / 8;
+        for (int idx = tid; idx < CH * per; idx += PREP_THREADS) {
+            const int row = idx / per, c = idx - row * per;
+            bf16* dst = sv + row * (dv + 8) + c * 8;
+            if (row < rows) cp_async16(dst, base + (size_t)row * channels + (size_t)2 * G * DQ + (size_t)head * dv + c * 8);
+            else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        }
+        cp_async_commit();
     }
     const float rate = expf(rate_log[head]) * LOG2E;
-    if (CHANNEL) {
+    if (CHANNEL && a_vec) {
+        constexpr int ITERS = (CH * (DQ / 8) + PREP_THREADS - 1) / PREP_THREADS;
+        uint4 raw[ITERS];
+#pragma unroll
+        for (int u = 0; u < ITERS; ++u) {
+            const int idx = tid + u * PREP_THREADS, row = idx / (DQ / 8), c = idx % (DQ / 8) * 8;
+            raw[u] = make_uint4(0, 0, 0, 0);
+            if (row < rows) raw[u] = *reinterpret_cast<const uint4*>(a_rows + (size_t)(tok0 + row) * a_stride + (size_t)head * DQ + c);
+        }
+#pragma unroll
+        for (int u = 0; u < ITERS; ++u) {
+            const int idx = tid + u * PREP_THREADS, row = idx / (DQ / 8), c = idx % (DQ / 8) * 8;
+            if (row >= CH) continue;
+            const float4 d0 = *reinterpret_cast<const float4*>(dt_bias + head * DQ + c), d1 = *reinterpret_cast<const float4*>(dt_bias + head * DQ + c + 4);
+            const float bias[8] = {d0.x, d0.y, d0.z, d0.w, d1.x, d1.y, d1.z, d1.w};
+            const uint32_t w[4] = {raw[u].x, raw[u].y, raw[u].z, raw[u].w};
+            float* dst = sG + row * LDG + c;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 a2 = bf2(w[e]);
+                dst[2 * e] = row < rows ? -rate * softplus_f(a2.x + bias[2 * e]) : 0.0f;
+                dst[2 * e + 1] = row < rows ? -rate * softplus_f(a2.y + bias[2 * e + 1]) : 0.0f;
+            }
+        }
+    } else if (CHANNEL) {
         for (int idx = tid; idx < CH * DQ; idx += PREP_THREADS) {
             const int row = idx / DQ, c = idx % DQ;
             float lg = 0.0f;
@@ -119,6 +174,7 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
         sG[tid] = tid < rows ? -rate * softplus_f(__bfloat162float(a_rows[(size_t)(tok0 + tid) * a_stride + head]) + dt_bias[head]) : 0.0f;
     }
     if (tid < CH) s_beta[tid] = tid < rows ? 1.0f / (1.0f + expf(-__bfloat162float(b_rows[(size_t)(tok0 + tid) * b_stride + head]))) : 0.0f;
+    cp_async_wait<0>();
     __syncthreads();
     // ---- running sums of the log-decays; unit lengths
     if (CHANNEL) {
@@ -192,11 +248,12 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
             } else {
                 uint32_t kh_[4], kl_[4], qh_[4], ql_[4];
                 if (I > 0) {
-                    const float r[4] = {ref[c], ref[c + 1], ref[c + 8], ref[c + 9]};
+                    const float2 ra = *reinterpret_cast<const float2*>(ref + c), rb = *reinterpret_cast<const float2*>(ref + c + 8);
+                    const float r[4] = {ra.x, ra.y, rb.x, rb.y};
 #pragma unroll
                     for (int u = 0; u < 4; ++u) {
-                        const float* gi = sG + ((u & 1) ? i1 : i0) * LDG + c + (u >> 1) * 8;
-                        const float e0 = ex2_approx(gi[0] - r[(u >> 1) * 2]), e1 = ex2_approx(gi[1] - r[(u >> 1) * 2 + 1]);
+                        const float2 gi = *reinterpret_cast<const float2*>(sG + ((u & 1) ? i1 : i0) * LDG + c + (u >> 1) * 8);
+                        const float e0 = ex2_approx(gi.x - r[(u >> 1) * 2]), e1 = ex2_approx(gi.y - r[(u >> 1) * 2 + 1]);
                         const float2 k2 = bf2(rk[u]), q2 = bf2(rq[u]);
                         split_bf16(k2.x * e0, k2.y * e1, kh_[u], kl_[u]);
                         split_bf16(q2.x * e0, q2.y * e1, qh_[u], ql_[u]);
@@ -205,31 +262,32 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
                     for (int J = 0; J < 3; ++J) {
                         if (J >= I) continue;
                         const int j = J * 16 + half * 8 + g;
-                        const float* gj = sG + j * LDG + c;
+                        const float2 ga = *reinterpret_cast<const float2*>(sG + j * LDG + c), gb = *reinterpret_cast<const float2*>(sG + j * LDG + c + 8);
                         const float2 x = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c)), y = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c + 8));
                         uint32_t bh0, bl0, bh1, bl1;
-                        split_bf16(x.x * ex2_approx(r[0] - gj[0]), x.y * ex2_approx(r[1] - gj[1]), bh0, bl0);
-                        split_bf16(y.x * ex2_approx(r[2] - gj[8]), y.y * ex2_approx(r[3] - gj[9]), bh1, bl1);
+                        split_bf16(x.x * ex2_approx(r[0] - ga.x), x.y * ex2_approx(r[1] - ga.y), bh0, bl0);
+                        split_bf16(y.x * ex2_approx(r[2] - gb.x), y.y * ex2_approx(r[3] - gb.y), bh1, bl1);
                         mma3(accA[J], kh_, kl_, bh0, bh1, bl0, bl1);
                         mma3(accP[J], qh_, ql_, bh0, bh1, bl0, bl1);
                     }
                 }
                 if (half == 0) {                               // rows 8 .. 15 of the block (the operands of rows 0 .. 7 are zero)
-                    const float r[4] = {mid[c], mid[c + 1], mid[c + 8], mid[c + 9]};
+                    const float2 ra = *reinterpret_cast<const float2*>(mid + c), rb = *reinterpret_cast<const float2*>(mid + c + 8);
+                    const float r[4] = {ra.x, ra.y, rb.x, rb.y};
                     kh_[0] = kh_[2] = kl_[0] = kl_[2] = qh_[0] = qh_[2] = ql_[0] = ql_[2] = 0u;
 #pragma unroll
                     for (int u = 1; u < 4; u += 2) {
-                        const float* gi = sG + i1 * LDG + c + (u >> 1) * 8;
-                        const float e0 = ex2_approx(gi[0] - r[(u >> 1) * 2]), e1 = ex2_approx(gi[1] - r[(u >> 1) * 2 + 1]);
+                        const float2 gi = *reinterpret_cast<const float2*>(sG + i1 * LDG + c + (u >> 1) * 8);
+                        const float e0 = ex2_approx(gi.x - r[(u >> 1) * 2]), e1 = ex2_approx(gi.y - r[(u >> 1) * 2 + 1]);
                         const float2 k2 = bf2(rk[u]), q2 = bf2(rq[u]);
                         split_bf16(k2.x * e0, k2.y * e1, kh_[u], kl_[u]);
                         split_bf16(q2.x * e0, q2.y * e1, qh_[u], ql_[u]);
                     }
-                    const float* gj = sG + i0 * LDG + c;      // token g of the block: the same index as row i0
+                    const float2 ga = *reinterpret_cast<const float2*>(sG + i0 * LDG + c), gb = *reinterpret_cast<const float2*>(sG + i0 * LDG + c + 8);   // token g of the block: the same index as row i0
                     const float2 x = bf2(rk[0]), y = bf2(rk[2]);
                     uint32_t bh0, bl0, bh1, bl1;
-                    split_bf16(x.x * ex2_approx(r[0] - gj[0]), x.y * ex2_approx(r[1] - gj[1]), bh0, bl0);
-                    split_bf16(y.x * ex2_approx(r[2] - gj[8]), y.y * ex2_approx(r[3] - gj[9]), bh1, bl1);
+                    split_bf16(x.x * ex2_approx(r[0] - ga.x), x.y * ex2_approx(r[1] - ga.y), bh0, bl0);
+                    split_bf16(y.x * ex2_approx(r[2] - gb.x), y.y * ex2_approx(r[3] - gb.y), bh1, bl1);
                     mma3(accA[3], kh_, kl_, bh0, bh1, bl0, bl1);
                     mma3(accP[3], qh_, ql_, bh0, bh1, bl0, bl1);
                 }
@@ -267,7 +325,8 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
             for (int c = 0; c < DQ; c += 2) {
                 const float2 ki = bf2(*reinterpret_cast<const uint32_t*>(sk + i * LDR + c)), kj = bf2(*reinterpret_cast<const uint32_t*>(sk + j * LDR + c));
                 const float2 qi = bf2(*reinterpret_cast<const uint32_t*>(sq + i * LDR + c));
-                const float x = kj.x * ex2_approx(sG[i * LDG + c] - sG[j * LDG + c]), y = kj.y * ex2_approx(sG[i * LDG + c + 1] - sG[j * LDG + c + 1]);
+                const float2 gi = *reinterpret_cast<const float2*>(sG + i * LDG + c), gj = *reinterpret_cast<const float2*>(sG + j * LDG + c);
+                const float x = kj.x * ex2_approx(gi.x - gj.x), y = kj.y * ex2_approx(gi.y - gj.y);
                 a = fmaf(ki.x, x, a); a = fmaf(ki.y, y, a);
                 b = fmaf(qi.x, x, b); b = fmaf(qi.y, y, b);
             }
@@ -305,12 +364,12 @@ __global__ void __launch_bounds__(PREP_THREADS, 2) prepare_kernel(
     // ---- forward substitution, a column per thread: x_i = rhs_i - sum_(j < i) L_ij x_j
     for (int col = tid; col < DQ + dv; col += PREP_THREADS) {
         const bool is_w = col < DQ;
-        const bf16* v = qkv + (size_t)tok0 * channels + (size_t)2 * G * DQ + (size_t)head * dv + (col - DQ);
+        const bf16* v = sv + (col - DQ);
         float x[CH];
 #pragma unroll
         for (int i = 0; i < CH; ++i) {
             if (is_w) x[i] = s_beta[i] * s_fk[i] * __bfloat162float(sk[i * LDR + col]) * ex2_approx(CHANNEL ? sG[i * LDG + col] : sG[i]);
-            else x[i] = i < rows ? s_beta[i] * __bfloat162float(v[(size_t)i * channels]) : 0.0f;
+            else x[i] = s_beta[i] * __bfloat162float(v[i * (dv + 8)]);
         }
 #pragma unroll
         for (int i = 1; i < CH; ++i) {
@@ -464,7 +523,8 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
         load_k(c);                                     // everyone has left the chunk before
         // U = U0 - W S
         {
-            float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            Sums3 acc;
+            acc.clear();
 #pragma unroll
             for (int kk = 0; kk < DQ / 16; ++kk) {
                 uint32_t ah[4], al[4], bh[4], bl[4];
@@ -472,16 +532,15 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
                 ldsm_x4(w_addr + PL_Q + kk * 32, al[0], al[1], al[2], al[3]);
                 ldsm_x4_trans(s_addr + kk * 16 * LDS * 2, bh[0], bh[1], bh[2], bh[3]);
                 ldsm_x4_trans(s_addr + PL_S + kk * 16 * LDS * 2, bl[0], bl[1], bl[2], bl[3]);
-                mma3(acc[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                mma3(acc[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                acc.add(ah, al, bh, bl);
             }
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
                 uint32_t hi, lo;
-                split_bf16(u[nt][0] - acc[nt][0], u[nt][1] - acc[nt][1], hi, lo);
+                split_bf16(u[nt][0] - acc.at(nt, 0), u[nt][1] - acc.at(nt, 1), hi, lo);
                 *reinterpret_cast<uint32_t*>(sU + i0 * LDS + col + nt * 8) = hi;
                 *reinterpret_cast<uint32_t*>(sU + CH * LDS + i0 * LDS + col + nt * 8) = lo;
-                split_bf16(u[nt][2] - acc[nt][2], u[nt][3] - acc[nt][3], hi, lo);
+                split_bf16(u[nt][2] - acc.at(nt, 2), u[nt][3] - acc.at(nt, 3), hi, lo);
                 *reinterpret_cast<uint32_t*>(sU + i1 * LDS + col + nt * 8) = hi;
                 *reinterpret_cast<uint32_t*>(sU + CH * LDS + i1 * LDS + col + nt * 8) = lo;
             }
@@ -491,7 +550,8 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
         load_w(c + 1);                                 // everyone is done with W
         // O = Q+ S + P U
         {
-            float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            Sums3 acc;
+            acc.clear();
 #pragma unroll
             for (int kk = 0; kk < DQ / 16; ++kk) {
                 uint32_t ah[4], al[4], bh[4], bl[4];
@@ -499,8 +559,7 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
                 ldsm_x4(q_addr + PL_Q + kk * 32, al[0], al[1], al[2], al[3]);
                 ldsm_x4_trans(s_addr + kk * 16 * LDS * 2, bh[0], bh[1], bh[2], bh[3]);
                 ldsm_x4_trans(s_addr + PL_S + kk * 16 * LDS * 2, bl[0], bl[1], bl[2], bl[3]);
-                mma3(acc[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                mma3(acc[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                acc.add(ah, al, bh, bl);
             }
 #pragma unroll
             for (int kk = 0; kk < CH / 16; ++kk) {
@@ -510,14 +569,13 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
                 ldsm_x4(p_addr + PL_P + kk * 32, al[0], al[1], al[2], al[3]);
                 ldsm_x4_trans(u_addr + (kk * 16 * LDS + wc * 16) * 2, bh[0], bh[1], bh[2], bh[3]);
                 ldsm_x4_trans(u_addr + PL_U + (kk * 16 * LDS + wc * 16) * 2, bl[0], bl[1], bl[2], bl[3]);
-                mma3(acc[0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                mma3(acc[1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                acc.add(ah, al, bh, bl);
             }
             float* dst = o + (size_t)(first + c * CH) * o_stride + (size_t)head * dv + vs0 + col;
 #pragma unroll
             for (int nt = 0; nt < 2; ++nt) {
-                if (i0 < rows) *reinterpret_cast<float2*>(dst + (size_t)i0 * o_stride + nt * 8) = make_float2(acc[nt][0], acc[nt][1]);
-                if (i1 < rows) *reinterpret_cast<float2*>(dst + (size_t)i1 * o_stride + nt * 8) = make_float2(acc[nt][2], acc[nt][3]);
+                if (i0 < rows) *reinterpret_cast<float2*>(dst + (size_t)i0 * o_stride + nt * 8) = make_float2(acc.at(nt, 0), acc.at(nt, 1));
+                if (i1 < rows) *reinterpret_cast<float2*>(dst + (size_t)i1 * o_stride + nt * 8) = make_float2(acc.at(nt, 2), acc.at(nt, 3));
             }
         }
         cp_async_wait<1>();                            // K
@@ -528,24 +586,28 @@ __global__ void __launch_bounds__(WALK_THREADS) walk_kernel(const bf16* __restri
         for (int mi = 0; mi < MT_W; ++mi) {
             const int m0 = (warp + WARPS * mi) * 16;
             if (m0 < DQ) {
-#pragma unroll
-                for (int nt = 0; nt < NT; ++nt) { S[mi][nt][0] *= last[mi][0]; S[mi][nt][1] *= last[mi][0]; S[mi][nt][2] *= last[mi][1]; S[mi][nt][3] *= last[mi][1]; }
                 // K^T as the row operand: tokens are its columns, read transposed from the [token][channel] tile
                 const uint32_t k_addr = (uint32_t)__cvta_generic_to_shared(sK + ((lane & 7) + (lane >> 4) * 8) * LDQ + m0 + ((lane >> 3) & 1) * 8);
+                Sums3 acc[NT / 2];
+#pragma unroll
+                for (int dt = 0; dt < NT / 2; ++dt) acc[dt].clear();
 #pragma unroll
                 for (int kk = 0; kk < CH / 16; ++kk) {
                     uint32_t ah[4], al[4];
                     ldsm_x4_trans(k_addr + kk * 16 * LDQ * 2, ah[0], ah[1], ah[2], ah[3]);
                     ldsm_x4_trans(k_addr + PL_Q + kk * 16 * LDQ * 2, al[0], al[1], al[2], al[3]);
 #pragma unroll
-                    for (int dt = 0; dt < NT; dt += 2) {
+                    for (int dt = 0; dt < NT / 2; ++dt) {
                         uint32_t bh[4], bl[4];
-                        ldsm_x4_trans(u_addr + (kk * 16 * LDS + dt * 8) * 2, bh[0], bh[1], bh[2], bh[3]);
-                        ldsm_x4_trans(u_addr + PL_U + (kk * 16 * LDS + dt * 8) * 2, bl[0], bl[1], bl[2], bl[3]);
-                        mma3(S[mi][dt], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                        mma3(S[mi][dt + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+                        ldsm_x4_trans(u_addr + (kk * 16 * LDS + dt * 16) * 2, bh[0], bh[1], bh[2], bh[3]);
+                        ldsm_x4_trans(u_addr + PL_U + (kk * 16 * LDS + dt * 16) * 2, bl[0], bl[1], bl[2], bl[3]);
+                        acc[dt].add(ah, al, bh, bl);
                     }
                 }
+#pragma unroll
+                for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) S[mi][nt][e] = fmaf(S[mi][nt][e], last[mi][e >> 1], acc[nt >> 1].at(nt & 1, e));
             }
         }
     }
@@ -576,15 +638,16 @@ MB_API int mb_delta_chunked(const void* qkv, const void* b_rows, int b_stride, c
     if (H <= 0 || G <= 0 || H % G != 0 || dv <= 0 || dv % VS != 0 || first_req < 0 || ((2 * G * DQ + H * dv) % 8) != 0) return MB_ERR_BAD_SIZE;
     if ((((uintptr_t)qkv | (uintptr_t)planes) & 15) != 0 || ((uintptr_t)floats & 7) != 0) return MB_ERR_BAD_SIZE;
     if (which == 0) {
+        const int a_vec = a_stride % 8 == 0 && (((uintptr_t)a_rows | (uintptr_t)dt_bias) & 15) == 0;      // decays per channel by 16-byte loads
         dim3 grid((max_query_len + CH - 1) / CH, H, requests - first_req);
         if (per_channel) {
-            cudaFuncSetAttribute(prepare_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PREP_SMEM(1));
-            return launch_kernel(prepare_kernel<true>, grid, PREP_THREADS, PREP_SMEM(1), s, 0, (const bf16*)qkv, (const bf16*)b_rows, b_stride,
-                                 (const bf16*)a_rows, a_stride, rate_log, dt_bias, cu_tokens, first_req, (bf16*)planes, floats, H, G, dv);
+            cudaFuncSetAttribute(prepare_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PREP_SMEM(1, dv));
+            return launch_kernel(prepare_kernel<true>, grid, PREP_THREADS, PREP_SMEM(1, dv), s, 0, (const bf16*)qkv, (const bf16*)b_rows, b_stride,
+                                 (const bf16*)a_rows, a_stride, rate_log, dt_bias, cu_tokens, first_req, (bf16*)planes, floats, H, G, dv, a_vec);
         }
-        cudaFuncSetAttribute(prepare_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PREP_SMEM(0));
-        return launch_kernel(prepare_kernel<false>, grid, PREP_THREADS, PREP_SMEM(0), s, 0, (const bf16*)qkv, (const bf16*)b_rows, b_stride,
-                             (const bf16*)a_rows, a_stride, rate_log, dt_bias, cu_tokens, first_req, (bf16*)planes, floats, H, G, dv);
+        cudaFuncSetAttribute(prepare_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PREP_SMEM(0, dv));
+        return launch_kernel(prepare_kernel<false>, grid, PREP_THREADS, PREP_SMEM(0, dv), s, 0, (const bf16*)qkv, (const bf16*)b_rows, b_stride,
+                             (const bf16*)a_rows, a_stride, rate_log, dt_bias, cu_tokens, first_req, (bf16*)planes, floats, H, G, dv, a_vec);
     }
     cudaFuncSetAttribute(walk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, WALK_SMEM);
     return launch_kernel(walk_kernel, dim3(requests - first_req, H, dv / VS), WALK_THREADS, WALK_SMEM, s, 0, (const bf16*)planes, (const float*)floats,

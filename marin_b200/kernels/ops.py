@@ -2015,13 +2015,13 @@ def _columns(t: torch.Tensor, T: int, n: int, dtype) -> int:
 def delta_conv(qkv: torch.Tensor, weight: torch.Tensor, ring: torch.Tensor, ctx, slots: torch.Tensor, out: torch.Tensor, first_req: int = 0,
                first_token: int = 0) -> None:
     """A causal convolution over time per channel, then silu, of the step's tokens from ``first_token`` on (the tokens of the requests from
-    ``first_req`` on); ``weight`` float32 ``[channels, taps]``, its last column on the current token.  ``ring`` (float32 ``[slots, taps,
+    ``first_req`` on); ``weight`` float32 ``[taps, channels]``, its last row on the current token.  ``ring`` (float32 ``[slots, taps,
     channels]``) keeps every request's latest inputs, that of position ``p`` in row ``p mod taps``, and is brought up to date."""
     _need_cuda(weight, ring, out, slots)
     T, channels = out.shape
-    taps = weight.shape[1]
+    taps = weight.shape[0]
     stride = _columns(qkv, T, channels, out.dtype)
-    assert weight.dtype == torch.float32 and weight.shape[0] == channels and ring.dtype == torch.float32 and tuple(ring.shape[1:]) == (taps, channels)
+    assert weight.dtype == torch.float32 and weight.shape[1] == channels and ring.dtype == torch.float32 and tuple(ring.shape[1:]) == (taps, channels)
     lib = _lib("mb_delta_rule")
     _cost(2 * (T - first_token) * channels * out.element_size(), 2.0 * (T - first_token) * channels * taps)
     _check(lib.mb_delta_conv(_c_void_p(qkv.data_ptr()), _c_int(stride), _code(out), _ptr(weight), _ptr(ring), _ptr(ctx.positions), _ptr(ctx.req_index),
@@ -2091,7 +2091,7 @@ def delta_single(qkv: torch.Tensor, conv_w: torch.Tensor, ring: torch.Tensor, in
     kernel; ``qkv`` as the projection left it, ``out`` a column block ``[T, H dv]``."""
     _need_cuda(conv_w, ring, state, norm_w, slots)
     T = qkv.shape[0]
-    channels, taps = 2 * G * d + H * dv, conv_w.shape[1]
+    channels, taps = 2 * G * d + H * dv, conv_w.shape[0]
     dtype = qkv.dtype
     _cost(requests * (2.0 * H * d * dv * 4 + channels * (2 * dtype.itemsize + taps * 4)), 6.0 * requests * H * d * dv)
     _check(_lib("mb_delta_rule").mb_delta_single(

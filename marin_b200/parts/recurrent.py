@@ -344,7 +344,7 @@ class DeltaRule(Mixer):
                 self.high_cols[whole] = (c, second.shape[0])
                 r, c = r + width, c + second.shape[0]
             self.w_low, self.w_high = rt.matrix(first_all), rt.matrix(second_all)
-        self.conv_w = rt.f32(torch.cat([tensors.pop(self._n(f"{p}_conv")).to(torch.float32) for p in "qkv"], dim=0))
+        self.conv_w = rt.f32(torch.cat([tensors.pop(self._n(f"{p}_conv")).to(torch.float32) for p in "qkv"], dim=0).t())     # [taps, channels]
         self.rate, self.dt_bias, self.norm_w = (rt.f32(tensors.pop(self._n(k))) for k in ("rate", "dt_bias", "norm"))
         self.w_o = rt.matrix(tensors.pop(self._n("o")))
         self.rt = rt
