@@ -106,6 +106,12 @@ class Mixer(Part):
     #: pad a captured batch stand for empty requests: length 0, the spare state slot (see ``CacheManager``).
     capturable = True
 
+    #: True if the mixer's work is one product of its input, something over the cache, and one product of the result: it then has
+    #: ``w_in`` (the first product's matrix), ``w_o`` and ``o_dim``, and ``forward`` takes ``rows`` (the first product's result, a column
+    #: block of a wider one) and ``out`` (a column block ``[T, o_dim]`` to leave the result in; nothing is projected or added then), so
+    #: that mixers side by side can share both products.
+    joins_products = False
+
     def cache_need(self):
         return None
 
@@ -454,16 +460,19 @@ class SinkAttention(Mixer):
         return ops.sink_decode_plan(rt.dtype, requests, self.heads, self.kv_heads, self.head_dim, self.v_head_dim, span,
                                     self.window or 0, self.chunk or 0, keep_first=self.keep_first)
 
-    def forward(self, x, ctx, cache, residual: torch.Tensor):
+    joins_products = True
+
+    def forward(self, x, ctx, cache, residual: torch.Tensor, rows=None, out=None):
         T = x.shape[0]
         ws = ctx.workspace
         writes = cache.owner
         if not writes and self.gate:
             raise ValueError("sink_attention: a gated layer cannot read another run's cache")   # its columns lie behind k and v
         w = self.w_in if writes else self.w_in[: self.q_dim]
-        ops.stage_name = "q|k|v|g"
-        rows = ws.get("qkvg", (T, w.shape[0]), x.dtype)
-        ops.gemm(x, w, rows)
+        if rows is None:
+            ops.stage_name = "q|k|v|g"
+            rows = ws.get("qkvg", (T, w.shape[0]), x.dtype)
+            ops.gemm(x, w, rows)
         ops.stage_name = "heads"
         q = ws.get("q", (T, self.q_dim), x.dtype)
         shared = None
@@ -476,7 +485,9 @@ class SinkAttention(Mixer):
         ops.qkv_finish(rows, q, self.q_b, self.k_b, self.v_b, self.qk_norm, self.q_weight, self.k_weight, self.norm_eps, ctx.positions,
                        pos.inv_freq, pos.rotary_dim, pos.magnitude, cache.slot_mapping, cache.k, cache.v, mode, shared, self.lam,
                        self.heads, self.kv_heads, self.head_dim, self.v_head_dim, writes, pos.interleaved)
-        out = ws.get("attn_out", (T, self.o_dim), x.dtype)
+        joined = out is not None
+        if not joined:
+            out = ws.get("attn_out", (T, self.o_dim), x.dtype)
         ops.stage_name = "attention"
         gate = rows[:, self.q_dim + self.k_dim + self.v_dim:] if self.gate else None
         plans = ctx.decode_plans
@@ -484,6 +495,8 @@ class SinkAttention(Mixer):
                            self.scale, self.window or 0, self.chunk or 0, self.sink, gate,
                            plans.get(self.decode_plan_key()) if plans else None, self.sink_logits, self.keep_first, self.softcap or 0.0,
                            self.out_scale)
+        if joined:
+            return None
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
         return None
@@ -817,11 +830,23 @@ class ShiftedMixer(Mixer):
         return self.inner.forward(shifted[0], ctx, inner_cache, residual)
 
 
+def _leaves(views):
+    """The views of a mixer that keeps several things, one by one."""
+    for v in views:
+        if isinstance(v, (tuple, list)):
+            yield from _leaves(v)
+        elif v is not None:
+            yield v
+
+
 @register_mixer("parallel_mixers")
 class ParallelMixers(Mixer):
     """Several mixers side by side on the same rows: ``sum_i scale_i mixer_i(x)``.  ``inner`` gives the mixers by name (their tensors lie in
     ``<name>.<inner name>``), ``scales`` their weights; an inner mixer takes its weight as its parameter ``out_scale``.  What each keeps between
-    steps is kept side by side: ``cache_need`` answers the tuple of their needs, the view is the tuple of their views."""
+    steps is kept side by side: ``cache_need`` answers the tuple of their needs, the view is the tuple of their views.
+
+    Where all of them allow it (``Mixer.joins_products``) their first products are one product of the input and, where their
+    results' widths are multiples of 8, their last ones one product of the results side by side."""
 
     def __init__(self, hidden: int, inner: Dict[str, PartSpec], name: str, scales: Optional[Dict[str, float]] = None):
         self.hidden, self.name = int(hidden), name
@@ -840,6 +865,23 @@ class ParallelMixers(Mixer):
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         for m in self.inner:
             m.load(tensors, rt)
+        self.w_in = self.w_o = None
+        if all(m.joins_products for m in self.inner):
+            # one matrix each; the inner mixers keep views of their blocks of the first (blocks start at multiples of 8 rows, so that
+            # every kernel can take them by 16-byte loads)
+            blocks, at, self.cols = [], 0, []
+            for m in self.inner:
+                n = m.w_in.shape[0]
+                self.cols.append((at, n))
+                blocks += [m.w_in, m.w_in.new_zeros(-n % 8, m.w_in.shape[1])]
+                at += n + -n % 8
+            self.w_in = torch.cat(blocks, dim=0).contiguous()
+            for m, (first, n) in zip(self.inner, self.cols):
+                m.w_in = self.w_in[first:first + n]
+            if all(m.o_dim % 8 == 0 for m in self.inner):     # (results side by side, each at a 16-byte boundary; else each has its own product)
+                self.w_o = torch.cat([m.w_o for m in self.inner], dim=1).contiguous()
+                for m in self.inner:
+                    m.w_o = None
         self.rt = rt
 
     def bytes_read(self, tokens: int, dtype) -> int:
@@ -876,7 +918,22 @@ class ParallelMixers(Mixer):
         outer = ctx.decode_plans
         if own:
             ctx.decode_plans = {**outer, **own}
-        for m, view in zip(self.inner, cache):
-            m.forward(x, ctx, view, residual)
+        if self.w_in is None:
+            for m, view in zip(self.inner, cache):
+                m.forward(x, ctx, view, residual)
+        else:
+            if not all(view.owner for view in _leaves(cache)):
+                raise ValueError("parallel_mixers: mixers that share their products cannot read another run's cache")
+            ops.stage_name = "inputs of both"
+            rows = ctx.workspace.get("joined_rows", (x.shape[0], self.w_in.shape[0]), x.dtype)
+            ops.gemm(x, self.w_in, rows)
+            outs = ctx.workspace.get("joined_out", (x.shape[0], self.w_o.shape[1]), x.dtype) if self.w_o is not None else None
+            at = 0
+            for m, view, (first, n) in zip(self.inner, cache, self.cols):
+                m.forward(x, ctx, view, residual, rows=rows[:, first:first + n], out=outs[:, at:at + m.o_dim] if outs is not None else None)
+                at += m.o_dim
+            if outs is not None:
+                ops.stage_name = "o"
+                ops.gemm(outs, self.w_o, residual, accumulate=True)
         ctx.decode_plans = outer
         return None

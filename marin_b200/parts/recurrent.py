@@ -294,6 +294,7 @@ class DeltaRule(Mixer):
         self.qk, self.hv = self.kv_heads * self.dim, self.heads * self.vdim
         self.channels = 2 * self.qk + self.hv
         self.decays = self.heads * self.dim if decay == "channel" else self.heads
+        self.o_dim = self.hv
         self.w_in = self.w_low = self.w_high = self.w_o = None
 
     def _n(self, key: str) -> str:
@@ -361,14 +362,17 @@ class DeltaRule(Mixer):
         chunked = self.heads * ops.delta_chunk_bytes(self.dim, self.vdim) // 64 if ops.delta_chunked_supported(dtype, self.dim, self.vdim) else 0
         return self.channels * element_size(dtype) + 4 * self.hv + chunked
 
-    def forward(self, x, ctx, cache, residual: torch.Tensor):
+    joins_products = True
+
+    def forward(self, x, ctx, cache, residual: torch.Tensor, rows=None, out=None):
         T = x.shape[0]
         ws = ctx.workspace
         H, G, d, dv = self.heads, self.kv_heads, self.dim, self.vdim
         matrices, ring = cache
-        ops.stage_name = "q|k|v|b"
-        rows = ws.get("delta_rows", (T, self.w_in.shape[0]), x.dtype)
-        ops.gemm(x, self.w_in, rows)
+        if rows is None:
+            ops.stage_name = "q|k|v|b"
+            rows = ws.get("delta_rows", (T, self.w_in.shape[0]), x.dtype)
+            ops.gemm(x, self.w_in, rows)
         high = None
         if self.w_low is not None:
             ops.stage_name = "decay, gate"
@@ -383,7 +387,9 @@ class DeltaRule(Mixer):
 
         inputs = ops.DeltaInputs(block("b"), block("a"), block("g"), self.rate, self.dt_bias)
         qkv = block("qkv")
-        out = ws.get("delta_out", (T, self.hv), x.dtype)
+        joined = out is not None
+        if not joined:
+            out = ws.get("delta_out", (T, self.hv), x.dtype)
         ops.stage_name = "delta rule"
         single = ctx.num_decode if ops.use_delta_single and ops.delta_single_supported(d, dv) else 0
         if single:                                             # requests with one token each come first in the batch
@@ -402,6 +408,8 @@ class DeltaRule(Mixer):
                 ops.delta_scan(conv, inputs, matrices.state, ctx, matrices.slots, o, H, G, d, dv, single)
             ops.stage_name = "norm, gate"
             ops.delta_norm(o, inputs.gate, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, H, dv, single)
+        if joined:
+            return None
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
         return None

@@ -67,13 +67,13 @@ CONFIG_B = {"architecture": "Pununex", "vocab": 170, "width": 128, "norm": {"eps
                         "mlp": _moe(128, 6, 1, identity=2, groups=(2, 1), scale=1.0, shared=64)}]}
 # Edges of the parameter space: no bigram embedding, no feed-forward, no mask, no cap, a window of one position, more kept
 # positions than the window is long, nothing kept, a convolution of a single tap, no identity outputs, no groups, all groups kept,
-# no shared expert, every expert chosen, decays of 16 channels over values of 128 and of 128 over 16.
+# no shared expert, every expert chosen, key heads much smaller and larger than the value heads.
 CONFIG_C = {"architecture": "Pununex", "vocab": 70, "width": 64, "norm": {"eps": 1e-6},
-            "layers": [{"type": "parallel", "mixer": _parallel(_attn(2, 2, 16, 16, 0.25), _delta(2, 1, 16, 128, 1), 1.0, 1.0), "mlp": None},
-                       {"type": "parallel", "mixer": _parallel(_attn(4, 1, 32, 48, 0.2, size=1, keep=2), _delta(1, 1, 128, 16, 2), 0.3, 0.9),
+            "layers": [{"type": "parallel", "mixer": _parallel(_attn(2, 2, 16, 16, 0.25), _delta(2, 1, 32, 128, 1), 1.0, 1.0), "mlp": None},
+                       {"type": "parallel", "mixer": _parallel(_attn(4, 1, 32, 48, 0.2, size=1, keep=2), _delta(1, 1, 128, 9, 2), 0.3, 0.9),
                         "mlp": _moe(32, 4, 4)},
                        {"type": "delta", "mixer": _delta(2, 2, 16, 16, 7), "mlp": _moe(64, 4, 2, groups=(2, 2), scale=0.5)},
-                       {"type": "parallel", "mixer": _parallel(_attn(2, 1, 16, 32, 0.3, size=24, softcap=3.0), _delta(3, 1, 16, 32, 4), 0.6, 0.6),
+                       {"type": "parallel", "mixer": _parallel(_attn(2, 1, 16, 32, 0.3, size=24, softcap=3.0), _delta(3, 1, 16, 48, 4), 0.6, 0.6),
                         "mlp": _moe(64, 2, 2, identity=2, shared=32)}]}
 CONFIGS = {"A": CONFIG_A, "B": CONFIG_B, "C": CONFIG_C}
 PAGE = {"A": 4, "B": 16, "C": 8}

@@ -147,7 +147,7 @@ def delta_part(m, hidden, eps, rt, w, per_channel):
 
 
 DELTAS = [_delta(4, 2, 10, 14, 3), _delta(2, 2, 64, 64, 4), _delta(6, 2, 32, 48, 2), _delta(1, 1, 128, 128, 4), _delta(3, 1, 16, 80, 7),
-          _delta(2, 1, 160, 32, 1), _delta(2, 2, 48, 12, 5), _delta(2, 1, 112, 256, 4), _delta(5, 5, 7, 6, 2)]
+          _delta(2, 1, 160, 32, 1), _delta(2, 2, 48, 12, 5), _delta(2, 1, 64, 256, 4), _delta(5, 5, 7, 6, 2)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -217,7 +217,7 @@ def recurrence(q, k, v, beta_raw, a_raw, rate, dt_bias, state, cuts, H, G, d, dv
 @pytest.mark.parametrize("chunked", [False, True], ids=["scan", "chunked"])
 @pytest.mark.parametrize("per_channel", [False, True], ids=["head", "channel"])
 @pytest.mark.parametrize("strength", [0.002, 0.3, 4.0, 60.0])
-@pytest.mark.parametrize("d,dv", [(32, 32), (64, 48), (128, 32)])
+@pytest.mark.parametrize("d,dv", [(32, 48), (64, 32), (128, 32)])
 def test_the_recurrence_is_exact_for_weak_and_strong_decays(chunked, per_channel, strength, d, dv):
     """The recurrence's own arithmetic is 32-bit: on bf16 inputs taken as they are the result and the final state agree with float64
     to about 1e-4, whatever the decays: from nothing forgotten to everything forgotten within a token (where the exponent of a
@@ -634,6 +634,6 @@ def test_the_command_line_takes_a_pununex_folder(tmp_path):
     e = subprocess.run(run + ["bench", model, "--prompt-tokens", "16", "--tokens", "8", "--runs", "2", "--warmup", "1", "--profile"],
                        capture_output=True, text=True)
     assert e.returncode == 0, e.stderr
-    for stage in ("embedding", "norm into the stream", "q|k|v", "attention", "delta rule", "convolution", "decay, gate", "router", "experts", "gate|up, relu",
+    for stage in ("embedding", "norm into the stream", "inputs of both", "q|k|v|b", "attention", "delta rule", "convolution", "decay, gate", "router", "experts", "gate|up, relu",
                   "head", "sampling"):
         assert stage in e.stdout, stage
