@@ -27,6 +27,8 @@ depth, vocabulary and heads, the closest of the engine's models (attention with 
 ``--arch vogunex`` measures Vogunex layers (attention over a window and pooled blocks with mixed head weights, a state space
 layer, attention over a shared latent with a window, in turn; dense and routed feed-forwards; a token shift before every
 mixer) beside the Nirotar layers at the same sizes, the closest of the engine's models.
+``--arch pununex`` measures Pununex layers (windowed attention with kept first positions beside a gated delta rule, and a delta
+rule alone, in turn; dense and routed feed-forwards, norms on the sublayers' outputs) beside the Vogunex layers at the same sizes.
 The default workload and its line are not touched by any of them.
 
 Peaks come from MEASURED_PEAKS.json beside this file if present, else 6.65 TB/s and 1.59 PFLOP/s.
