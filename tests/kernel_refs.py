@@ -103,14 +103,15 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
     out.copy_(res.view(T, H * d).to(out.dtype))
 
 
-def swiglu(gate_up, out, interleaved=False):
+def swiglu(gate_up, out, interleaved=False, activation="silu"):
     T, I = out.shape
     if interleaved:
         blocks = gate_up.float().view(T, I // 16, 2, 16)
         g, u = blocks[:, :, 0, :].reshape(T, I), blocks[:, :, 1, :].reshape(T, I)
     else:
         g, u = gate_up[:, :I].float(), gate_up[:, I:].float()
-    out.copy_((g / (1.0 + torch.exp(-g)) * u).to(out.dtype))
+    act = torch.clamp(g, min=0.0) if activation == "relu" else g / (1.0 + torch.exp(-g))
+    out.copy_((act * u).to(out.dtype))
 
 
 def interleave_gate_up(gate, up):
@@ -122,9 +123,9 @@ def can_fuse_swiglu(dtype, hidden, intermediate):
     return dtype == torch.bfloat16 and intermediate % 16 == 0 and hidden % 8 == 0
 
 
-def gemm_swiglu(x, w_interleaved, out, workspace=None):
+def gemm_swiglu(x, w_interleaved, out, workspace=None, activation="silu"):
     y = x.float() @ w_interleaved.float().t()
-    swiglu(y, out, interleaved=True)
+    swiglu(y, out, True, activation)
 
 
 def gather_rows(src, rows, out):
