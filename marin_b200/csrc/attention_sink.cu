@@ -9,17 +9,64 @@
 //   * values that are the leading `dv` elements of the key rows (a latent shared by keys and values): the value pointer is
 //     the key pointer and `v_stride`, the distance between two positions' values, is the key rows' width;
 //   * an output gate: the result is multiplied element by element with sigmoid(g), g a column block of the fused
-//     projection; and a plain factor `out_scale`.
-// This file holds the head preparation (biases, RMS norm of q and k per head or over the whole projection, partial
-// rotation with scaled sines and cosines, value mixing with the values an earlier layer left for the same tokens, cache
-// write) and the plain attention kernel that serves any size in both dtypes.  Sums, norms, angles, scores and weights
-// are float32.
+//     projection; and a plain factor `out_scale`;
+//   * several maps per head over the same values (differential attention: Ye, Dong, Xia, Sun, Zhu, Huang, Wei, "Differential
+//     Transformer"): the keys of a kv head's maps lie side by side in one key row, a map's query is zero outside its own part of that
+//     row, so that to the attention kernels the maps are query heads like any others that share a kv head; their results are
+//     combined, o = a_1 - lambda a_2, o / rms(o) * factor (pair_combine_kernel, or the ends of the tensor-core kernels).
+// This file holds the head preparation (biases, a short causal convolution per channel over the projection's rows, RMS norm of q
+// and k per head or over the whole projection, partial rotation with scaled sines and cosines, value mixing with the values an
+// earlier layer left for the same tokens, cache write) and the plain attention kernel that serves any size in both dtypes.  Sums,
+// norms, angles, scores and weights are float32.
 #define MB_LIB "attention_sink"
 #define MB_LIB_ID 13
 #include "common.cuh"
 #include "launch.cuh"
 
 #define QF_THREADS 256            // at least; 1024 where a token's q and k have 4,096 elements and more
+
+// A causal convolution over the rows of the projection, one per channel (q, k and v columns), before norm and rotation: with
+// u = projection + bias, y_t = sum_j w[j] u_(t - taps + 1 + j), zeros before the sequence's start.  A request keeps its latest u as a
+// ring of `taps` rows (float32 [slot][taps][channels], position p in row p mod taps).  The step's tokens below `singles` are the only ones
+// of their requests: they replace their ring row here (nobody in the step reads it); the rows of longer portions are kept by
+// conv_ring_kernel behind this one.
+struct ConvRows {
+    const float* w;               // [taps][channels], the last row on the current token; nullptr: no convolution
+    float* ring;
+    const int* slots;
+    const int* req_index;
+    const int* cu_tokens;
+    int taps, channels, singles;
+};
+
+// Channel c of token t (its projection's row `row`, position pos): bias and convolution.  first: the request's first token of the step.
+template <typename T>
+__device__ __forceinline__ float conv_channel(const ConvRows& cv, const T* row, int row_stride, int t, int c, float bias, int first, int pos, float* kept) {
+    const float now = to_f32(row[c]) + bias;
+    if (cv.w == nullptr) return now;
+    float sum = 0.0f;
+    for (int back = min(cv.taps - 1, pos); back > 0; --back) {
+        const float u = t - back >= first ? to_f32(row[c - (ptrdiff_t)back * row_stride]) + bias : kept[(size_t)((pos - back) % cv.taps) * cv.channels + c];
+        sum = fmaf(cv.w[(size_t)(cv.taps - 1 - back) * cv.channels + c], u, sum);
+    }
+    if (t < cv.singles && cv.taps > 1) kept[(size_t)(pos % cv.taps) * cv.channels + c] = now;
+    return fmaf(cv.w[(size_t)(cv.taps - 1) * cv.channels + c], now, sum);
+}
+
+// The rings after the step, requests first_req .. : what their last taps - 1 tokens (or as many as they brought) left in front of the convolution.
+template <typename T>
+__global__ void conv_ring_kernel(const T* __restrict__ row, int row_stride, const float* __restrict__ q_b, const float* __restrict__ k_b,
+                                 const float* __restrict__ v_b, ConvRows cv, const int* __restrict__ positions, int first_req, int q_cols, int k_cols) {
+    PDL_ENTER();
+    row = pdl_fresh(row);
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, req = first_req + blockIdx.y;
+    if (c >= cv.channels) return;
+    const float* b = c < q_cols ? q_b : c < q_cols + k_cols ? k_b : v_b;
+    const float bias = b != nullptr ? b[c < q_cols ? c : c < q_cols + k_cols ? c - q_cols : c - q_cols - k_cols] : 0.0f;
+    const int end = cv.cu_tokens[req + 1], first = max(cv.cu_tokens[req], end - (cv.taps - 1));
+    float* kept = cv.ring + (size_t)cv.slots[req] * cv.taps * cv.channels;
+    for (int t = first; t < end; ++t) kept[(size_t)(positions[t] % cv.taps) * cv.channels + c] = to_f32(row[(size_t)t * row_stride + c]) + bias;
+}
 
 // ---- heads of the fused q|k|v(|g) projection, a token per block ---------------------------------------------------------
 // A row of `row` holds q (H heads of d), k (K heads of d), v (K heads of dv), then whatever follows (the gate's columns).
@@ -29,15 +76,17 @@
 // rot_mag.
 // v_mode 0: values as they are; 1: they are also left in v_shared (activation dtype [tokens][K dv]) for later layers;
 // 2: v <- (1 - lam) v + lam v_shared, lam = *v_lambda, and the mixed values go to the cache.
+// maps > 1: H and K count maps (heads times maps, a head's maps side by side), there are K / maps value heads; key map m of a kv
+// head goes to elements m d .. of its row of maps * d, a query map likewise, with zeros around it.
 template <typename T>
 __global__ void __launch_bounds__(1024) qkv_finish_kernel(
     const T* __restrict__ row, int row_stride, T* __restrict__ q_out, const float* __restrict__ q_b, const float* __restrict__ k_b,
     const float* __restrict__ v_b, int norm_mode, const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
     const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dim, float rot_mag,
     const int* __restrict__ slot_mapping, T* __restrict__ k_cache, T* __restrict__ v_cache, int v_mode, T* __restrict__ v_shared,
-    const float* __restrict__ v_lambda, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved) {
+    const float* __restrict__ v_lambda, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved, int maps, ConvRows cv) {
     PDL_ENTER();
-    row = pdl_fresh(row); v_shared = pdl_fresh(v_shared);
+    row = pdl_fresh(row); v_shared = pdl_fresh(v_shared); cv.ring = pdl_fresh(cv.ring);
     extern __shared__ float smem[];
     const int heads = write_kv ? H + K : H;
     const int half = rot_dim >> 1;
@@ -57,13 +106,21 @@ __global__ void __launch_bounds__(1024) qkv_finish_kernel(
             cs_tab[half + i] = sn * rot_mag;
         }
     }
-    // every element of q and k (+ bias) into shared memory as float32, all threads side by side
+    int first = 0, pos = 0;
+    float* kept = nullptr;
+    if (cv.w != nullptr) {
+        const int req = cv.req_index[t];
+        first = cv.cu_tokens[req];
+        pos = positions[t];
+        kept = cv.ring + (size_t)cv.slots[req] * cv.taps * cv.channels;
+    }
+    // every element of q and k (+ bias, through the convolution) into shared memory as float32, all threads side by side
     const int qk = heads * d, q_len = H * d;
     for (int idx = threadIdx.x; idx < qk; idx += threads) {
-        float v = to_f32(src[idx]);
-        if (idx < q_len) { if (q_b != nullptr) v += q_b[idx]; }
-        else if (k_b != nullptr) v += k_b[idx - q_len];
-        vals[idx] = v;
+        float bias = 0.0f;
+        if (idx < q_len) { if (q_b != nullptr) bias = q_b[idx]; }
+        else if (k_b != nullptr) bias = k_b[idx - q_len];
+        vals[idx] = conv_channel(cv, src, row_stride, t, idx, bias, first, pos, kept);
     }
     __syncthreads();
     // sums of squares per head: a warp per head, lanes in a fixed order
@@ -82,7 +139,8 @@ __global__ void __launch_bounds__(1024) qkv_finish_kernel(
     }
     __syncthreads();
     const int slot = write_kv ? slot_mapping[t] : -1;
-    T* k_dst = slot >= 0 ? k_cache + (((size_t)(slot / page_size)) * K * page_size + (size_t)(slot % page_size)) * d : nullptr;
+    const int KG = K / maps, wide = d * maps;                  // kv heads, and the width of a key row
+    T* k_dst = slot >= 0 ? k_cache + (((size_t)(slot / page_size)) * KG * page_size + (size_t)(slot % page_size)) * wide : nullptr;
     // a warp per head, lanes along the head: no division per element, 64-byte runs per store
     for (int head = warp; head < heads; head += warps) {
         const bool is_q = head < H;
@@ -98,7 +156,12 @@ __global__ void __launch_bounds__(1024) qkv_finish_kernel(
             w = is_q ? q_w + (size_t)head * d : k_w + (size_t)kh * d;
         }
         const float* hv = vals + (size_t)head * d;
-        T* dst = is_q ? q_out + (size_t)t * q_len + (size_t)head * d : k_dst + (size_t)kh * page_size * d;
+        T* dst = is_q ? q_out + ((size_t)t * H + head) * wide + (head % maps) * d : k_dst + (size_t)(kh / maps) * page_size * wide + (kh % maps) * d;
+        if (is_q && maps > 1) {
+            T* whole = dst - (head % maps) * d;
+            for (int i = lane; i < wide; i += 32)
+                if (i / d != head % maps) whole[i] = from_f32<T>(0.0f);
+        }
         for (int i = lane; i < d; i += 32) {
             float a = hv[i] * factor * (w != nullptr ? w[i] : 1.0f);
             if (i < rot_dim) {                                 // (rot_dim is 0 without a rotation)
@@ -115,14 +178,13 @@ __global__ void __launch_bounds__(1024) qkv_finish_kernel(
     if (!write_kv) return;
     const float lam = v_mode == 2 ? *v_lambda : 0.0f;
     const int vcol0 = (H + K) * d;
-    for (int kh = warp; kh < K; kh += warps) {
-        T* dst = slot >= 0 ? v_cache + ((((size_t)(slot / page_size)) * K + kh) * page_size + (size_t)(slot % page_size)) * dv : nullptr;
+    for (int kh = warp; kh < KG; kh += warps) {
+        T* dst = slot >= 0 ? v_cache + ((((size_t)(slot / page_size)) * KG + kh) * page_size + (size_t)(slot % page_size)) * dv : nullptr;
         for (int e = lane; e < dv; e += 32) {
             const int i = kh * dv + e;
-            float v = to_f32(src[vcol0 + i]);
-            if (v_b != nullptr) v += v_b[i];
-            if (v_mode == 1) v_shared[(size_t)t * K * dv + i] = from_f32<T>(v);
-            else if (v_mode == 2) v = (1.0f - lam) * v + lam * to_f32(v_shared[(size_t)t * K * dv + i]);
+            float v = conv_channel(cv, src, row_stride, t, vcol0 + i, v_b != nullptr ? v_b[i] : 0.0f, first, pos, kept);
+            if (v_mode == 1) v_shared[(size_t)t * KG * dv + i] = from_f32<T>(v);
+            else if (v_mode == 2) v = (1.0f - lam) * v + lam * to_f32(v_shared[(size_t)t * KG * dv + i]);
             if (dst != nullptr) dst[e] = from_f32<T>(v);
         }
     }
@@ -151,15 +213,54 @@ __device__ __forceinline__ void load8(const float* p, float* x) {
     x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
 }
 
+// conv_channel for eight neighbouring channels from c on; x comes in as projection + bias of the current token.
+__device__ __forceinline__ void conv_run8(const ConvRows& cv, const bf16* row, int row_stride, int t, int c, const float* bias, int first, int pos, float* kept,
+                                          float* x) {
+    if (cv.w == nullptr) return;
+    float sum[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sum[e] = 0.0f;
+    auto add = [&](int back) {
+        float u[8], w[8];
+        if (t - back >= first) {
+            unpack8(*reinterpret_cast<const uint4*>(row + c - (ptrdiff_t)back * row_stride), u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) u[e] += bias[e];
+        } else {
+            load8(kept + (size_t)((pos - back) % cv.taps) * cv.channels + c, u);
+        }
+        load8(cv.w + (size_t)(cv.taps - 1 - back) * cv.channels + c, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sum[e] = fmaf(w[e], u[e], sum[e]);
+    };
+    const int most = min(cv.taps - 1, pos);
+    if (cv.taps <= 4) {                        // (unrolled: the loads of all rows in flight at once)
+#pragma unroll
+        for (int back = 3; back > 0; --back)
+            if (back <= most) add(back);
+    } else {
+        for (int back = most; back > 0; --back) add(back);
+    }
+    if (t < cv.singles && cv.taps > 1) {
+        float* dst = kept + (size_t)(pos % cv.taps) * cv.channels + c;
+        *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]);
+        *reinterpret_cast<float4*>(dst + 4) = make_float4(x[4], x[5], x[6], x[7]);
+    }
+    float w[8];
+    load8(cv.w + (size_t)(cv.taps - 1) * cv.channels + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = fmaf(w[e], x[e], sum[e]);
+}
+
 template <int RUNS>
 __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
     const bf16* __restrict__ row, int row_stride, bf16* __restrict__ q_out, const float* __restrict__ q_b, const float* __restrict__ k_b,
     const float* __restrict__ v_b, int norm_mode, const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
     const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dim, float rot_mag,
     const int* __restrict__ slot_mapping, bf16* __restrict__ k_cache, bf16* __restrict__ v_cache, int v_mode, bf16* __restrict__ v_shared,
-    const float* __restrict__ v_lambda, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved) {
+    const float* __restrict__ v_lambda, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved, int maps, ConvRows cv) {
     PDL_ENTER();
-    row = pdl_fresh(row); v_shared = pdl_fresh(v_shared);
+    row = pdl_fresh(row); v_shared = pdl_fresh(v_shared); cv.ring = pdl_fresh(cv.ring);
     extern __shared__ __align__(16) float smem[];
     __shared__ float scratch[32];
     const int heads = write_kv ? H + K : H;
@@ -179,6 +280,14 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
             cs_tab[half + i] = sn * rot_mag;
         }
     }
+    int first = 0, pos = 0;
+    float* kept = nullptr;
+    if (cv.w != nullptr) {
+        const int req = cv.req_index[t];
+        first = cv.cu_tokens[req];
+        pos = positions[t];
+        kept = cv.ring + (size_t)cv.slots[req] * cv.taps * cv.channels;
+    }
     const int runs = heads * d / 8, q_runs = H * d / 8;
     float x[RUNS][8];
     float ss_q = 0.0f, ss_k = 0.0f;
@@ -188,12 +297,13 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
         if (v < runs) {
             unpack8(*reinterpret_cast<const uint4*>(src + v * 8), x[u]);
             const float* bias = v < q_runs ? q_b : k_b;
+            float b[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
             if (bias != nullptr) {
-                float b[8];
                 load8(bias + (v < q_runs ? v : v - q_runs) * 8, b);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) x[u][e] += b[e];
             }
+            conv_run8(cv, src, row_stride, t, v * 8, b, first, pos, kept, x[u]);
             float ss = 0.0f;
 #pragma unroll
             for (int e = 0; e < 8; ++e) ss += x[u][e] * x[u][e];
@@ -222,7 +332,8 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
         }
     }
     const int slot = write_kv ? slot_mapping[t] : -1;
-    bf16* k_dst = slot >= 0 ? k_cache + (((size_t)(slot / page_size)) * K * page_size + (size_t)(slot % page_size)) * d : nullptr;
+    const int KG = K / maps, wide = d * maps;                  // kv heads, and the width of a key row
+    bf16* k_dst = slot >= 0 ? k_cache + (((size_t)(slot / page_size)) * KG * page_size + (size_t)(slot % page_size)) * wide : nullptr;
 #pragma unroll
     for (int u = 0; u < RUNS; ++u) {
         const int v = threadIdx.x + u * threads;
@@ -278,22 +389,31 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
 #pragma unroll
             for (int e = 0; e < 8; ++e) a[e] = low ? a[e] * cs[e] - b[e] * sn[e] : a[e] * cs[e] + b[e] * sn[e];
         }
-        bf16* dst = is_q ? q_out + (size_t)t * H * d + (size_t)v * 8 : k_dst + (size_t)kh * page_size * d + i0;
-        *reinterpret_cast<uint4*>(dst) = pack8(a);
+        if (maps == 1) {
+            bf16* dst = is_q ? q_out + (size_t)t * H * d + (size_t)v * 8 : k_dst + (size_t)kh * page_size * d + i0;
+            *reinterpret_cast<uint4*>(dst) = pack8(a);
+        } else if (is_q) {
+            const int m = head % maps;
+            bf16* dst = q_out + ((size_t)t * H + head) * wide + i0;
+            for (int o = 0; o < maps; ++o) *reinterpret_cast<uint4*>(dst + o * d) = o == m ? pack8(a) : make_uint4(0, 0, 0, 0);
+        } else {
+            *reinterpret_cast<uint4*>(k_dst + (size_t)(kh / maps) * page_size * wide + (kh % maps) * d + i0) = pack8(a);
+        }
     }
     if (!write_kv) return;
     const float lam = v_mode == 2 ? *v_lambda : 0.0f;
     const int vcol0 = (H + K) * d;
-    for (int v = threadIdx.x; v < K * dv / 8; v += threads) {
+    for (int v = threadIdx.x; v < KG * dv / 8; v += threads) {
         float val[8];
         unpack8(*reinterpret_cast<const uint4*>(src + vcol0 + v * 8), val);
+        float b[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
         if (v_b != nullptr) {
-            float b[8];
             load8(v_b + v * 8, b);
 #pragma unroll
             for (int e = 0; e < 8; ++e) val[e] += b[e];
         }
-        bf16* shared_at = v_shared + (size_t)t * K * dv + v * 8;
+        conv_run8(cv, src, row_stride, t, vcol0 + v * 8, b, first, pos, kept, val);
+        bf16* shared_at = v_shared + (size_t)t * KG * dv + v * 8;
         if (v_mode == 1) {
             *reinterpret_cast<uint4*>(shared_at) = pack8(val);
         } else if (v_mode == 2) {
@@ -304,7 +424,7 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
         }
         if (slot >= 0) {
             const int kh = (v * 8) / dv, e0 = v * 8 - kh * dv;
-            *reinterpret_cast<uint4*>(v_cache + ((((size_t)(slot / page_size)) * K + kh) * page_size + (size_t)(slot % page_size)) * dv + e0) = pack8(val);
+            *reinterpret_cast<uint4*>(v_cache + ((((size_t)(slot / page_size)) * KG + kh) * page_size + (size_t)(slot % page_size)) * dv + e0) = pack8(val);
         }
     }
 }
@@ -315,8 +435,12 @@ MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out
                          int norm_mode, const float* q_w, const float* k_w, float eps, const int* positions, const float* inv_freq,
                          int rot_dim, float rot_mag, const int* slot_mapping, void* k_cache, void* v_cache, int v_mode, void* v_shared,
                          const float* v_lambda, int tokens, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved,
+                         int maps, const float* conv_w, float* ring, const int* slots, const int* req_index, const int* cu_tokens, int taps, int singles,
                          cudaStream_t s) {
     if (tokens <= 0) return 0;
+    if (maps < 1 || H % maps != 0 || K % maps != 0) return MB_ERR_BAD_SIZE;
+    if (conv_w != nullptr && (taps < 1 || taps > 64 || !write_kv)) return MB_ERR_BAD_SIZE;
+    const ConvRows cv = {conv_w, ring, slots, req_index, cu_tokens, taps, (H + K) * d + K / maps * dv, singles};
     if (d <= 0 || dv <= 0 || H <= 0 || K <= 0 || rot_dim > d || (rot_dim & 1) || norm_mode < 0 || norm_mode > 2) return MB_ERR_BAD_SIZE;
     if ((v_mode == 1 || v_mode == 2) && v_shared == nullptr) return MB_ERR_BAD_SIZE;
     if (v_mode == 2 && v_lambda == nullptr) return MB_ERR_BAD_SIZE;
@@ -326,7 +450,7 @@ MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out
     const int runs8 = (H + K) * d / 8;
     if (dtype == MB_BF16 && d % 8 == 0 && dv % 8 == 0 && (interleaved ? rot_dim % 8 == 0 : (rot_dim / 2) % 8 == 0) && row_stride % 8 == 0 && runs8 <= 1024 * 2 &&
         aligned16(row) && aligned16(q_out) && aligned16(q_b) && aligned16(k_b) && aligned16(v_b) && aligned16(q_w) && aligned16(k_w) &&
-        aligned16(k_cache) && aligned16(v_cache) && aligned16(v_shared)) {
+        aligned16(k_cache) && aligned16(v_cache) && aligned16(v_shared) && aligned16(conv_w) && aligned16(ring)) {
 #define QV_LAUNCH(RUNS, threads)                                                                                                        \
     do {                                                                                                                                \
         if (smem > 48 * 1024) {                                                                                                         \
@@ -335,7 +459,7 @@ MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out
         }                                                                                                                               \
         return launch_kernel(qkv_finish_vec_kernel<RUNS>, tokens, threads, smem, s, 0, (const bf16*)row, row_stride, (bf16*)q_out, q_b, k_b, \
                              v_b, norm_mode, q_w, k_w, eps, positions, inv_freq, rot_dim, rot_mag, slot_mapping, (bf16*)k_cache,         \
-                             (bf16*)v_cache, v_mode, (bf16*)v_shared, v_lambda, H, K, d, dv, page_size, write_kv, interleaved);          \
+                             (bf16*)v_cache, v_mode, (bf16*)v_shared, v_lambda, H, K, d, dv, page_size, write_kv, interleaved, maps, cv);          \
     } while (0)
         const int quarter = (((runs8 + 3) / 4 + 31) / 32) * 32;
         if (tokens >= 512 && quarter <= 256) QV_LAUNCH(4, quarter < 64 ? 64 : quarter);
@@ -352,11 +476,54 @@ MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out
         }                                                                                                                            \
         return launch_kernel(qkv_finish_kernel<TT>, tokens, (H + K) * d < 4096 ? QF_THREADS : tokens <= 64 ? 1024 : 512, smem, s, 0, (const TT*)row, row_stride, (TT*)q_out, q_b, k_b, \
                              v_b, norm_mode, q_w, k_w, eps, positions, inv_freq, rot_dim, rot_mag, slot_mapping, (TT*)k_cache,      \
-                             (TT*)v_cache, v_mode, (TT*)v_shared, v_lambda, H, K, d, dv, page_size, write_kv, interleaved);          \
+                             (TT*)v_cache, v_mode, (TT*)v_shared, v_lambda, H, K, d, dv, page_size, write_kv, interleaved, maps, cv);          \
     } while (0)
     if (dtype == MB_F32) QF_LAUNCH(float);
     if (dtype == MB_BF16) QF_LAUNCH(bf16);
 #undef QF_LAUNCH
+    return MB_ERR_BAD_DTYPE;
+}
+
+MB_API int mb_conv_ring(const void* row, int row_stride, int dtype, const float* q_b, const float* k_b, const float* v_b, float* ring, const int* slots,
+                        const int* cu_tokens, const int* positions, int taps, int first_req, int requests, int q_cols, int k_cols, int v_cols, cudaStream_t s) {
+    if (requests <= first_req || taps <= 1) return 0;
+    if (taps > 64 || first_req < 0) return MB_ERR_BAD_SIZE;
+    const int channels = q_cols + k_cols + v_cols;
+    const ConvRows cv = {nullptr, ring, slots, nullptr, cu_tokens, taps, channels, 0};
+    dim3 grid((channels + 127) / 128, requests - first_req);
+    if (dtype == MB_F32)
+        return launch_kernel(conv_ring_kernel<float>, grid, 128, 0, s, 0, (const float*)row, row_stride, q_b, k_b, v_b, cv, positions, first_req, q_cols, k_cols);
+    if (dtype == MB_BF16)
+        return launch_kernel(conv_ring_kernel<bf16>, grid, 128, 0, s, 0, (const bf16*)row, row_stride, q_b, k_b, v_b, cv, positions, first_req, q_cols, k_cols);
+    return MB_ERR_BAD_DTYPE;
+}
+
+// ---- two maps of a head combined: out = n / rms(n) * factor, n = a_1 - lam a_2, a warp per (token, head) -----------------
+// a: float32 [tokens][2 H][dv], a head's maps side by side.
+template <typename T>
+__global__ void pair_combine_kernel(const float* __restrict__ a, T* __restrict__ out, int out_stride, float lam, float eps, float factor, int first_token,
+                                    int pairs, int H, int dv) {
+    PDL_ENTER();
+    a = pdl_fresh(a);
+    const int p = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (p >= pairs) return;
+    const int t = first_token + p / H, head = p % H;
+    const float* a1 = a + ((size_t)t * H + head) * 2 * dv;
+    const float* a2 = a1 + dv;
+    float ss = 0.0f;
+    for (int i = lane; i < dv; i += 32) { const float v = a1[i] - lam * a2[i]; ss = fmaf(v, v, ss); }
+    const float f = factor / sqrtf(warp_sum(ss) / (float)dv + eps);
+    T* dst = out + (size_t)t * out_stride + (size_t)head * dv;
+    for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>((a1[i] - lam * a2[i]) * f);
+}
+
+MB_API int mb_pair_combine(const float* a, void* out, int out_stride, int dtype, float lam, float eps, float factor, int first_token, int tokens, int H, int dv,
+                           cudaStream_t s) {
+    if (tokens <= first_token) return 0;
+    if (H <= 0 || dv <= 0 || first_token < 0 || out_stride < H * dv) return MB_ERR_BAD_SIZE;
+    const int pairs = (tokens - first_token) * H, blocks = (pairs + 7) / 8;
+    if (dtype == MB_F32) return launch_kernel(pair_combine_kernel<float>, blocks, 256, 0, s, 0, a, (float*)out, out_stride, lam, eps, factor, first_token, pairs, H, dv);
+    if (dtype == MB_BF16) return launch_kernel(pair_combine_kernel<bf16>, blocks, 256, 0, s, 0, a, (bf16*)out, out_stride, lam, eps, factor, first_token, pairs, H, dv);
     return MB_ERR_BAD_DTYPE;
 }
 
@@ -369,7 +536,7 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
     const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
     const int* __restrict__ block_table, int max_pages, const int* __restrict__ req_index, const int* __restrict__ positions,
     int H, int K, int d, int dv, int page_size, float scale, int window, int chunk, int sink, const float* __restrict__ sink_logit,
-    int v_stride, const T* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride) {
+    int v_stride, const T* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride, float* __restrict__ wide_out) {
     PDL_ENTER();
     q = pdl_fresh(q); k_cache = pdl_fresh(k_cache); v_cache = pdl_fresh(v_cache); gate = pdl_fresh(gate);
     extern __shared__ float smem[];
@@ -442,7 +609,8 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
         if (dd < dv) {
             float o = acc[r] / l * out_scale;
             if (grow != nullptr) o *= 1.0f / (1.0f + expf(-to_f32(grow[dd])));
-            orow[dd] = from_f32<T>(o);
+            if (wide_out != nullptr) wide_out[((size_t)t * H + head) * dv + dd] = o;
+            else orow[dd] = from_f32<T>(o);
         }
     }
 }
@@ -451,12 +619,13 @@ __global__ void __launch_bounds__(SK_THREADS) attention_sink_kernel(
 // sink_logit: null (a sink of score 0, if `sink`) or a float32 score per query head.  v_stride: elements between the values of
 // two positions of a page (dv for value pages of their own; the key rows' width where values are the start of the key rows).
 // keep: first positions that are always seen; softcap 0: scores are not capped; out rows are out_stride elements apart.
+// wide_out: null, or float32 [tokens][H][dv] that takes the result instead of `out`.
 MB_API int mb_attention_sink(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype, const int* block_table,
                              int max_pages, const int* req_index, const int* positions, int tokens, int H, int K, int d, int dv,
                              int page_size, float scale, int window, int chunk, int sink, const float* sink_logit, int v_stride,
-                             const void* gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
+                             const void* gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride, float* wide_out, cudaStream_t s) {
     if (tokens <= 0) return 0;
-    if (v_stride < dv || keep < 0 || softcap < 0.0f || out_stride < H * dv) return MB_ERR_BAD_SIZE;
+    if (v_stride < dv || keep < 0 || softcap < 0.0f || (wide_out == nullptr && out_stride < H * dv)) return MB_ERR_BAD_SIZE;
     if (d <= 0 || dv <= 0 || dv > SK_THREADS * SK_MAX_PER_THREAD || K <= 0 || H % K != 0 || window < 0 || chunk < 0) return MB_ERR_BAD_SIZE;
     dim3 grid(tokens, H);
     const size_t smem = (size_t)(d + SK_THREADS + 32) * sizeof(float);
@@ -464,10 +633,10 @@ MB_API int mb_attention_sink(const void* q, const void* k_cache, const void* v_c
     if (dtype == MB_F32)
         return launch_kernel(attention_sink_kernel<float>, grid, SK_THREADS, smem, s, 0, (const float*)q, (const float*)k_cache,
                              (const float*)v_cache, (float*)out, block_table, max_pages, req_index, positions, H, K, d, dv, page_size,
-                             scale, window, chunk, sink, sink_logit, v_stride, (const float*)gate, gate_stride, keep, softcap, out_scale, out_stride);
+                             scale, window, chunk, sink, sink_logit, v_stride, (const float*)gate, gate_stride, keep, softcap, out_scale, out_stride, wide_out);
     if (dtype == MB_BF16)
         return launch_kernel(attention_sink_kernel<bf16>, grid, SK_THREADS, smem, s, 0, (const bf16*)q, (const bf16*)k_cache,
                              (const bf16*)v_cache, (bf16*)out, block_table, max_pages, req_index, positions, H, K, d, dv, page_size,
-                             scale, window, chunk, sink, sink_logit, v_stride, (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
+                             scale, window, chunk, sink, sink_logit, v_stride, (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride, wide_out);
     return MB_ERR_BAD_DTYPE;
 }

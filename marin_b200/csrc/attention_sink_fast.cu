@@ -1,6 +1,7 @@
 // bf16 softmax attention with a sink, a chunked mask or a window, value heads of their own width and an output gate, on the
 // tensor cores (mma.sync), compiled for one head layout:
-//   -DHEAD_DIM (keys and queries), -DV_DIM (values), -DGROUP (query heads per kv head); both sizes multiples of 16 up to 128.
+//   -DHEAD_DIM (keys and queries; a multiple of 16 up to 256), -DV_DIM (values; a multiple of 16 up to 128), -DGROUP (query heads per kv
+//   head).
 // A position i sees the keys j <= i with j >= lo(i) = max(i - window + 1 (window > 0), floor(i / chunk) chunk (chunk > 0), 0) and the
 // sequence's first `keep` positions.  Scores may be capped, s <- cap tanh(s / cap); the sink's score is not.  The result is multiplied
 // by `out_scale`; output rows are `out_stride` elements apart.
@@ -13,6 +14,8 @@
 // Single tokens: the visible keys of a sequence split over CTAs, partial (max, sum, accumulator) merged by a second kernel
 // in chunk order, which also adds the sink and applies the gate.
 // K pages [page][kv_head][offset][HEAD_DIM], V pages [page][kv_head][offset][V_DIM].
+// Two maps per head over the same values (attention_sink.cu): query heads 2 h and 2 h + 1 are head h's maps; prompt portions leave
+// both results in float32 (wide_out), single tokens' parts are merged and combined in one kernel.
 // -DV_IN_K: there are no value pages; a position's values are the first V_DIM elements of its key row (a latent that keys and
 // values share), so a key block in shared memory serves both products and nothing is fetched twice.  The pages then hold one
 // kv head that every query head reads: the launchers' `K` only counts groups of GROUP query heads (a CTA's rows), so any
@@ -123,7 +126,7 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
     const bf16* __restrict__ q, const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache, bf16* __restrict__ out,
     const int* __restrict__ block_table, int max_pages, const int* __restrict__ cu_tokens, const int* __restrict__ seq_lens,
     int first_req, int K, int page_shift, float scale, int window, int chunk, int sink, const float* __restrict__ sink_logit,
-    const bf16* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride) {
+    const bf16* __restrict__ gate, int gate_stride, int keep, float softcap, float out_scale, int out_stride, float* __restrict__ wide_out) {
     PDL_ENTER_EARLY();
     q = pdl_fresh(q); k_cache = pdl_fresh(k_cache); v_cache = pdl_fresh(v_cache); gate = pdl_fresh(gate);
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -274,7 +277,8 @@ __global__ void __launch_bounds__(128, 2) attn_sink_prefill_kernel(
                     a *= sigmoid_of(gg.x);
                     b *= sigmoid_of(gg.y);
                 }
-                *reinterpret_cast<uint32_t*>(dst + i * 8 + col) = pack_bf16(a, b);
+                if (wide_out != nullptr) *reinterpret_cast<float2*>(wide_out + (t * H + h) * DV + i * 8 + col) = make_float2(a, b);
+                else *reinterpret_cast<uint32_t*>(dst + i * 8 + col) = pack_bf16(a, b);
             }
         }
     }
@@ -536,6 +540,60 @@ __global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_kernel(
     }
 }
 
+// The same for heads of two maps (query heads 2 h and 2 h + 1; no sink, no gate), a block per (request, head): both maps' parts are
+// merged, n = a_1 - lam a_2, out = n / rms(n) * factor with the mean over the head's V_DIM numbers and eps under the root.
+static_assert(V_DIM <= MG_THREADS, "one output per thread");
+__global__ void __launch_bounds__(MG_THREADS) attn_sink_merge_pair_kernel(
+    const float* __restrict__ part_acc, const float* __restrict__ part_ml, const int* __restrict__ seq_lens, int split, int window, int chunk_size,
+    int R, int H, float lam, float eps, float factor, bf16* __restrict__ out, int keep, int out_stride) {
+    PDL_ENTER();
+    part_acc = pdl_fresh(part_acc); part_ml = pdl_fresh(part_ml);
+    __shared__ float wgt[2][MG_MAX_CHUNKS], scratch[32];
+    const int pairs = H >> 1, r = blockIdx.x / pairs, p = blockIdx.x % pairs;
+    const int len = seq_lens[r];
+    if (len <= 0) return;
+    const int pos = len - 1;
+    const int first_block = first_seen(pos, window, chunk_size) / BN;
+    const int behind = (first_block - kept_blocks(keep, first_block)) * BN;
+    const int chunks = min((len - behind + split - 1) / split, MG_MAX_CHUNKS);
+    float n = 0.0f;                                            // this thread's number of the combined head
+    for (int m = 0; m < 2; ++m) {
+        const int h = 2 * p + m;
+        float mx = -INFINITY;
+        for (int c = threadIdx.x; c < chunks; c += MG_THREADS) {
+            const float mc = part_ml[(((size_t)c * R + r) * H + h) * 2];
+            wgt[m][c] = mc;
+            mx = fmaxf(mx, mc);
+        }
+        const float M = block_max(mx, scratch);
+        float part = 0.0f;
+        for (int c = threadIdx.x; c < chunks; c += MG_THREADS) {
+            const float mc = wgt[m][c];
+            const float f = mc == -INFINITY ? 0.0f : exp2f(mc - M);
+            wgt[m][c] = f;
+            part = fmaf(part_ml[(((size_t)c * R + r) * H + h) * 2 + 1], f, part);
+        }
+        const float inv = 1.0f / block_sum(part, scratch);     // (its barriers publish wgt)
+        if (threadIdx.x < DV) {
+            float a = 0.0f;
+            int c = 0;
+            for (; c + 8 <= chunks; c += 8) {                  // eight loads in flight, added in chunk order
+                float x[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) x[u] = part_acc[(((size_t)(c + u) * R + r) * H + h) * DV + threadIdx.x];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) a = fmaf(x[u], wgt[m][c + u], a);
+            }
+            for (; c < chunks; ++c) a = fmaf(part_acc[(((size_t)c * R + r) * H + h) * DV + threadIdx.x], wgt[m][c], a);
+            a *= inv;
+            n = m == 0 ? a : n - lam * a;
+        }
+    }
+    const float ss = block_sum(threadIdx.x < DV ? n * n : 0.0f, scratch);
+    if (threadIdx.x < DV)
+        out[(size_t)r * out_stride + (size_t)p * DV + threadIdx.x] = __float2bfloat16_rn(n / sqrtf(ss / (float)DV + eps) * factor);
+}
+
 static int page_shift_of(int page_size) {
     int s = 0;
     while ((1 << s) < page_size) ++s;
@@ -569,17 +627,27 @@ MB_API int mb_attn_sink_merge(const float* part_acc, const float* part_ml, void*
                          (bf16*)out, keep, out_scale, out_stride);
 }
 
-// Prompt portions: requests first_req .. first_req + count - 1 of the step.
+// Heads of two maps: parts of K * GROUP query heads, out bf16 rows of K * GROUP / 2 heads.
+MB_API int mb_attn_sink_merge_pair(const float* part_acc, const float* part_ml, void* out, const int* seq_lens, int requests, int K, int window, int chunk,
+                                   int split, int keep, float lam, float eps, float factor, int out_stride, cudaStream_t s) {
+    if (requests <= 0) return 0;
+    if (split <= 0 || keep < 0 || (K * GROUP) % 2 != 0 || out_stride < K * GROUP / 2 * DV) return MB_ERR_BAD_SIZE;
+    return launch_kernel(attn_sink_merge_pair_kernel, requests * (K * GROUP / 2), MG_THREADS, 0, s, 0, (const float*)part_acc, (const float*)part_ml, seq_lens,
+                         split, window, chunk, requests, K * GROUP, lam, eps, factor, (bf16*)out, keep, out_stride);
+}
+
+// Prompt portions: requests first_req .. first_req + count - 1 of the step.  wide_out: null, or float32 [tokens][K * GROUP][V_DIM] that
+// takes the result instead of `out`.
 MB_API int mb_attn_sink_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                 int max_pages, const int* cu_tokens, const int* seq_lens, int first_req, int count, int max_query_len,
                                 int K, int page_size, float scale, int window, int chunk, int sink, const void* gate, int gate_stride,
-                                const float* sink_logit, int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
+                                const float* sink_logit, int keep, float softcap, float out_scale, int out_stride, float* wide_out, cudaStream_t s) {
     if (count <= 0 || max_query_len <= 0) return 0;
     const int shift = page_shift_of(page_size);
-    if (shift < 0 || window < 0 || chunk < 0 || keep < 0 || out_stride < K * GROUP * DV || out_stride % 2 != 0) return MB_ERR_BAD_SIZE;
+    if (shift < 0 || window < 0 || chunk < 0 || keep < 0 || (wide_out == nullptr && (out_stride < K * GROUP * DV || out_stride % 2 != 0))) return MB_ERR_BAD_SIZE;
     cudaFuncSetAttribute(attn_sink_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
     dim3 grid((max_query_len + BM - 1) / BM, K * GROUP, count);
     return launch_kernel(attn_sink_prefill_kernel, grid, 128, PF_SMEM, s, 0, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
                          (bf16*)out, block_table, max_pages, cu_tokens, seq_lens, first_req, K, shift, scale, window, chunk, sink, sink_logit,
-                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
+                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride, wide_out);
 }

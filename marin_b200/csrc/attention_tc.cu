@@ -1,5 +1,5 @@
-// Prefill attention on the 5th-generation tensor cores (tcgen05 / TMEM), compiled per head size (-DHEAD_DIM=64|128)
-// and group size (-DGROUP).  With -DV_IN_K the values are the first V_DIM (64 or 128) elements of the key rows (a latent
+// Prefill attention on the 5th-generation tensor cores (tcgen05 / TMEM), compiled per head size (-DHEAD_DIM=64|128, -DV_DIM=64|128 for
+// the values where they differ) and group size (-DGROUP).  With -DV_IN_K the values are the first V_DIM (64 or 128) elements of the key rows (a latent
 // that keys and values share: one kv head, HEAD_DIM any multiple of 16 from 64 to 192): nothing is loaded for V, the
 // P V product reads the key tile again, and the tile is free once that product is done.  A CTA takes 128 consecutive query tokens of one request and one query head and
 // walks the keys in blocks of 64:
@@ -27,6 +27,9 @@
 // the keys, meet at a barrier every block and are slower too: 1,800 cycles.)
 // The sequence's first `keep` positions may stay visible behind a window or chunk: their blocks come before the window's in the list
 // of blocks a tile walks.  Scores may be capped, s <- cap tanh(s / cap) (an instantiation of its own: CAP); the sink's is not.
+// -DPAIR: query heads 2 h and 2 h + 1 are two maps of head h over the same keys' rows and values (attention_sink.cu).  A CTA takes 64 tokens of both:
+// rows 0 .. 63 are the first map's, rows 64 .. 127 the second's, so that every block of keys and values is fetched once for both; at
+// the end the second map's rows hand their results over in shared memory and the first's write n / rms(n) * factor, n = a_1 - lam a_2.
 // Two CTAs fit an SM: one's softmax overlaps the other's MMAs.  Needs pages of at least 16 positions.  Waits are
 // bounded and record a code in *error_flag.
 // The mma.sync kernel in attention_fast.cu is the fallback and the plain twin (the reference's counterpart:
@@ -50,8 +53,7 @@ static_assert(HEAD_DIM % 16 == 0 && HEAD_DIM >= 64 && HEAD_DIM <= 192, "key rows
 static_assert((V_DIM == 64 || V_DIM == 128) && V_DIM <= HEAD_DIM, "values are the first 64 or 128 elements of the key rows");
 #define TA_V_IN_K 1
 #else
-static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "the tcgen05 attention kernel takes heads of 64 or 128");
-static_assert(V_DIM == HEAD_DIM, "values as wide as the keys");
+static_assert((HEAD_DIM == 64 || HEAD_DIM == 128) && (V_DIM == 64 || V_DIM == 128), "the tcgen05 attention kernel takes heads of 64 or 128");
 #define TA_V_IN_K 0
 #endif
 
@@ -61,6 +63,15 @@ static_assert(V_DIM == HEAD_DIM, "values as wide as the keys");
                                        // may be partly filled: the copy zero-fills past the row's end, no MMA reads there)
 #define NHV (DV / 64)
 #define TA_BM 128
+#ifdef PAIR
+#define TA_PAIR 1
+#define TA_TOK 64                      // tokens of a tile
+static_assert(GROUP % 2 == 0 && !TA_V_IN_K, "two maps: pairs of query heads, values of their own");
+static_assert(64 * V_DIM * 4 <= 2 * 2 * 64 * (V_DIM + HEAD_DIM), "the handed-over rows fit the key and value buffers");
+#else
+#define TA_PAIR 0
+#define TA_TOK TA_BM
+#endif
 #define TA_BN 64
 #define TA_Q_BYTES (NH * TA_BM * 128)
 #define TA_K_BYTES (NH * TA_BN * 128)   // a block of keys
@@ -227,7 +238,7 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     bf16* __restrict__ out, const int* __restrict__ block_table, int max_pages, const int* __restrict__ cu_tokens,
     const int* __restrict__ seq_lens, int first_req, int K, int page_shift, float scale, int window, int* __restrict__ error_flag,
     int box_rows, int chunk, int sink, const float* __restrict__ sink_logit, const bf16* __restrict__ gate, int gate_stride, int keep,
-    float softcap, float out_scale, int out_stride) {
+    float softcap, float out_scale, int out_stride, float lam, float eps) {
     extern __shared__ __align__(1024) uint8_t smem[];     // the swizzled tiles need 1024-byte alignment (checked below)
     uint8_t* sQ = smem;
     uint8_t* sKV = sQ + TA_Q_BYTES;                       // [buffer][K then V][half][64 rows][128 B]
@@ -245,12 +256,12 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
     volatile int* abort = (volatile int*)(tmem_slot + 1);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     PDL_ENTER_EARLY();
-    const int r = first_req + blockIdx.z, h = blockIdx.y, qt = gridDim.x - 1 - blockIdx.x;   // long tiles first
+    const int r = first_req + blockIdx.z, h = blockIdx.y * (TA_PAIR + 1), qt = gridDim.x - 1 - blockIdx.x;   // long tiles first
     const int tok0 = cu_tokens[r], n = cu_tokens[r + 1] - tok0;
-    if (qt * TA_BM >= n) return;                           // nothing to do here (before any tensor memory is taken)
+    if (qt * TA_TOK >= n) return;                           // nothing to do here (before any tensor memory is taken)
     if ((smem_u32(smem) & 1023u) != 0) { if (threadIdx.x == 0) atomicExch(error_flag, 20); return; }
     const int len = seq_lens[r], pos0 = len - n;
-    const int rows = min(TA_BM, n - qt * TA_BM);
+    const int rows = min(TA_TOK, n - qt * TA_TOK);
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
         for (int b = 0; b < 2; ++b) { mbar_init(&k_full[b], 1); mbar_init(&v_full[b], 1); mbar_init(&v_free[b], 1); }
@@ -264,7 +275,7 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(TA_TMEM_COLS) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    const int q_first = pos0 + qt * TA_BM, q_last = q_first + rows - 1;
+    const int q_first = pos0 + qt * TA_TOK, q_last = q_first + rows - 1;
     const int k_lo = first_seen(q_first, window, chunk);   // the first key a position sees never decreases with the position
     const int kh = h / GROUP;
     const int kb_first = k_lo / TA_BN, kb_last = q_last / TA_BN;
@@ -330,7 +341,10 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
         if (keys && lane == 0) {
             mbar_expect_tx(q_full, TA_Q_BYTES);
 #pragma unroll
-            for (int hf = 0; hf < NH; ++hf) tma_load_2d(sQ + hf * (TA_BM * 128), &map_q, h * D + hf * 64, tok0 + qt * TA_BM, q_full);
+            for (int hf = 0; hf < NH; ++hf)
+#pragma unroll
+                for (int m = 0; m <= TA_PAIR; ++m)
+                    tma_load_2d(sQ + hf * (TA_BM * 128) + m * (TA_TOK * 128), &map_q, (h + m) * D + hf * 64, tok0 + qt * TA_TOK, q_full);
         }
         load_block(0, row_of(0));
         // the K buffer of block j is free once S of block j - 2 is done, the V buffer once P V of block j - 2 is (rows
@@ -430,7 +444,7 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
         }
     } else {
         // ---- the rows: thread t owns query row t ----
-        const int row_t = threadIdx.x;
+        const int row_t = TA_PAIR ? threadIdx.x & (TA_TOK - 1) : threadIdx.x;
         const int qp = q_first + row_t;
         const int lo_t = first_seen(qp, window, chunk);
         // a score in log2 units is sl2 times the product, or cap_l2 tanh(to_cap times it)
@@ -554,6 +568,52 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
             ok = wait_or_abort(&v_free[(nblk - 1) & 1], ((nblk - 1) >> 1) & 1, abort, error_flag, 24);
             ok = __all_sync(0xffffffffu, ok);
         }
+#if TA_PAIR
+        // every product has ended (v_free of the last block): the key and value buffers are free
+        float* handed = reinterpret_cast<float*>(sKV);         // [V_DIM][64]: column by column, a thread per row
+        const float inv = 1.0f / l_run;
+        if (ok) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (warp >= 2) {
+#pragma unroll
+                for (int c = 0; c < DV / 32; ++c) {
+                    float ov[32];
+                    tmem_ld32(lane_base + TA_O_COL + c * 32, ov);
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) handed[(c * 32 + j) * TA_TOK + row_t] = ov[j] * inv * lam;
+                }
+            }
+        }
+        asm volatile("bar.sync 1, 128;" ::: "memory");         // all four row warps, whether their waits ended or not
+        if (ok && warp < 2) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int c = 0; c < DV / 32; ++c) {
+                float ov[32];
+                tmem_ld32(lane_base + TA_O_COL + c * 32, ov);
+#pragma unroll
+                for (int j = 0; j < 32; ++j) {
+                    float* at = handed + (c * 32 + j) * TA_TOK + row_t;
+                    const float v = fmaf(ov[j], inv, -*at);
+                    *at = v;
+                    ss = fmaf(v, v, ss);
+                }
+            }
+            const float f = out_scale / sqrtf(ss / (float)DV + eps);
+            if (row_t < rows) {
+                bf16* dst = out + (size_t)(tok0 + qt * TA_TOK + row_t) * out_stride + (size_t)(h >> 1) * DV;
+#pragma unroll
+                for (int q8 = 0; q8 < DV / 8; ++q8) {
+                    uint4 packed;
+                    __nv_bfloat162* p2 = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        p2[e] = __floats2bfloat162_rn(handed[(q8 * 8 + 2 * e) * TA_TOK + row_t] * f, handed[(q8 * 8 + 2 * e + 1) * TA_TOK + row_t] * f);
+                    reinterpret_cast<uint4*>(dst)[q8] = packed;
+                }
+            }
+        }
+#else
         if (ok) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const float inv = out_scale / l_run;
@@ -588,6 +648,7 @@ __global__ void __launch_bounds__(256, 2) attn_prefill_tc_kernel(
                 }
             }
         }
+#endif
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
@@ -612,14 +673,14 @@ static int map_2d(CUtensorMap* map, const void* base, uint64_t rows, uint64_t co
 }
 
 // Prefill attention of requests first_req .. first_req+requests-1 (tokens cu_tokens[r]..cu_tokens[r+1], all `tokens`
-// rows of q and out belong to the step); cache_pages pages of page_size (>= 16) positions.
+// rows of q and out belong to the step); cache_pages pages of page_size (>= 16) positions.  lam, eps: with -DPAIR (no sink, no gate).
 MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                               int max_pages, const int* cu_tokens, const int* seq_lens, int first_req, int requests,
                               int max_query_len, int tokens, int K, int page_size, long long cache_pages, float scale,
                               int window, int* error_flag, int chunk, int sink, const void* gate, int gate_stride, const float* sink_logit,
-                              int keep, float softcap, float out_scale, int out_stride, cudaStream_t s) {
+                              int keep, float softcap, float out_scale, int out_stride, float lam, float eps, cudaStream_t s) {
     if (requests <= 0 || max_query_len <= 0) return 0;
-    if (keep < 0 || softcap < 0.0f || out_stride < K * GROUP * DV || out_stride % 8 != 0 || ((uintptr_t)out & 15)) return MB_ERR_BAD_SIZE;
+    if (keep < 0 || softcap < 0.0f || out_stride < K * GROUP / (TA_PAIR + 1) * DV || (TA_PAIR && (gate != nullptr || sink)) || out_stride % 8 != 0 || ((uintptr_t)out & 15)) return MB_ERR_BAD_SIZE;
     if (chunk < 0 || (gate != nullptr && (((uintptr_t)gate & 15) || gate_stride % 8 != 0))) return MB_ERR_BAD_SIZE;
     int page_shift = -1;
     for (int b = 4; b < 16; ++b)
@@ -634,7 +695,7 @@ MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_
         configured = true;
     }
     CUtensorMap mq, mk, mv;
-    int rc = map_2d(&mq, q, (uint64_t)tokens, (uint64_t)K * GROUP * D, TA_BM);
+    int rc = map_2d(&mq, q, (uint64_t)tokens, (uint64_t)K * GROUP * D, TA_TOK);
     if (rc) return rc;
     const uint64_t cache_rows = (uint64_t)cache_pages * K * page_size;
     const int box_rows = page_size < TA_BN ? page_size : TA_BN;
@@ -642,8 +703,8 @@ MB_API int mb_attn_prefill_tc(const void* q, const void* k_cache, const void* v_
     if (rc) return rc;
     rc = TA_V_IN_K ? map_2d(&mv, k_cache, cache_rows, D, box_rows) : map_2d(&mv, v_cache, cache_rows, DV, box_rows);
     if (rc) return rc;
-    dim3 grid((max_query_len + TA_BM - 1) / TA_BM, K * GROUP, requests);
+    dim3 grid((max_query_len + TA_TOK - 1) / TA_TOK, K * GROUP / (TA_PAIR + 1), requests);
     return launch_kernel(softcap > 0.0f ? attn_prefill_tc_kernel<true> : attn_prefill_tc_kernel<false>, grid, 256, TA_SMEM, s, 0, mq, mk, mv, (bf16*)out,
                          block_table, max_pages, cu_tokens, seq_lens, first_req, K, page_shift, scale, window, error_flag, box_rows, chunk, sink, sink_logit,
-                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride);
+                         (const bf16*)gate, gate_stride, keep, softcap, out_scale, out_stride, lam, eps);
 }

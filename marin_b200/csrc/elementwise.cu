@@ -89,14 +89,15 @@ MB_API int mb_last_token(const int* ids, const int* cu_tokens, const int* slots,
     return launch_kernel(last_token_kernel, (requests + 127) / 128, 128, 0, s, 0, ids, cu_tokens, slots, last, requests);
 }
 
-// ---- RMSNorm over rows of a float32 matrix ---------------------------------------------------------
+// ---- RMSNorm over rows of a float32 matrix; `then_add` [n] (or null) is added to the rows themselves behind it (an offset of a sublayer that reads
+// the norm: the sum is the same whenever it is added, and the rows are here anyway) ---------------------------------------------------------
 template <typename TO>
-__global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps, int unit_offset,
-                               TO* __restrict__ out, int n) {
+__global__ void rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ w, float eps, int unit_offset,
+                               TO* __restrict__ out, int n, const float* __restrict__ then_add) {
     PDL_ENTER();
     x = pdl_fresh(x);
     __shared__ float scratch[32];
-    const float* row = x + (size_t)blockIdx.x * n;
+    float* row = x + (size_t)blockIdx.x * n;
     TO* dst = out + (size_t)blockIdx.x * n;
     float ss = 0.0f;
     for (int i = threadIdx.x; i < n; i += blockDim.x) { float v = row[i]; ss += v * v; }
@@ -104,19 +105,21 @@ __global__ void rmsnorm_kernel(const float* __restrict__ x, const float* __restr
     const float scale = 1.0f / sqrtf(ss / (float)n + eps);
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
         const float wi = unit_offset ? 1.0f + w[i] : w[i];
-        dst[i] = from_f32<TO>(row[i] * scale * wi);
+        const float v = row[i];
+        dst[i] = from_f32<TO>(v * scale * wi);
+        if (then_add != nullptr) row[i] = v + then_add[i];
     }
 }
 
 // The same with the row held in registers: 16-byte loads, one pass over memory.  n is a multiple of 4, at most
 // 1024 * R (R float4 per thread).
 template <typename TO, int R>
-__global__ void __launch_bounds__(256) rmsnorm_vec_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps,
-                                                          int unit_offset, TO* __restrict__ out, int n) {
+__global__ void __launch_bounds__(256) rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ w, float eps,
+                                                          int unit_offset, TO* __restrict__ out, int n, const float* __restrict__ then_add) {
     PDL_ENTER();
     x = pdl_fresh(x);
     __shared__ float scratch[32];
-    const float4* row = reinterpret_cast<const float4*>(x + (size_t)blockIdx.x * n);
+    float4* row = reinterpret_cast<float4*>(x + (size_t)blockIdx.x * n);
     const float4* w4 = reinterpret_cast<const float4*>(w);
     const int n4 = n >> 2;
     float4 v[R];
@@ -146,26 +149,30 @@ __global__ void __launch_bounds__(256) rmsnorm_vec_kernel(const float* __restric
                 packed.y = *reinterpret_cast<uint32_t*>(&hi);
                 reinterpret_cast<uint2*>(dst)[i] = packed;
             }
+            if (then_add != nullptr) {
+                const float4 t = reinterpret_cast<const float4*>(then_add)[i];
+                row[i] = make_float4(v[r].x + t.x, v[r].y + t.y, v[r].z + t.z, v[r].w + t.w);
+            }
         }
     }
 }
 
-MB_API int mb_rmsnorm(const float* x, const float* w, float eps, int unit_offset, void* out, int out_dtype,
-                      int rows, int n, cudaStream_t s) {
+MB_API int mb_rmsnorm(float* x, const float* w, float eps, int unit_offset, void* out, int out_dtype,
+                      int rows, int n, const float* then_add, cudaStream_t s) {
     if (rows <= 0) return 0;
     if (out_dtype != MB_F32 && out_dtype != MB_BF16) return MB_ERR_BAD_DTYPE;
-    const bool vec = n % 4 == 0 && n <= 8192 && n >= 512 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0;
+    const bool vec = n % 4 == 0 && n <= 8192 && n >= 512 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)then_add & 15) == 0;
     if (vec && n <= 4096) {
-        if (out_dtype == MB_F32) return launch_kernel(rmsnorm_vec_kernel<float, 4>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (float*)out, n);
-        return launch_kernel(rmsnorm_vec_kernel<bf16, 4>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n);
+        if (out_dtype == MB_F32) return launch_kernel(rmsnorm_vec_kernel<float, 4>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (float*)out, n, then_add);
+        return launch_kernel(rmsnorm_vec_kernel<bf16, 4>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n, then_add);
     }
     if (vec) {
-        if (out_dtype == MB_F32) return launch_kernel(rmsnorm_vec_kernel<float, 8>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (float*)out, n);
-        return launch_kernel(rmsnorm_vec_kernel<bf16, 8>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n);
+        if (out_dtype == MB_F32) return launch_kernel(rmsnorm_vec_kernel<float, 8>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (float*)out, n, then_add);
+        return launch_kernel(rmsnorm_vec_kernel<bf16, 8>, rows, 256, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n, then_add);
     }
     const int threads = n >= 1024 ? 256 : 128;
-    if (out_dtype == MB_F32) return launch_kernel(rmsnorm_kernel<float>, rows, threads, 0, s, 0, x, w, eps, unit_offset, (float*)out, n);
-    return launch_kernel(rmsnorm_kernel<bf16>, rows, threads, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n);
+    if (out_dtype == MB_F32) return launch_kernel(rmsnorm_kernel<float>, rows, threads, 0, s, 0, x, w, eps, unit_offset, (float*)out, n, then_add);
+    return launch_kernel(rmsnorm_kernel<bf16>, rows, threads, 0, s, 0, x, w, eps, unit_offset, (bf16*)out, n, then_add);
 }
 
 // ---- per-head RMSNorm of q and k, rotation of q and k, k and v into their pages ---------------------
@@ -350,9 +357,10 @@ MB_API int mb_qk_norm_rope_write(const void* qkv, int dtype, void* q_out, const 
 }
 
 // ---- SwiGLU: out[t, i] = g / (1 + exp(-g)) * u with g = gu[t, i], u = gu[t, I + i]; or, interleaved, with gate and
-// up in alternating blocks of 16 columns: g = gu[t, 32 (i / 16) + i % 16], u = 16 columns further.  act 1: max(g, 0) * u ----
+// up in alternating blocks of 16 columns: g = gu[t, 32 (i / 16) + i % 16], u = 16 columns further.  act 1: max(g, 0) * u; act 2: the tanh
+// form of gelu.  All of it times `factor`; output rows out_stride apart ----
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t total, int interleaved, int act) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t total, int interleaved, int act, float factor, int out_stride) {
     PDL_ENTER();
     gu = pdl_fresh(gu);
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -362,7 +370,8 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const size_t gi = interleaved ? (i >> 4) * 32 + (i & 15) : i;
         const size_t ui = interleaved ? gi + 16 : I + i;
         const float g = to_f32(gu[t * 2 * I + gi]), u = to_f32(gu[t * 2 * I + ui]);
-        out[idx] = from_f32<T>((act == 1 ? fmaxf(g, 0.0f) : g / (1.0f + expf(-g))) * u);
+        const float a = act == 1 ? fmaxf(g, 0.0f) : act == 2 ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
+        out[t * out_stride + i] = from_f32<T>(a * u * factor);
     }
 }
 
@@ -385,13 +394,14 @@ MB_API int mb_rope_table(const int* positions, const float* inv_freq, int half, 
     return launch_kernel(rope_table_kernel, dim3((total + 255) / 256), dim3(256), 0, s, 0, positions, inv_freq, half, out, T);
 }
 
-MB_API int mb_swiglu(const void* gate_up, void* out, int dtype, int tokens, int I, int interleaved, int act, cudaStream_t s) {
+MB_API int mb_swiglu(const void* gate_up, void* out, int dtype, int tokens, int I, int interleaved, int act, float factor, int out_stride, cudaStream_t s) {
     const size_t total = (size_t)tokens * I;
     if (total == 0) return 0;
+    if (act < 0 || act > 2 || out_stride < I) return MB_ERR_BAD_SIZE;
     const int threads = 256;
     const int blocks = (int)((total + threads - 1) / threads < 148 * 16 ? (total + threads - 1) / threads : 148 * 16);
-    if (dtype == MB_F32) return launch_kernel(swiglu_kernel<float>, blocks, threads, 0, s, 0, (const float*)gate_up, (float*)out, I, total, interleaved, act);
-    else if (dtype == MB_BF16) return launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, s, 0, (const bf16*)gate_up, (bf16*)out, I, total, interleaved, act);
+    if (dtype == MB_F32) return launch_kernel(swiglu_kernel<float>, blocks, threads, 0, s, 0, (const float*)gate_up, (float*)out, I, total, interleaved, act, factor, out_stride);
+    else if (dtype == MB_BF16) return launch_kernel(swiglu_kernel<bf16>, blocks, threads, 0, s, 0, (const bf16*)gate_up, (bf16*)out, I, total, interleaved, act, factor, out_stride);
     else return MB_ERR_BAD_DTYPE;
     return mb_last_error();
 }
@@ -408,6 +418,24 @@ __global__ void gather_rows_kernel(const float* __restrict__ src, const int* __r
 MB_API int mb_gather_rows(const float* src, const int* rows, float* out, int count, int h, cudaStream_t s) {
     if (count <= 0) return 0;
     return launch_kernel(gather_rows_kernel, count, 256, 0, s, 0, src, rows, out, h);
+}
+
+// ---- out = x (+ y) (+ v, one vector for every row): float32 rows, x and out may be the same -----------------------------------
+__global__ void stream_enter_kernel(const float* x, const float* __restrict__ y, const float* __restrict__ v, float* out, int n) {
+    PDL_ENTER();
+    x = pdl_fresh(x); y = pdl_fresh(y);
+    const size_t at = (size_t)blockIdx.x * n;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        float a = x[at + i];
+        if (y != nullptr) a += y[at + i];
+        if (v != nullptr) a += v[i];
+        out[at + i] = a;
+    }
+}
+
+MB_API int mb_stream_enter(const float* x, const float* y, const float* v, float* out, int rows, int n, cudaStream_t s) {
+    if (rows <= 0) return 0;
+    return launch_kernel(stream_enter_kernel, rows, 256, 0, s, 0, x, y, v, out, n);
 }
 
 // ---- y += x (float32 residual, x in the activation dtype) ---------------------------------------------

@@ -217,7 +217,7 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
                                                       int mode, int T, int N, int K, int kb_per_split,
                                                       float* __restrict__ partials, int* __restrict__ counters,
                                                       int* __restrict__ error_flag, int cluster_reduce,
-                                                      const TcNormOut norm, const TcRowScale scale, const TcHeadsOut heads) {
+                                                      const TcNormOut norm, const TcRowScale scale, const TcHeadsOut heads, const TcGlu glu) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ float s_scale[BN];
     __shared__ float s_head[TC_BM], s_part[4];
@@ -554,8 +554,8 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
         }
         if (direct && norm.weight != nullptr) {
             store_chunk_norm(out, t0 + c0, n, n < N, T, N, v, norm, norm.sumsq + (size_t)(blockIdx.x * 4 + warp) * T, lane);
-        } else if (direct && (mode == TC_OUT_SWIGLU || mode == TC_OUT_REGLU)) {
-            if (n0 + warp * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + warp * 32, lane, T, N, v, mode == TC_OUT_REGLU);
+        } else if (direct && tc_gated(mode)) {
+            if (n0 + warp * 32 < N) store_chunk_glu(out, mode, t0 + c0, n0 + warp * 32, lane, T, N, v, glu);
         } else if (n < N) {
             if (direct) store_chunk(out, mode, t0 + c0, n, T, N, v);
             else {
@@ -686,7 +686,7 @@ __global__ void __launch_bounds__(320) gemm_tc_persistent_kernel(const __grid_co
                                                                  int* __restrict__ error_flag, const TcNormOut norm,
                                                                  const TcRowScale scale, const TcStreamK sk, const TcHeadsOut heads,
                                                                  const float* __restrict__ rope,
-                                                                 const __grid_constant__ CUtensorMap map_out, int reduce_out) {
+                                                                 const __grid_constant__ CUtensorMap map_out, int reduce_out, const TcGlu glu) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ float s_pscale[2][BN];          // the per-token factors of a coupled norm, for the tile in each accumulator
     // heads finished in the epilogue: per half of the columns (its four warps), two staging buffers of sixteen tokens
@@ -930,8 +930,8 @@ __global__ void __launch_bounds__(320) gemm_tc_persistent_kernel(const __grid_co
                 }
                 if (norm.weight != nullptr) {
                     store_chunk_norm(out, t0 + c0, n, n < N, T, N, v, norm, norm.sumsq + (size_t)(tile_row * 4 + quarter) * T, lane);
-                } else if (mode == TC_OUT_SWIGLU || mode == TC_OUT_REGLU) {
-                    if (n0 + quarter * 32 < N) store_chunk_swiglu(out, t0 + c0, n0 + quarter * 32, lane, T, N, v, mode == TC_OUT_REGLU);
+                } else if (tc_gated(mode)) {
+                    if (n0 + quarter * 32 < N) store_chunk_glu(out, mode, t0 + c0, n0 + quarter * 32, lane, T, N, v, glu);
                 } else if (reduce_out) {
                     // "+=" into float32 without reading the old values: the four warps that share this half of the columns
                     // lay sixteen tokens of the tile into shared memory and one thread hands them to a TMA reduction
@@ -1052,10 +1052,17 @@ __global__ void __launch_bounds__(320) gemm_tc_persistent_kernel(const __grid_co
 #define TC_STAGES16 6          // ring depth with up to 16 tokens per CTA
 #endif
 
+static const TcGlu TC_PLAIN_GLU = {1.0f, 0, 0, nullptr};
+
+static bool glu_fits(const TcGlu& glu, int mode, int N) {
+    if (!tc_gated(mode)) return glu.from == 0;
+    return glu.from >= 0 && glu.from % 32 == 0 && glu.from < N && (glu.from == 0 || glu.rows != nullptr) && (glu.stride == 0 || glu.stride >= (N - glu.from) / 2);
+}
+
 template <int BN, int STAGES>
 static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int mode, int T, int N, int K, int splits,
                      int kb_per_split, float* partials, int* counters, int* error_flag, int cluster_reduce,
-                     const TcNormOut& norm, const TcRowScale& scale, const TcHeadsOut& heads, cudaStream_t s) {
+                     const TcNormOut& norm, const TcRowScale& scale, const TcHeadsOut& heads, const TcGlu& glu, cudaStream_t s) {
     constexpr int smem = STAGES * TcSmem<BN>::STAGE_BYTES + 1024 + 256;
     static_assert(STAGES * TcSmem<BN>::STAGE_BYTES >= BN * TC_BM * 4, "the cluster reduction reuses the pipeline buffers");
     static bool configured = false;
@@ -1067,7 +1074,7 @@ static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* out, in
     const bool clustered = cluster_reduce && splits > 1;
     return launch_kernel(gemm_tc_kernel<BN, STAGES>, dim3((N + TC_BM - 1) / TC_BM, (T + BN - 1) / BN, splits), dim3(128), smem, s,
                          clustered ? splits : 0, mw, mx, out, mode, T, N, K, kb_per_split, partials, counters, error_flag,
-                         clustered ? 1 : 0, norm, scale, heads);
+                         clustered ? 1 : 0, norm, scale, heads, glu);
 }
 
 // Tiles a launch with `bn` tokens per CTA would have (for the caller's choice of split).
@@ -1086,7 +1093,7 @@ static bool tc_reduce_out() {
 template <int BN, int STAGES, bool SK>
 static int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mx, void* out, int mode, int T, int N, int K, int ctas,
                              int* error_flag, const TcNormOut& norm, const TcRowScale& scale, TcStreamK sk, cudaStream_t s,
-                             const TcHeadsOut& heads = TcHeadsOut{}, const float* rope = nullptr) {
+                             const TcGlu& glu, const TcHeadsOut& heads = TcHeadsOut{}, const float* rope = nullptr) {
     // "+=" into float32 with nothing riding on it: by TMA reduction, if the rows of out can be a tensor map's
     CUtensorMap mo = mw;
     int reduce_out = 0;
@@ -1118,15 +1125,15 @@ static int launch_persistent(const CUtensorMap& mw, const CUtensorMap& mx, void*
         grid = groups * tiles_t;
     }
     return launch_kernel(gemm_tc_persistent_kernel<BN, STAGES, SK>, dim3(grid), dim3(320), smem, s, 0, mw, mx, out, mode, T, N, K,
-                         error_flag, norm, scale, sk, heads, rope, mo, reduce_out);
+                         error_flag, norm, scale, sk, heads, rope, mo, reduce_out, glu);
 }
 
 static int persistent_dispatch(const void* x, const void* w, void* out, int mode, int T, int N, int K, int bn, int ctas,
                                int* error_flag, const TcNormOut& norm, const TcRowScale& scale, const TcStreamK& sk, cudaStream_t s,
-                               const TcHeadsOut& heads = TcHeadsOut{}, const float* rope = nullptr) {
+                               const TcHeadsOut& heads = TcHeadsOut{}, const float* rope = nullptr, const TcGlu& glu = TC_PLAIN_GLU) {
     if (T <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ctas <= 0) return MB_ERR_BAD_SIZE;
-    if (mode < 0 || mode > 5 || ((mode == 3 || mode == 5) && N % 32 != 0)) return MB_ERR_BAD_DTYPE;
+    if (mode < 0 || mode >= TC_OUT_MODES || (tc_gated(mode) && N % 32 != 0) || !glu_fits(glu, mode, N)) return MB_ERR_BAD_DTYPE;
     if (norm.weight != nullptr && (mode != TC_OUT_F32_ACC || norm.scaled == nullptr || norm.sumsq == nullptr)) return MB_ERR_BAD_DTYPE;
     if (scale.sumsq != nullptr && (scale.slots <= 0 || scale.dim <= 0)) return MB_ERR_BAD_SIZE;
     CUtensorMap mw, mx;
@@ -1136,22 +1143,22 @@ static int persistent_dispatch(const void* x, const void* w, void* out, int mode
     if (rc) return rc;
     if (sk.partials != nullptr) {
         switch (bn) {                                   // stream-K: three widths
-            case 128: return launch_persistent<128, 6, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s);
-            case 192: return launch_persistent<192, 5, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s);
-            case 256: return launch_persistent<256, 4, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s);
+            case 128: return launch_persistent<128, 6, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu);
+            case 192: return launch_persistent<192, 5, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu);
+            case 256: return launch_persistent<256, 4, true>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu);
             default: return MB_ERR_BAD_SIZE;
         }
     }
     switch (bn) {
-        case 128: return launch_persistent<128, 6, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 144: return launch_persistent<144, 6, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 160: return launch_persistent<160, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 176: return launch_persistent<176, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 192: return launch_persistent<192, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 208: return launch_persistent<208, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 224: return launch_persistent<224, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 240: return launch_persistent<240, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
-        case 256: return launch_persistent<256, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, heads, rope);
+        case 128: return launch_persistent<128, 6, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 144: return launch_persistent<144, 6, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 160: return launch_persistent<160, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 176: return launch_persistent<176, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 192: return launch_persistent<192, 5, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 208: return launch_persistent<208, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 224: return launch_persistent<224, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 240: return launch_persistent<240, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
+        case 256: return launch_persistent<256, 4, false>(mw, mx, out, mode, T, N, K, ctas, error_flag, norm, scale, sk, s, glu, heads, rope);
         default: return MB_ERR_BAD_SIZE;
     }
 }
@@ -1218,7 +1225,7 @@ MB_API int mb_gemm_tc_persistent_heads(const void* x, const void* w, int T, int 
 // (one zeroed int per tile).  bn in {16, 32, 64, 128, 256}.
 static int gemm_tc_dispatch(const void* x, const void* w, void* out, int mode, int T, int N, int K, int bn, int splits,
                             float* partials, int* counters, int* error_flag, int cluster_reduce, const TcNormOut& norm,
-                            const TcRowScale& scale, const TcHeadsOut& heads, cudaStream_t s) {
+                            const TcRowScale& scale, const TcHeadsOut& heads, cudaStream_t s, const TcGlu& glu = TC_PLAIN_GLU) {
     if (T <= 0 || N <= 0) return 0;
     // heads are finished only where the K slices of a tile meet as a cluster
     if (heads.q_out != nullptr && (!cluster_reduce || splits < 2 || N % TC_BM != 0 || bn > 128 || T > bn)) return MB_ERR_BAD_SIZE;
@@ -1227,7 +1234,7 @@ static int gemm_tc_dispatch(const void* x, const void* w, void* out, int mode, i
     if (norm.weight != nullptr && !cluster_reduce && splits > 1) return MB_ERR_BAD_SIZE;
     if (scale.sumsq != nullptr && (scale.slots <= 0 || scale.dim <= 0 || (!cluster_reduce && splits > 1))) return MB_ERR_BAD_SIZE;
     if (K <= 0 || K % 8 != 0 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15)) return MB_ERR_BAD_SIZE;
-    if (mode < 0 || mode > 5 || ((mode == 3 || mode == 5) && (splits > 1 || N % 32 != 0))) return MB_ERR_BAD_DTYPE;
+    if (mode < 0 || mode >= TC_OUT_MODES || (tc_gated(mode) && (splits > 1 || N % 32 != 0)) || !glu_fits(glu, mode, N)) return MB_ERR_BAD_DTYPE;
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     if (splits < 1) splits = 1;
     if (splits > total_kb) splits = total_kb;
@@ -1246,11 +1253,11 @@ static int gemm_tc_dispatch(const void* x, const void* w, void* out, int mode, i
     rc = make_map(&mx, x, T, K, bn);
     if (rc) return rc;
     switch (bn) {
-        case 16: return launch_tc<16, TC_STAGES16>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, s);
-        case 32: return launch_tc<32, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, s);
-        case 64: return launch_tc<64, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, s);
-        case 128: return launch_tc<128, 3>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, s);
-        case 256: return launch_tc<256, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, s);
+        case 16: return launch_tc<16, TC_STAGES16>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, glu, s);
+        case 32: return launch_tc<32, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, glu, s);
+        case 64: return launch_tc<64, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, glu, s);
+        case 128: return launch_tc<128, 3>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, glu, s);
+        case 256: return launch_tc<256, 4>(mw, mx, out, mode, T, N, K, splits, kb_per_split, partials, counters, error_flag, cluster_reduce, norm, scale, heads, glu, s);
         default: return MB_ERR_BAD_SIZE;
     }
 }
@@ -1268,6 +1275,23 @@ MB_API int mb_gemm_tc(const void* x, const void* w, void* out, int mode, int T, 
 MB_API int mb_gemm_tc_cluster(const void* x, const void* w, void* out, int mode, int T, int N, int K, int bn, int splits,
                               int* error_flag, cudaStream_t s) {
     return gemm_tc_dispatch(x, w, out, mode, T, N, K, bn, splits, nullptr, nullptr, error_flag, 1, TcNormOut{}, TcRowScale{}, TcHeadsOut{}, s);
+}
+
+// A gated product with its further choices (TcGlu; mode one of the gated ones): ctas 0: one CTA per tile of bn tokens; else the persistent
+// kernel, stream-K where parked is given (see mb_gemm_tc_persistent_streamk, whose conditions hold).
+MB_API int mb_gemm_tc_glu(const void* x, const void* w, void* out, int mode, int T, int N, int K, int bn, int ctas, float factor, int stride, int from,
+                          void* rows, float* parked, long long parked_floats, int* flags, int* error_flag, cudaStream_t s) {
+    if (T <= 0 || N <= 0) return 0;
+    if (!tc_gated(mode)) return MB_ERR_BAD_DTYPE;
+    const TcGlu glu = {factor, stride, from, (bf16*)rows};
+    if (ctas <= 0) return gemm_tc_dispatch(x, w, out, mode, T, N, K, bn, 1, nullptr, nullptr, error_flag, 1, TcNormOut{}, TcRowScale{}, TcHeadsOut{}, s, glu);
+    if (parked != nullptr) {
+        const int sms = sm_count_of_current_device();
+        const int tiles_n = (N + TC_BM - 1) / TC_BM, tiles_t = bn > 0 ? (T + bn - 1) / bn : 0;
+        if (sms <= 0 || flags == nullptr || tiles_t <= 0 || ctas > sms || tiles_t > ctas || tiles_n < ctas / tiles_t || parked_floats < (long long)ctas * bn * TC_BM)
+            return MB_ERR_BAD_SIZE;
+    }
+    return persistent_dispatch(x, w, out, mode, T, N, K, bn, ctas, error_flag, TcNormOut{}, TcRowScale{}, TcStreamK{parked, flags, 0}, s, TcHeadsOut{}, nullptr, glu);
 }
 
 // Slots of sums of squares per token that a "+=" product over N weight rows with `splits` K slices writes.

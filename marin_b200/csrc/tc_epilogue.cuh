@@ -11,7 +11,20 @@
 #define TC_OUT_F32_ACC 2
 #define TC_OUT_SWIGLU 3       // w holds gate and up rows interleaved in blocks of 16; out [T, N/2] bf16 = silu(gate) * up
 #define TC_OUT_REGLU 5        // as TC_OUT_SWIGLU with max(gate, 0) * up
+#define TC_OUT_GEGLU 6        // as TC_OUT_SWIGLU with the tanh form of gelu of the gate
 #define TC_OUT_RELU2 4        // out bf16 = max(x w^T, 0)^2: the activation of a feed-forward without a gate
+#define TC_OUT_MODES 7
+
+__host__ __device__ __forceinline__ bool tc_gated(int mode) { return mode == TC_OUT_SWIGLU || mode == TC_OUT_REGLU || mode == TC_OUT_GEGLU; }
+
+// A gated mode's further choices: the result times `factor`; output rows `stride` elements apart (0: as many as there are
+// gate rows); and `from` weight rows (a multiple of 32) ahead of the gate and up rows that are a plain product, written in bf16 to `rows`
+// [T][from]: what a feed-forward and whatever else reads the same input take from it is one product.
+struct TcGlu {
+    float factor;
+    int stride, from;
+    bf16* rows;
+};
 
 __device__ __forceinline__ float relu2_of(float v) { v = fmaxf(v, 0.0f); return v * v; }
 
@@ -58,21 +71,31 @@ __device__ __forceinline__ void store_chunk(void* out, int mode, int t_first, in
     }
 }
 
-// SwiGLU in the epilogue.  The weight rows of a warp's 32 accumulator lanes are 16 gate rows followed by the 16 up
+// A gated activation in the epilogue.  The weight rows of a warp's 32 accumulator lanes are 16 gate rows followed by the 16 up
 // rows of the same intermediate indices, so lane l < 16 holds gate(i) and lane l + 16 holds up(i): one shuffle brings
-// them together and out[t, i] = g / (1 + exp(-g)) * u is written in bf16 (crates/tensor/src/silu.rs:18; the fast
-// exponential and division are accurate to a few float32 ulps, far inside the bf16 rounding of the result).  All 32
-// lanes must call this; n_base is the warp's first weight row (a multiple of 32).  relu: max(g, 0) * u instead.
-__device__ __forceinline__ void store_chunk_swiglu(void* out, int t_first, int n_base, int lane, int T, int N, const float* v, bool relu) {
+// them together and out[t, i] = act(g) * u is written in bf16: g / (1 + exp(-g)) (crates/tensor/src/silu.rs:18; the fast
+// exponential and division are accurate to a few float32 ulps, far inside the bf16 rounding of the result), max(g, 0), or the tanh form of
+// gelu, 0.5 g (1 + tanh(y)) = g / (1 + exp(-2 y)).  All 32 lanes must call this; n_base is the warp's first weight row (a multiple of 32).
+__device__ __forceinline__ float glu_gate(int mode, float g) {
+    if (mode == TC_OUT_REGLU) return fmaxf(g, 0.0f);
+    const float y = mode == TC_OUT_GEGLU ? 1.5957691216057308f * fmaf(0.044715f * g, g * g, g) : g;
+    return __fdividef(g, 1.0f + __expf(-y));
+}
+
+__device__ __forceinline__ void store_chunk_glu(void* out, int mode, int t_first, int n_base, int lane, int T, int N, const float* v, const TcGlu& glu) {
+    if (n_base < glu.from) {                                   // (a warp's rows are all on one side)
+#pragma unroll
+        for (int j = 0; j < 16; ++j)
+            if (t_first + j < T) glu.rows[(size_t)(t_first + j) * glu.from + n_base + lane] = __float2bfloat16_rn(v[j]);
+        return;
+    }
     bf16* o = (bf16*)out;
-    const int half = N >> 1;
-    const int i = (n_base >> 1) + (lane & 15);
+    const int half = (N - glu.from) >> 1, stride = glu.stride > 0 ? glu.stride : half;
+    const int i = ((n_base - glu.from) >> 1) + (lane & 15);
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
         const float u = __shfl_down_sync(0xffffffffu, v[j], 16);
-        const float g = v[j];
-        if (lane < 16 && t_first + j < T && i < half)
-            o[(size_t)(t_first + j) * half + i] = __float2bfloat16_rn((relu ? fmaxf(g, 0.0f) : __fdividef(g, 1.0f + __expf(-g))) * u);
+        if (lane < 16 && t_first + j < T && i < half) o[(size_t)(t_first + j) * stride + i] = __float2bfloat16_rn(glu_gate(mode, v[j]) * u * glu.factor);
     }
 }
 

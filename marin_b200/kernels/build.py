@@ -163,6 +163,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "mb_ssm": ["ssm.cu"],
     "mb_layer_norm": ["layer_norm.cu"],
     "mb_delta_rule": ["delta_rule.cu"],
+    "mb_gated_linear": ["gated_linear.cu"],
     "mb_host": ["host/cache_core.cpp", "host/scheduler.cpp", "host/sampler.cpp", "host/safetensors.cpp"],
 }
 
@@ -200,16 +201,18 @@ def attention_job(d: int, group: int) -> tuple:
     return (["attention_fast.cu"], [f"HEAD_DIM={d}", f"GROUP={group}"])
 
 
-def attention_tc_job(d: int, group: int, dv: int = 0, values_in_keys: bool = False) -> tuple:
-    """Sources and defines of the tensor-core prefill attention kernel for one head layout (``values_in_keys``: the
-    values are the first ``dv`` elements of the key rows)."""
-    if not values_in_keys:
-        return (["attention_tc.cu"], [f"HEAD_DIM={d}", f"GROUP={group}"])
-    return (["attention_tc.cu"], [f"HEAD_DIM={d}", f"V_DIM={dv}", f"GROUP={group}", "V_IN_K"])
+def attention_tc_job(d: int, group: int, dv: int = 0, values_in_keys: bool = False, pair: bool = False) -> tuple:
+    """Sources and defines of the tensor-core prefill attention kernel for one head layout (``dv`` 0: values as wide as the keys;
+    ``values_in_keys``: the values are the first ``dv`` elements of the key rows; ``pair``: query heads are pairs of maps)."""
+    if values_in_keys:
+        return (["attention_tc.cu"], [f"HEAD_DIM={d}", f"V_DIM={dv}", f"GROUP={group}", "V_IN_K"])
+    return (["attention_tc.cu"], [f"HEAD_DIM={d}", f"GROUP={group}"] + ([f"V_DIM={dv}"] if dv not in (0, d) else []) + (["PAIR"] if pair else []))
 
 
-def attention_tc_name(d: int, group: int, dv: int = 0, values_in_keys: bool = False) -> str:
-    return f"mb_attention_tc_d{d}_g{group}" if not values_in_keys else f"mb_attention_tc_d{d}_v{dv}_g{group}_vk"
+def attention_tc_name(d: int, group: int, dv: int = 0, values_in_keys: bool = False, pair: bool = False) -> str:
+    if values_in_keys:
+        return f"mb_attention_tc_d{d}_v{dv}_g{group}_vk"
+    return f"mb_attention_tc_d{d}" + (f"_v{dv}" if dv not in (0, d) else "") + f"_g{group}" + ("_pair" if pair else "")
 
 
 #: One or two layouts of every source that is otherwise compiled for a model's own sizes when it first runs (the names and

@@ -144,13 +144,27 @@ def embed_bigram(ctx, table: torch.Tensor, pairs: torch.Tensor, last: torch.Tens
                "last token kept")
 
 
-def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, unit_offset: bool = False) -> None:
-    _need_cuda(x, weight, out)
+def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, unit_offset: bool = False,
+            then_add: Optional[torch.Tensor] = None) -> None:
+    """``out = x / sqrt(mean(x^2) + eps) * weight`` (``1 + weight`` with ``unit_offset``); behind it ``x += then_add`` (float32 ``[n]``) where that
+    is given."""
+    _need_cuda(x, weight, out, then_add)
+    assert then_add is None or (then_add.dtype == torch.float32 and then_add.numel() == x.shape[1])
     rows, n = x.shape
     assert x.dtype == torch.float32 and weight.dtype == torch.float32 and weight.numel() == n and out.shape == x.shape
-    _cost(_size(x) + _size(out) + _size(weight), 4.0 * rows * n)
+    _cost(_size(x) * (2 if then_add is not None else 1) + _size(out) + _size(weight), 4.0 * rows * n)
     _check(_lib("mb_elementwise").mb_rmsnorm(_ptr(x), _ptr(weight), _c_float(eps), _c_int(int(unit_offset)), _ptr(out),
-                                            _code(out), _c_int(rows), _c_int(n), _stream()), "rmsnorm")
+                                            _code(out), _c_int(rows), _c_int(n), _ptr(then_add), _stream()), "rmsnorm")
+
+
+def stream_enter(x: torch.Tensor, y: Optional[torch.Tensor], v: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """``out = x (+ y) (+ v)``: float32 rows, ``v`` one vector for every row; ``out`` may be ``x``."""
+    _need_cuda(x, y, v, out)
+    rows, n = x.shape
+    assert x.dtype == torch.float32 and out.dtype == torch.float32 and out.shape == x.shape and x.is_contiguous() and out.is_contiguous()
+    assert (y is None or (y.dtype == torch.float32 and y.shape == x.shape and y.is_contiguous())) and (v is None or (v.dtype == torch.float32 and v.numel() == n))
+    _cost(_size(x) + _size(out) + (_size(y) if y is not None else 0))
+    _check(_lib("mb_elementwise").mb_stream_enter(_ptr(x), _ptr(y), _ptr(v), _ptr(out), _c_int(rows), _c_int(n), _stream()), "stream entered")
 
 
 #: bf16 products go to the tcgen05 kernel when their shape allows (False: always the plain kernel)
@@ -721,7 +735,7 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
                                          _c_int(ctx.max_query_len), _c_int(T), _c_int(K), _c_int(page_size),
                                          ctypes.c_longlong(k_cache.shape[0]), _c_float(scale), _c_int(window),
                                          _ptr(_scratch_for(q.device).error), _c_int(0), _c_int(0), _ptr(None), _c_int(0), _ptr(None),
-                                         _c_int(0), _c_float(0.0), _c_float(1.0), _c_int(H * d), _stream()),
+                                         _c_int(0), _c_float(0.0), _c_float(1.0), _c_int(H * d), _c_float(0.0), _c_float(0.0), _stream()),
                    "attention (prefill, tensor cores)")
         elif ctx.num_requests > nd:
             _attention_cost(q, T - nd, H, K, d, "prefill")
@@ -738,19 +752,20 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
 
 
 #: activations of a gated feed-forward and, for each, the output mode of the tensor-core product that applies it in its epilogue
-GLU_ACTIVATIONS = {"silu": 0, "relu": 1}
-_GLU_MODES = {"silu": 3, "relu": 5}
+GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
+_GLU_MODES = {"silu": 3, "relu": 5, "gelu_tanh": 6}
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, activation: str = "silu") -> None:
-    """``out[t, i] = act(g) * u`` (``activation`` "silu" or "relu"); gate and up are the two halves of a row of ``gate_up``, or (``interleaved``)
-    alternate in blocks of 16 columns."""
-    _need_cuda(gate_up, out)
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleaved: bool = False, activation: str = "silu", factor: float = 1.0) -> None:
+    """``out[t, i] = act(g) * u * factor`` (``activation`` "silu", "relu" or "gelu_tanh"); gate and up are the two halves of a row of ``gate_up``, or
+    (``interleaved``) alternate in blocks of 16 columns.  ``out`` may be a column block of a wider buffer."""
+    _need_cuda(gate_up)
     T, I = out.shape
+    assert out.is_cuda and out.stride(1) == 1
     assert gate_up.shape == (T, 2 * I) and gate_up.dtype == out.dtype and (not interleaved or I % 16 == 0)
     _cost(_size(gate_up) + _size(out), 8.0 * T * I)
     _check(_lib("mb_elementwise").mb_swiglu(_ptr(gate_up), _ptr(out), _code(out), _c_int(T), _c_int(I), _c_int(int(interleaved)),
-                                           _c_int(GLU_ACTIVATIONS[activation]), _stream()), "swiglu")
+                                           _c_int(GLU_ACTIVATIONS[activation]), _c_float(factor), _c_int(out.stride(0)), _stream()), "swiglu")
 
 
 def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
@@ -765,14 +780,45 @@ def can_fuse_swiglu(dtype, hidden: int, intermediate: int) -> bool:
     return dtype == torch.bfloat16 and intermediate % 16 == 0 and hidden % 8 == 0
 
 
-def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor, workspace=None, activation: str = "silu") -> None:
-    """``out = act(x Wg^T) * (x Wu^T)`` (``activation`` "silu" or "relu") with ``w_interleaved = interleave_gate_up(Wg, Wu)``: on the tensor cores the
-    activation is applied to the float32 accumulators in the epilogue and the ``[T, 2 I]`` intermediate never
+def gemm_glu_rows(x: torch.Tensor, w: torch.Tensor, rows: Optional[torch.Tensor], out: torch.Tensor, activation: str, factor: float = 1.0) -> None:
+    """One tensor-core product for a feed-forward's gate and up projections and for whatever else reads the same input: ``w`` is a plain matrix of
+    ``rows.shape[1]`` rows (a multiple of 32; ``rows`` None: there is none), whose result goes to ``rows``, above ``interleave_gate_up(Wg, Wu)``, whose
+    activated result times ``factor`` goes to ``out`` (rows may be strided).  bfloat16 only."""
+    _need_cuda(x, w, rows)
+    T, K = x.shape
+    N, P = w.shape[0], rows.shape[1] if rows is not None else 0
+    I = (N - P) // 2
+    assert w.shape[1] == K and tuple(out.shape) == (T, I) and out.is_cuda and out.stride(1) == 1 and P % 32 == 0 and (N - P) % 32 == 0 and K % 8 == 0
+    assert x.dtype == w.dtype == out.dtype == torch.bfloat16 and (rows is None or (rows.dtype == torch.bfloat16 and tuple(rows.shape) == (T, P)))
+    if T == 0:
+        return
+    s = _scratch_for(x.device)
+    _cost(_size(w) + _size(x) + T * (I + P) * 2, 2.0 * T * N * K)
+    parked = flags = None
+    ctas, floats, what = 0, 0, "gemm+glu (tensor cores"
+    if many_tokens(T, N):
+        ctas, bn = SM_COUNT, stream_k_plan(T, N, K)
+        what += ", persistent"
+        if bn is not None:
+            parked, flags, floats = s.parked, s.parked_flags, s.parked.numel()
+            what += ", stream-K"
+        else:
+            bn = persistent_plan(T, N)
+    else:
+        bn, _ = gemm_plan(T, N, K)
+    _check(_lib("mb_gemm_tc").mb_gemm_tc_glu(
+        _ptr(x), _ptr(w), _ptr(out), _c_int(_GLU_MODES[activation]), _c_int(T), _c_int(N), _c_int(K), _c_int(bn), _c_int(ctas), _c_float(factor),
+        _c_int(out.stride(0)), _c_int(P), _ptr(rows), _ptr(parked), ctypes.c_longlong(floats), _ptr(flags), _ptr(s.error), _stream()), what + ")")
+
+
+def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor, workspace=None, activation: str = "silu", factor: float = 1.0) -> None:
+    """``out = act(x Wg^T) * (x Wu^T) * factor`` (``activation`` "silu", "relu" or "gelu_tanh") with ``w_interleaved = interleave_gate_up(Wg, Wu)``: on the
+    tensor cores the activation is applied to the float32 accumulators in the epilogue and the ``[T, 2 I]`` intermediate never
     exists; otherwise the product and the activation run as two kernels."""
     scaled = x if isinstance(x, NormedRows) else None
     if scaled is not None:
         x = scaled.rows
-    _need_cuda(x, w_interleaved, out)
+    _need_cuda(x, w_interleaved)
     T, K = x.shape
     N = w_interleaved.shape[0]
     I = N // 2
@@ -782,7 +828,12 @@ def gemm_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor,
     if not fused:
         tmp = workspace.get("gate_up", (T, N), x.dtype) if workspace is not None else torch.empty(T, N, device=x.device, dtype=x.dtype)
         gemm(scaled if scaled is not None else x, w_interleaved, tmp)
-        swiglu(tmp, out, True, activation)
+        swiglu(tmp, out, True, activation, factor)
+        return
+    if factor != 1.0 or out.stride(0) != I:
+        if scaled is not None:
+            raise KernelError("gemm_swiglu: a factor does not go with rows that have a pending norm")
+        gemm_glu_rows(x, w_interleaved, None, out, activation, factor)
         return
     s = _scratch_for(x.device)
     mode = _GLU_MODES[activation]
@@ -1235,31 +1286,85 @@ VALUE_MODES = {None: 0, "leave": 1, "mix": 2}
 
 def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Optional[str], q_w, k_w, eps: float, positions,
                inv_freq, rot_dim: int, rot_mag: float, slot_mapping, k_cache, v_cache, value_mode: Optional[str], v_shared,
-               v_lambda, H: int, K: int, d: int, dv: int, write_kv: bool = True, interleaved: bool = False) -> None:
+               v_lambda, H: int, K: int, d: int, dv: int, write_kv: bool = True, interleaved: bool = False, maps: int = 1,
+               conv: Optional["ConvRows"] = None, ctx=None) -> None:
     """Finishes the heads of a fused projection whose rows hold q | k | v (| more columns that are left alone): biases, the
     RMS norm of q and k (``norm`` "head": per head with a weight ``[d]``; "whole": over the whole of q, and of k, with weights
     ``[H d]`` / ``[K d]``), the rotation of the first ``rot_dim`` elements of each head (half-split pairs, or neighbours
     ``(2i, 2i + 1)`` if ``interleaved``; sines and cosines times ``rot_mag``), and the values: as they are, also left in ``v_shared`` ("leave"), or mixed with what ``v_shared`` holds,
-    ``(1 - lam) v + lam v_shared`` ("mix").  Queries go to ``q_out``, keys and values into their pages."""
+    ``(1 - lam) v + lam v_shared`` ("mix").  Queries go to ``q_out``, keys and values into their pages.
+
+    ``maps`` > 1: ``H`` and ``K`` count maps (a head's maps side by side), there are ``K / maps`` value heads; a key row of ``maps d`` elements holds
+    its kv head's maps side by side, a query map lies in a row as wide with zeros outside its own part.  ``conv``: a short causal convolution per
+    channel between bias and norm, its rows' state in a ring (``ctx`` is then needed)."""
     _need_cuda(q_out, q_b, k_b, v_b, q_w, k_w, positions, inv_freq, slot_mapping, k_cache, v_cache, v_shared, v_lambda)
     T = rows.shape[0]
     assert rows.is_cuda and rows.stride(1) == 1             # (it may be a column block of a wider product)
-    assert tuple(q_out.shape) == (T, H * d) and q_out.dtype == rows.dtype and rows.shape[1] >= ((H + K) * d + K * dv if write_kv else H * d)
-    assert k_cache.dtype == rows.dtype and v_cache.dtype == rows.dtype and k_cache.shape[3] == d and v_cache.shape[3] == dv
-    assert v_shared is None or (v_shared.dtype == rows.dtype and v_shared.numel() >= T * K * dv)
+    KG = K // maps
+    assert tuple(q_out.shape) == (T, H * d * maps) and q_out.dtype == rows.dtype and rows.shape[1] >= ((H + K) * d + KG * dv if write_kv else H * d)
+    assert k_cache.dtype == rows.dtype and v_cache.dtype == rows.dtype and k_cache.shape[3] == d * maps and v_cache.shape[3] == dv
+    assert k_cache.shape[1] == KG and H % maps == 0 and K % maps == 0
+    assert v_shared is None or (v_shared.dtype == rows.dtype and v_shared.numel() >= T * KG * dv)
     page_size = k_cache.shape[2]
-    _cost(2 * T * ((H + K) * d + K * dv) * rows.element_size(), 10.0 * T * (H + K) * d)
+    _cost(2 * T * ((H + K) * d + KG * dv) * rows.element_size(), 10.0 * T * (H + K) * d)
+    single = 0
+    if conv is not None:
+        channels = (H + K) * d + KG * dv
+        taps = conv.weight.shape[0]
+        _need_cuda(conv.weight, conv.slots)
+        assert write_kv and conv.weight.dtype == torch.float32 and conv.weight.shape[1] == channels
+        assert conv.ring.is_cuda and conv.ring.dtype == torch.float32 and tuple(conv.ring.shape[1:]) == (taps, channels) and conv.ring.is_contiguous()
+        single = ctx.num_decode
+        if launch_log is not None:
+            _pending_cost["bytes"] += ctx.num_decode * taps * channels * 4 + taps * channels * 4
     _check(_lib("mb_attention_sink").mb_qkv_finish(
         _ptr(rows), _c_int(rows.stride(0)), _code(rows), _ptr(q_out), _ptr(q_b), _ptr(k_b), _ptr(v_b), _c_int(NORM_MODES[norm]), _ptr(q_w),
         _ptr(k_w), _c_float(eps), _ptr(positions), _ptr(inv_freq), _c_int(rot_dim if inv_freq is not None else 0), _c_float(rot_mag),
         _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _c_int(VALUE_MODES[value_mode]), _ptr(v_shared), _ptr(v_lambda), _c_int(T),
-        _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_int(int(write_kv)), _c_int(int(interleaved)), _stream()),
-        "q|k|v heads (sink attention)")
+        _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_int(int(write_kv)), _c_int(int(interleaved)), _c_int(maps),
+        *((_ptr(conv.weight), _ptr(conv.ring), _ptr(conv.slots), _ptr(ctx.req_index), _ptr(ctx.cu_tokens), _c_int(taps)) if conv is not None
+          else (None, None, None, None, None, _c_int(0))), _c_int(single), _stream()), "q|k|v heads (sink attention)")
+    if conv is not None and ctx.num_requests > single and taps > 1:
+        _cost((ctx.num_requests - single) * (taps - 1) * channels * (4 + rows.element_size()))
+        _check(_lib("mb_attention_sink").mb_conv_ring(
+            _ptr(rows), _c_int(rows.stride(0)), _code(rows), _ptr(q_b), _ptr(k_b), _ptr(v_b), _ptr(conv.ring), _ptr(conv.slots), _ptr(ctx.cu_tokens),
+            _ptr(positions), _c_int(taps), _c_int(single), _c_int(ctx.num_requests), _c_int(H * d), _c_int(K * d), _c_int(KG * dv), _stream()),
+            "convolution's last rows kept")
+
+
+class ConvRows:
+    """A short convolution over the rows of a projection (``qkv_finish``): ``weight`` float32 ``[taps, channels]``, the last row on the current
+    token; ``ring`` float32 ``[slots, taps, channels]``: the input of position ``p`` in row ``p mod taps``."""
+    __slots__ = ("weight", "ring", "slots")
+
+    def __init__(self, weight: torch.Tensor, ring: torch.Tensor, slots: torch.Tensor):
+        self.weight, self.ring, self.slots = weight, ring, slots
+
+
+class MapPair:
+    """Two maps per head (``attention_sink``): with ``a_1``, ``a_2`` what query heads ``2 h`` and ``2 h + 1`` would give, head ``h``'s result is
+    ``n / sqrt(mean(n^2) + eps) * factor``, ``n = a_1 - lam a_2``."""
+    __slots__ = ("lam", "eps")
+
+    def __init__(self, lam: float, eps: float):
+        self.lam, self.eps = float(lam), float(eps)
+
+
+def pair_combine(parts: torch.Tensor, pair: MapPair, factor: float, out: torch.Tensor, H: int, dv: int, first_token: int = 0) -> None:
+    """The maps' results ``parts`` (float32 ``[T, 2 H dv]``, a head's two side by side) combined into ``out`` ``[T, H dv]`` (rows may be strided)."""
+    _need_cuda(parts)
+    T = out.shape[0]
+    assert parts.dtype == torch.float32 and tuple(parts.shape) == (T, 2 * H * dv) and out.is_cuda and out.stride(1) == 1 and out.shape[1] == H * dv
+    _cost((T - first_token) * H * dv * (8 + out.element_size()))
+    _check(_lib("mb_attention_sink").mb_pair_combine(_ptr(parts), _c_void_p(out.data_ptr()), _c_int(out.stride(0)), _code(out), _c_float(pair.lam),
+                                                    _c_float(pair.eps), _c_float(factor), _c_int(first_token), _c_int(T), _c_int(H), _c_int(dv), _stream()),
+           "attention (two maps combined)")
 
 
 def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d: int, dv: int, scale: float, window: int = 0,
                    chunk: int = 0, sink: bool = True, gate: Optional[torch.Tensor] = None, plan=None,
-                   sink_logits: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0, out_scale: float = 1.0) -> None:
+                   sink_logits: Optional[torch.Tensor] = None, keep_first: int = 0, softcap: float = 0.0, out_scale: float = 1.0,
+                   pair: Optional[MapPair] = None) -> None:
     """Causal softmax attention of the step's tokens over the paged cache.  A position sees the keys before it (its own
     included), of them only the last ``window`` (0: all) and only those of its own chunk of ``chunk`` positions (0: no
     chunks).  ``sink``: ``exp(sink_logits[head])`` is added to the softmax's denominator (float32 ``[H]``, not scaled; None: a
@@ -1267,14 +1372,18 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     multiplied by ``sigmoid(gate)``.  ``v_cache`` may be ``k_cache`` itself: the values are then the first ``dv`` elements
     of the key rows (a latent that keys and values share).  ``keep_first``: the sequence's first positions are seen however
     old they are.  ``softcap`` > 0: scores become ``softcap tanh(s / softcap)`` (the sink's does not).  The result is multiplied
-    by ``out_scale``; ``out`` may be a column block of a wider buffer."""
+    by ``out_scale``; ``out`` may be a column block of a wider buffer.  ``pair``: the ``H`` query heads are pairs of maps whose results are combined
+    (no sink, no gate); ``out`` then has ``H / 2`` heads."""
     _need_cuda(q, k_cache, v_cache, block_table, sink_logits)
     assert out.is_cuda and out.stride(1) == 1
-    more = (_c_int(keep_first), _c_float(softcap), _c_float(out_scale), _c_int(out.stride(0)))
+    maps = 2 if pair is not None else 1
+    if pair is not None and (sink or gate is not None or H % 2 != 0):
+        raise KernelError("attention_sink: pairs of maps go without a sink and a gate")
+    more = (_c_int(keep_first), _c_float(softcap), _c_float(out_scale if pair is None else 1.0), _c_int(out.stride(0)))
     T = q.shape[0]
     page_size = k_cache.shape[2]
     values_in_keys = v_cache.data_ptr() == k_cache.data_ptr()
-    assert tuple(q.shape) == (T, H * d) and tuple(out.shape) == (T, H * dv) and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
+    assert tuple(q.shape) == (T, H * d) and tuple(out.shape) == (T, H // maps * dv) and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype
     assert k_cache.shape[3] == d and (v_cache.shape[3] == dv or (values_in_keys and dv <= d))
     assert sink_logits is None or (sink and sink_logits.dtype == torch.float32 and sink_logits.numel() == H)
     v_stride = d if values_in_keys else dv
@@ -1285,7 +1394,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     if T == 0:
         return
     size = q.element_size()
-    per_row = H * (d + (3 if gate is not None else 2) * dv) * size
+    per_row = H * (d + (3 if gate is not None else 2) * dv) // maps * size
     key_bytes = (d if values_in_keys else K * (d + dv)) * size      # what one cached position holds for this layer
     if use_fast_sink_attention and fast_sink_attention_supported(q.dtype, H, K, d, dv, values_in_keys) and page_size & (page_size - 1) == 0:
         kv_heads = K
@@ -1303,45 +1412,59 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
             acc = ctx.workspace.get("sink_parts", (plan.chunks, nd, H, dv), torch.float32)
             ml = ctx.workspace.get("sink_part_sums", (plan.chunks, nd, H, 2), torch.float32)
             if launch_log is not None:
-                _cost(nd * per_row + 2 * _size(acc), 0.0, key_bytes, 2.0 * H * (d + dv))
+                _cost(nd * per_row + 2 * _size(acc), 0.0, key_bytes, 2.0 * H * (d // maps + dv))
                 _pending_cost["rows"], _pending_cost["window"] = "decode", window
             _check(lib.mb_attn_sink_decode(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(acc), _ptr(ml), _ptr(block_table),
                                            _c_int(max_pages), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(page_size), _c_float(scale),
                                            _c_int(window), _c_int(chunk), _c_int(plan.split), _c_int(plan.chunks), _c_int(keep_first), _c_float(softcap), _stream()),
                    "attention (sink, decode)")
-            _cost(_size(acc) + nd * H * dv * size * (2 if gate is not None else 1))
-            _check(lib.mb_attn_sink_merge(_ptr(acc), _ptr(ml), _ptr(out), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(window),
-                                          _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _c_int(plan.split), _ptr(sink_logits),
-                                          _c_int(keep_first), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink, parts merged)")
+            _cost(_size(acc) + nd * H // maps * dv * size * (2 if gate is not None else 1))
+            if pair is not None:
+                _check(lib.mb_attn_sink_merge_pair(_ptr(acc), _ptr(ml), _c_void_p(out.data_ptr()), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(window),
+                                                   _c_int(chunk), _c_int(plan.split), _c_int(keep_first), _c_float(pair.lam), _c_float(pair.eps),
+                                                   _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink, parts and maps merged)")
+            else:
+                _check(lib.mb_attn_sink_merge(_ptr(acc), _ptr(ml), _ptr(out), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(window),
+                                              _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _c_int(plan.split), _ptr(sink_logits),
+                                              _c_int(keep_first), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink, parts merged)")
         if ctx.num_requests > nd and launch_log is not None:
-            _cost((T - nd) * per_row, 0.0, key_bytes, 2.0 * H * (d + dv))
+            _cost((T - nd) * per_row, 0.0, key_bytes, 2.0 * H * (d // maps + dv))
             _pending_cost["rows"], _pending_cost["window"] = "prefill", window
         if (ctx.num_requests > nd and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
                 and (gate is None or (gate.data_ptr() % 16 == 0 and gate_stride % 8 == 0)) and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0):
-            # heads of 64 or 128 with values as wide: the tcgen05 kernel that plain causal attention uses takes the chunked
+            # heads of 64 or 128: the tcgen05 kernel that plain causal attention uses takes the chunked
             # mask, the kept positions, the cap, the sink and the gate as parameters; over a shared latent one CTA per query head reads the one kv head's rows
             g = H // kv_heads
-            tc = build.load(build.attention_tc_name(d, g, dv, values_in_keys), *build.attention_tc_job(d, g, dv, values_in_keys))
+            tc = build.load(build.attention_tc_name(d, g, dv, values_in_keys, pair is not None), *build.attention_tc_job(d, g, dv, values_in_keys, pair is not None))
             _check(tc.mb_attn_prefill_tc(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
                                          _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
                                          _c_int(ctx.max_query_len), _c_int(T), _c_int(kv_heads), _c_int(page_size),
                                          ctypes.c_longlong(k_cache.shape[0]), _c_float(scale), _c_int(window),
                                          _ptr(_scratch_for(q.device).error), _c_int(chunk), _c_int(int(sink)), _ptr(gate),
-                                         _c_int(gate_stride), _ptr(sink_logits), *more, _stream()), "attention (sink, prefill, tensor cores)")
+                                         _c_int(gate_stride), _ptr(sink_logits), *more[:2], _c_float(out_scale), more[3],
+                                         _c_float(pair.lam if pair is not None else 0.0), _c_float(pair.eps if pair is not None else 0.0), _stream()),
+                   "attention (sink, prefill, tensor cores)")
         elif ctx.num_requests > nd:
+            wide = ctx.workspace.get("map_results", (T, H * dv), torch.float32) if pair is not None else None
             _check(lib.mb_attn_sink_prefill(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
                                             _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
                                             _c_int(ctx.max_query_len), _c_int(K), _c_int(page_size), _c_float(scale), _c_int(window),
-                                            _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _ptr(sink_logits), *more, _stream()),
+                                            _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _ptr(sink_logits), *more, _ptr(wide), _stream()),
                    "attention (sink, prefill)")
+            if pair is not None:
+                pair_combine(wide, pair, out_scale, out, H // 2, dv, nd)      # (requests with one token each come first: token nd is the portions' first)
         return
+    wide = ctx.workspace.get("map_results", (T, H * dv), torch.float32) if pair is not None else None
     if launch_log is not None:
-        _cost(T * per_row, 0.0, key_bytes, 2.0 * H * (d + dv))
+        _cost(T * per_row, 0.0, key_bytes, 2.0 * H * (d // maps + dv))
         _pending_cost["rows"], _pending_cost["window"] = "all", window
     _check(_lib("mb_attention_sink").mb_attention_sink(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _code(q), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(ctx.req_index),
         _ptr(ctx.positions), _c_int(T), _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_float(scale), _c_int(window),
-        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), *more, _stream()), "attention (sink)")
+        _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), *more, _ptr(wide), _stream()),
+        "attention (sink)")
+    if pair is not None:
+        pair_combine(wide, pair, out_scale, out, H // 2, dv)
 
 
 #: bf16 sink attention goes to the tensor-core kernels where the head layout allows (False: always the plain kernel)
@@ -1361,19 +1484,18 @@ def sink_group(H: int, K: int, values_in_keys: bool = False) -> int:
 
 
 def tc_sink_attention_supported(d: int, dv: int, values_in_keys: bool = False) -> bool:
-    """Head layouts the tcgen05 prompt kernel is compiled for: keys and values of 64 or of 128; or values that are the
+    """Head layouts the tcgen05 prompt kernel is compiled for: keys and values of 64 or of 128 each; or values that are the
     first 64 or 128 elements of key rows of 64 to 192 (a multiple of 16)."""
     if values_in_keys:
         return dv in (64, 128) and dv <= d <= 192 and d % 16 == 0
-    return d == dv and d in (64, 128)
+    return d in (64, 128) and dv in (64, 128)
 
 
 def fast_sink_attention_supported(dtype, H: int, K: int, d: int, dv: int, values_in_keys: bool = False) -> bool:
-    """Head sizes in multiples of 16, values up to 128 wide, keys up to 128 (up to 256 where the values are the start of
-    the key rows), at most 16 query heads per kv head (any number of heads over a shared latent)."""
+    """Head sizes in multiples of 16, values up to 128 wide, keys up to 256, at most 16 query heads per kv head (any number of heads over a shared latent)."""
     if values_in_keys and K != 1:
         return False
-    return (dtype == torch.bfloat16 and d % 16 == 0 and dv % 16 == 0 and 16 <= d <= (256 if values_in_keys else 128) and 16 <= dv <= 128
+    return (dtype == torch.bfloat16 and d % 16 == 0 and dv % 16 == 0 and 16 <= d <= 256 and 16 <= dv <= 128
             and H % K == 0 and 1 <= sink_group(H, K, values_in_keys) <= SINK_GROUP_MAX and (not values_in_keys or dv <= d))
 
 
@@ -1389,7 +1511,7 @@ def _sink_lib(d: int, dv: int, group: int, values_in_keys: bool = False):
     return build.load(_sink_name(d, dv, group, values_in_keys), *_sink_job(d, dv, group, values_in_keys))
 
 
-def sink_attention_jobs(dtype, H: int, K: int, d: int, dv: int, values_in_keys: bool = False) -> dict:
+def sink_attention_jobs(dtype, H: int, K: int, d: int, dv: int, values_in_keys: bool = False, pair: bool = False) -> dict:
     """The kernels a sink-attention mixer of this head layout runs: the head preparation and the plain kernel, and the
     tensor-core kernels compiled for the layout where it allows."""
     jobs = library_jobs("mb_attention_sink")
@@ -1397,7 +1519,7 @@ def sink_attention_jobs(dtype, H: int, K: int, d: int, dv: int, values_in_keys: 
         g = sink_group(H, K, values_in_keys)
         jobs[_sink_name(d, dv, g, values_in_keys)] = _sink_job(d, dv, g, values_in_keys)
         if use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys):
-            jobs[build.attention_tc_name(d, H // K, dv, values_in_keys)] = build.attention_tc_job(d, H // K, dv, values_in_keys)
+            jobs[build.attention_tc_name(d, H // K, dv, values_in_keys, pair)] = build.attention_tc_job(d, H // K, dv, values_in_keys, pair)
     return jobs
 
 
@@ -2158,3 +2280,67 @@ def delta_rule_jobs(dtype, d: int, dv: int) -> dict:
     if use_chunked_delta_rule and delta_chunked_supported(dtype, d, dv):
         jobs[f"mb_delta_rule_chunked_d{d}_v{_delta_slice(dv)}"] = _delta_chunked_job(d, dv)
     return jobs
+
+
+# ---- gated linear attention: a decay per key channel and token (csrc/gated_linear.cu, gated_linear_chunked.cu) ------------------------
+class GlaInputs:
+    """What the recurrence reads: ``q``, ``k`` (``[T, heads dim]``), ``v`` and the ``gate`` (``[T, heads vdim]``) and ``low`` (``[T, rank]``), column blocks
+    of one product's rows; ``w2`` ``[heads dim, rank]`` in the activation dtype and ``bias`` float32 ``[heads dim]``, which make the decays' input of
+    ``low``; ``inv_tau``: ``log alpha = -softplus(-z) * inv_tau``."""
+    __slots__ = ("q", "k", "v", "gate", "low", "w2", "bias", "inv_tau")
+
+    def __init__(self, q, k, v, gate, low, w2, bias, inv_tau: float):
+        self.q, self.k, self.v, self.gate, self.low, self.w2, self.bias, self.inv_tau = q, k, v, gate, low, w2, bias, float(inv_tau)
+
+
+def _gla_args(inp: GlaInputs, H: int, d: int, dv: int):
+    """The inputs' pointers, their common row stride and the second matrix, checked."""
+    T, rank = inp.low.shape
+    stride, dtype = inp.q.stride(0), inp.q.dtype
+    _need_cuda(inp.w2, inp.bias)
+    for t, n in ((inp.q, H * d), (inp.k, H * d), (inp.v, H * dv), (inp.low, rank)):
+        assert t.is_cuda and tuple(t.shape) == (T, n) and t.dtype == dtype and (T == 0 or (t.stride(1) == 1 and t.stride(0) == stride))
+    assert inp.gate is None or (tuple(inp.gate.shape) == (T, H * dv) and inp.gate.dtype == dtype and inp.gate.stride(1) == 1)
+    assert tuple(inp.w2.shape) == (H * d, rank) and inp.w2.dtype == dtype and inp.bias.dtype == torch.float32 and inp.bias.numel() == H * d
+    p = lambda t: _c_void_p(t.data_ptr())
+    return (p(inp.q), p(inp.k), p(inp.v), p(inp.low), _c_int(stride), _c_int(_DTYPE_CODE[dtype]), _ptr(inp.w2), _ptr(inp.bias), _c_int(rank),
+            _c_float(inp.inv_tau))
+
+
+def _gla_bytes(inp: GlaInputs, tokens: int, requests: int, H: int, d: int, dv: int) -> float:
+    return tokens * (2 * H * d + H * dv + inp.low.shape[1]) * inp.q.element_size() + _size(inp.w2) + requests * H * d * dv * 8
+
+
+def gla_scan(inp: GlaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, o: torch.Tensor, H: int, d: int, dv: int, first_req: int = 0) -> None:
+    """The recurrence token by token over requests ``first_req`` on: ``o`` float32 ``[T, heads vdim]``, states updated in place."""
+    _need_cuda(state, slots, o)
+    assert o.dtype == torch.float32 and state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, d, dv)
+    tokens = inp.q.shape[0] - first_req
+    _cost(_gla_bytes(inp, tokens, ctx.num_requests - first_req, H, d, dv) + tokens * H * dv * 4, 4.0 * tokens * H * d * dv)
+    _check(_lib("mb_gated_linear").mb_gla_scan(*_gla_args(inp, H, d, dv), _ptr(state), _ptr(ctx.cu_tokens), _ptr(slots), _ptr(o), _c_int(first_req),
+                                              _c_int(ctx.num_requests), _c_int(H), _c_int(d), _c_int(dv), _stream()), "gated linear attention (token by token)")
+
+
+#: requests with one token each go to the kernel that does all of it (False: recurrence and norm as kernels of their own)
+use_gla_single = True
+
+
+def gla_single_supported(d: int, dv: int) -> bool:
+    return 1 <= d <= 256 and 4 <= dv <= 256 and dv % 4 == 0 and (dv // 4) * (16 if d > 128 else 8) <= 512
+
+
+def gla_single(inp: GlaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, gate: str, norm_w: torch.Tensor, eps: float, factor: float, out: torch.Tensor,
+               requests: int, H: int, d: int, dv: int) -> None:
+    """Single tokens of the step's first ``requests`` requests, from the projections' rows to the gated heads in ``out`` (rows may be strided)."""
+    _need_cuda(state, slots, norm_w)
+    assert state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, d, dv) and out.stride(1) == 1 and out.shape[1] == H * dv
+    assert inp.gate.stride(0) == inp.q.stride(0) and norm_w.dtype == torch.float32 and norm_w.numel() == dv
+    _cost(_gla_bytes(inp, requests, requests, H, d, dv) + requests * 2 * H * dv * inp.q.element_size(), 4.0 * requests * H * d * dv)
+    _check(_lib("mb_gated_linear").mb_gla_single(
+        *_gla_args(inp, H, d, dv), _ptr(state), _ptr(ctx.seq_lens), _ptr(slots), _c_void_p(inp.gate.data_ptr()), _c_int(DELTA_GATES[gate]), _ptr(norm_w),
+        _c_float(eps), _c_float(factor), _c_void_p(out.data_ptr()), _c_int(out.stride(0)), _c_int(requests), _c_int(H), _c_int(d), _c_int(dv), _stream()),
+        "gated linear attention (single tokens)")
+
+
+def gla_jobs(dtype, d: int, dv: int) -> dict:
+    return library_jobs("mb_gated_linear", "mb_delta_rule")

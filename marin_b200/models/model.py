@@ -8,6 +8,7 @@ import torch
 
 from ..kernels import ops
 from ..parts.base import Runtime
+from ..parts.embedding import PassEntry
 from ..parts.registry import lookup
 from ..parts.spec import ModelSpec, TensorSpec
 
@@ -19,7 +20,10 @@ class Model:
         self.blocks = [lookup("block", layer.block)(layer) for layer in spec.layers]
         self.final_norm = lookup("norm", spec.final_norm.kind)(**spec.final_norm.params)
         self.head = lookup("head", spec.head.kind)(**spec.head.params)
+        self.pass_entry = PassEntry(spec.pass_vectors) if spec.pass_vectors is not None else None
         for i, entry in enumerate(spec.schedule):
+            if entry.enters is not None and (self.pass_entry is None or spec.streams > 0 or not 0 <= entry.enters < spec.pass_vectors.shape[0]):
+                raise ValueError(f"schedule entry {i} starts pass {entry.enters} of a loop without a vector for it (or over several streams)")
             if not 0 <= entry.layer < len(self.blocks):
                 raise ValueError(f"schedule entry {i} names layer {entry.layer}, the model has {len(self.blocks)}")
             if entry.cache_of is not None:
@@ -29,6 +33,8 @@ class Model:
 
     def tensor_specs(self) -> List[TensorSpec]:
         specs = list(self.embedding.tensor_specs())
+        if self.pass_entry is not None:
+            specs += self.pass_entry.tensor_specs()
         for block in self.blocks:
             specs += block.tensor_specs()
         specs += self.final_norm.tensor_specs()
@@ -51,7 +57,7 @@ class Model:
     # ---- what the code around the model asks of it: every answer is the sum of the parts' own answers ----------------
     def parts(self) -> List[object]:
         """Every part of the model once: embedding, the blocks' parts in layer order, final norm, head."""
-        out = [self.embedding]
+        out = [self.embedding] + ([self.pass_entry] if self.pass_entry is not None else [])
         for block in self.blocks:
             out += block.parts() if hasattr(block, "parts") else [block]
         return out + [self.final_norm, self.head]
@@ -113,6 +119,8 @@ class Model:
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.rt = rt
         self.embedding.load(tensors, rt)
+        if self.pass_entry is not None:
+            self.pass_entry.load(tensors, rt)
         for block in self.blocks:
             block.load(tensors, rt)
         self.final_norm.load(tensors, rt)
@@ -147,12 +155,17 @@ class Model:
             self.embedding.forward(ctx.token_ids, hidden, ctx.positions, **extra)
         if observe is not None:
             observe(0, hidden)
+        kept = self.pass_entry.keep(hidden, ctx) if self.pass_entry is not None else None
         carried = None            # the next block's first norm, if the block before could carry it on its last product
         schedule = self.spec.schedule
         for i, entry in enumerate(schedule):
             block = self.blocks[entry.layer]
+            if entry.enters is not None:
+                ops.stage_name = "pass entered"
+                self.pass_entry.forward(hidden, entry.enters, kept)
             if getattr(block, "chains_norm", False):
-                following = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) else None
+                # (the norm of a run that starts a pass cannot ride on the run before: the stream changes in between)
+                following = self.blocks[schedule[i + 1].layer] if i + 1 < len(schedule) and schedule[i + 1].enters is None else None
                 carried = block.forward(hidden, ctx, caches.view(i, ctx), x_in=carried, next_block=following)
             else:
                 block.forward(hidden, ctx, caches.view(i, ctx))

@@ -279,3 +279,56 @@ class PostNormBlock(Part):
         else:
             self._join(0, y, hidden, rows if goes_on and not wide else None)
         return rows if goes_on else None
+
+
+@register_block("parallel_prenorm")
+class ParallelBlock(Part):
+    """``x <- x + m (mixer(h) + feedforward(h))`` with one norm, ``h = norm1(x)``, that both sublayers read (a layer without a feed-forward has the mixer
+    alone).  ``block_params["residual_mult"]``: ``m`` (1 without it); mixer and feed-forward take it as their ``out_scale``, so that it multiplies
+    float32 numbers before they are rounded.  A row the mixer adds to every token (``Mixer.row_bias``) rides on the norm's kernel."""
+
+    def __init__(self, spec: LayerSpec):
+        names = spec.names
+        m = float(spec.block_params.get("residual_mult", 1.0))
+        scale = {} if m == 1.0 else {"out_scale": m}
+        self.norm1 = lookup("norm", spec.norm.kind)(name=f"{spec.prefix}.{names['norm1']}", **spec.norm.params)
+        if not (hasattr(self.norm1, "weight") and hasattr(self.norm1, "unit_offset")):
+            raise ValueError("parallel_prenorm: the norm has to be an RMS norm")
+        self.mixer = lookup("mixer", spec.mixer.kind)(name=f"{spec.prefix}.{names['mixer']}", **{**spec.mixer.params, **scale})
+        self.feedforward = None
+        if spec.feedforward is not None:
+            self.feedforward = lookup("feedforward", spec.feedforward.kind)(name=f"{spec.prefix}.{names['feedforward']}", **{**spec.feedforward.params, **scale})
+
+    def parts(self) -> List[Part]:
+        return [p for p in (self.norm1, self.mixer, self.feedforward) if p is not None]
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [s for p in self.parts() for s in p.tensor_specs()]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        for p in self.parts():
+            p.load(tensors, rt)
+        self.mixer.adds_row_bias = False
+        self.rt = rt
+
+    def weight_bytes(self, dtype) -> int:
+        return sum(p.weight_bytes(dtype) for p in self.parts())
+
+    def bytes_read(self, tokens: int, dtype) -> int:
+        return sum(p.bytes_read(tokens, dtype) for p in self.parts())
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return sum(p.flops(tokens, pairs) for p in self.parts())
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        jobs: Dict[str, tuple] = {}
+        for p in self.parts():
+            jobs.update(p.kernel_jobs(dtype))
+        return jobs
+
+    def forward(self, hidden: torch.Tensor, ctx, cache):
+        ops.stage_name = "norm"
+        x = self.norm1.forward(hidden, ctx.workspace.get("normed", tuple(hidden.shape), self.rt.dtype), self.mixer.row_bias)
+        self.mixer.forward(x, ctx, cache, hidden)
+        if self.feedforward is not None:
+            self.feedforward.forward(x, ctx, hidden)

@@ -78,6 +78,37 @@ class TokenEmbedding(Part):
         return out
 
 
+class PassEntry(Part):
+    """What enters the residual stream where a loop's passes start: row ``n`` of a learned tensor ``[passes, hidden]`` before pass ``n``, and before it, in
+    every pass but the first, the embedding's output (``keep`` makes the copy that is added)."""
+
+    def __init__(self, spec: TensorSpec):
+        self.spec = spec
+        self.vectors: Optional[torch.Tensor] = None
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        return [self.spec]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        self.vectors = rt.f32(tensors.pop(self.spec.name))
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return 0.0
+
+    def workspace_per_token(self, dtype) -> int:
+        return 4 * self.spec.shape[1] if self.spec.shape[0] > 1 else 0
+
+    def keep(self, hidden: torch.Tensor, ctx) -> Optional[torch.Tensor]:
+        if self.spec.shape[0] < 2:
+            return None
+        kept = ctx.workspace.get("embedding_output", tuple(hidden.shape), torch.float32)
+        ops.stream_enter(hidden, None, None, kept)
+        return kept
+
+    def forward(self, hidden: torch.Tensor, index: int, kept: Optional[torch.Tensor]) -> None:
+        ops.stream_enter(hidden, kept if index > 0 else None, self.vectors[index], hidden)
+
+
 @register_head("linear")
 class LinearHead(Part):
     """``logits = rows W^T`` in float32; ``tied_to`` names the embedding whose table is the

@@ -31,10 +31,12 @@ class FeedForward(Part):
 @register_feedforward("swiglu")
 class SwiGLU(FeedForward):
     """``down( g / (1 + exp(-g)) * u )`` with ``g = x W_gate^T`` and ``u = x W_up^T``, no bias
-    (crates/model/src/qwen3/mlp.rs:22-37, crates/tensor/src/silu.rs:18).  ``activation`` "relu": ``down( max(g, 0) * u )``."""
+    (crates/model/src/qwen3/mlp.rs:22-37, crates/tensor/src/silu.rs:18).  ``activation`` "relu": ``down( max(g, 0) * u )``; "gelu_tanh":
+    the tanh form of gelu.  ``out_scale``: the result times a number (applied before ``down``, which is linear)."""
 
     def __init__(self, hidden: int, intermediate: int, name: str, activation: str = "silu",
-                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight")):
+                 names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), out_scale: float = 1.0):
+        self.out_scale = float(out_scale)
         self.hidden, self.intermediate, self.name, self.activation = int(hidden), int(intermediate), name, activation
         if activation not in ops.GLU_ACTIVATIONS:
             raise ValueError(f"swiglu: unknown activation {activation!r}")
@@ -57,7 +59,9 @@ class SwiGLU(FeedForward):
             self.w_gate_up = rt.matrix(torch.cat([gate, up], dim=0))
         self.w_down = rt.matrix(tensors.pop(self.down_name))
 
-    couples_norm = True
+    @property
+    def couples_norm(self) -> bool:
+        return self.out_scale == 1.0
 
     def forward(self, x, ctx, residual: torch.Tensor, then_norm=None):
         T = x.shape[0]
@@ -65,11 +69,11 @@ class SwiGLU(FeedForward):
         act = ws.get("ffn_act", (T, self.intermediate), x.dtype)
         ops.stage_name = "gate|up, SwiGLU" if self.activation == "silu" else f"gate|up, {self.activation}"
         if self.fused:
-            ops.gemm_swiglu(x, self.w_gate_up, act, ws, self.activation)
+            ops.gemm_swiglu(x, self.w_gate_up, act, ws, self.activation, self.out_scale)
         else:
             gate_up = ws.get("gate_up", (T, 2 * self.intermediate), x.dtype)
             ops.gemm(x, self.w_gate_up, gate_up)
-            ops.swiglu(gate_up, act, activation=self.activation)
+            ops.swiglu(gate_up, act, activation=self.activation, factor=self.out_scale)
         ops.stage_name = "down"
         return ops.gemm(act, self.w_down, residual, accumulate=True, then_norm=then_norm)
 

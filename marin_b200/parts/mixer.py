@@ -112,6 +112,11 @@ class Mixer(Part):
     #: that mixers side by side can share both products.
     joins_products = False
 
+    #: a vector (float32 ``[hidden]``, after ``load``) that the mixer adds to every row of the residual: the output projection's bias, times whatever
+    #: multiplies the result.  A block whose norm adds it to the rows (``RMSNorm.forward(then_add=)``) sets ``adds_row_bias`` to False.
+    row_bias: Optional[torch.Tensor] = None
+    adds_row_bias = True
+
     def cache_need(self):
         return None
 
@@ -364,18 +369,37 @@ class SinkAttention(Mixer):
     ``keep_first`` (with ``window``): the sequence's first positions are seen however old they are, at their true positions; their
     pages are never given back.  ``softcap``: scores become ``softcap tanh(s / softcap)``, the sink's does not.  ``out_scale``: the
     result times a number (applied to the heads' outputs, the output projection being linear).
+
+    ``taps``: a causal convolution per channel of q, k and v between the projection (with its bias) and norm and rotation (weights ``[channels,
+    taps]``, the last column on the current token; no activation); the last inputs of each channel are a state beside the pages.
+    ``out_bias``: the output projection has a bias.
+
+    ``differential`` (a number, ``diff``): differential attention (Ye, Dong, Xia, Sun, Zhu, Huang, Wei, "Differential Transformer"): every head has
+    two maps, attentions of their own over the same values (q has ``heads * 2 * head_dim`` rows, k ``kv_heads * 2 * head_dim``, head by head map 1, map
+    2; norm and rotation per map).  ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` (vectors of ``head_dim``),
+    ``o = a_1 - lambda a_2``, divided by its root mean square over the head's values, times ``1 - diff``.  A page row holds a kv head's two
+    keys side by side and its values once; the maps are query heads that are zero in the other map's half, so they run as ``2 heads`` query heads of
+    ``2 head_dim`` over ``kv_heads`` kv heads, and every row of keys and values is fetched once for both.
     """
 
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight", "g": "g_proj.weight",
              "q_bias": "q_proj.bias", "k_bias": "k_proj.bias", "v_bias": "v_proj.bias",
-             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "lam": "value_mix", "sink": "sink"}
+             "q_norm": "q_norm.weight", "k_norm": "k_norm.weight", "lam": "value_mix", "sink": "sink", "o_bias": "o_proj.bias",
+             "q_conv": "q_conv.weight", "k_conv": "k_conv.weight", "v_conv": "v_conv.weight", "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2"}
 
     def __init__(self, hidden: int, heads: int, kv_heads: int, head_dim: int, name: str, position: PartSpec,
                  v_head_dim: Optional[int] = None, scale: Optional[float] = None, bias: bool = False, qk_norm: Optional[str] = "head",
                  norm_eps: float = 1e-6, window: Optional[int] = None, chunk: Optional[int] = None, sink: bool = True,
                  value_mix: Optional[str] = None, first_of_mix: bool = False, gate: bool = False, names=None, keep_first: int = 0,
-                 softcap: Optional[float] = None, out_scale: float = 1.0):
+                 softcap: Optional[float] = None, out_scale: float = 1.0, taps: Optional[int] = None, out_bias: bool = False,
+                 differential: Optional[float] = None):
         self.hidden, self.heads, self.kv_heads, self.head_dim = int(hidden), int(heads), int(kv_heads), int(head_dim)
+        self.taps, self.out_bias = int(taps) if taps else None, bool(out_bias)
+        self.diff, self.maps = (float(differential), 2) if differential is not None else (None, 1)
+        if self.maps > 1 and (sink or gate or value_mix is not None or qk_norm == "whole"):
+            raise ValueError("sink_attention: differential attention goes without a sink, a gate, mixed values and a norm over the whole projection")
+        if self.taps is not None and self.taps > 64:
+            raise ValueError("sink_attention: more than 64 taps are not supported")
         if self.heads % self.kv_heads != 0:
             raise ValueError(f"{heads} heads cannot share {kv_heads} kv heads evenly")
         if qk_norm not in (None, "head", "whole"):
@@ -393,9 +417,10 @@ class SinkAttention(Mixer):
         self.value_mix, self.first_of_mix = value_mix, bool(first_of_mix)
         self.position = lookup("position", position.kind)(**position.params)
         self.names = dict(self.NAMES, **(names or {}))
-        self.q_dim, self.k_dim = self.heads * self.head_dim, self.kv_heads * self.head_dim
+        self.q_dim, self.k_dim = self.heads * self.maps * self.head_dim, self.kv_heads * self.maps * self.head_dim
         self.v_dim, self.o_dim = self.kv_heads * self.v_head_dim, self.heads * self.v_head_dim
-        self.w_in = self.w_o = self.q_weight = self.k_weight = self.q_b = self.k_b = self.v_b = self.lam = None
+        self.row_dim = self.maps * self.head_dim                # a key row's width
+        self.w_in = self.w_o = self.q_weight = self.k_weight = self.q_b = self.k_b = self.v_b = self.lam = self.conv_w = self.pair = None
 
     def _n(self, key: str) -> str:
         return f"{self.name}.{self.names[key]}"
@@ -403,7 +428,10 @@ class SinkAttention(Mixer):
     def cache_need(self):
         # (a chunked mask never looks behind its chunk's start, but pages are not given back there: the keys a window
         # has passed are dropped by the cache manager, a chunk's are only skipped)
-        return PagedKV(self.kv_heads, self.head_dim, self.window, self.v_head_dim, keep_first=self.keep_first)
+        pages = PagedKV(self.kv_heads, self.row_dim, self.window, self.v_head_dim, keep_first=self.keep_first)
+        if self.taps is None:
+            return pages
+        return (pages, StateNeed((self.taps, self.q_dim + self.k_dim + self.v_dim), torch.float32))
 
     def tensor_specs(self) -> List[TensorSpec]:
         h = self.hidden
@@ -422,6 +450,12 @@ class SinkAttention(Mixer):
             specs.append(TensorSpec(self._n("lam"), (), "bias", 0.5))
         if self.learned_sink:
             specs.append(TensorSpec(self._n("sink"), (self.heads,), "bias"))
+        if self.taps is not None:
+            specs += [TensorSpec(self._n(f"{p}_conv"), (n, self.taps), "bias", 1.0 / self.taps) for p, n in (("q", self.q_dim), ("k", self.k_dim), ("v", self.v_dim))]
+        if self.out_bias:
+            specs.append(TensorSpec(self._n("o_bias"), (h,), "bias"))
+        if self.maps > 1:
+            specs += [TensorSpec(self._n(k), (self.head_dim,), "bias") for k in ("lq1", "lk1", "lq2", "lk2")]
         return specs
 
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
@@ -439,25 +473,44 @@ class SinkAttention(Mixer):
             self.lam = rt.f32(tensors.pop(self._n("lam"))).reshape(1)
         if self.learned_sink:
             self.sink_logits = rt.f32(tensors.pop(self._n("sink")))
+        if self.taps is not None:
+            self.conv_w = rt.f32(torch.cat([tensors.pop(self._n(f"{p}_conv")).to(torch.float32) for p in "qkv"], dim=0).t())      # [taps, channels]
+        if self.out_bias:
+            self.row_bias = rt.f32(tensors.pop(self._n("o_bias"))) * self.out_scale
+        if self.maps > 1:
+            lq1, lk1, lq2, lk2 = (tensors.pop(self._n(k)).to("cpu", torch.float64) for k in ("lq1", "lk1", "lq2", "lk2"))
+            lam = math.exp(float((lq1 * lk1).sum())) - math.exp(float((lq2 * lk2).sum())) + self.diff
+            self.pair = ops.MapPair(lam, self.norm_eps)
         self.position.load(tensors, rt)
         self.rt = rt
 
     def flops(self, tokens: int, pairs: int = 0) -> float:
         w = self.window + self.keep_first if self.window else 0
+        if self.chunk and not w:
+            c = self.chunk
+            if tokens > 1 and pairs == tokens * (tokens + 1) // 2:
+                pairs = tokens // c * (c * (c + 1) // 2) + tokens % c * (tokens % c + 1) // 2
+            else:
+                pairs = min(pairs, tokens * c)
         if w and tokens > w and pairs == tokens * (tokens + 1) // 2:
             pairs = w * (w + 1) // 2 + (tokens - w) * w          # one prompt from its first position: the window's pairs
         elif w:
             pairs = min(pairs, tokens * w)
-        return super().flops(tokens, pairs) + 2.0 * pairs * self.heads * (self.head_dim + self.v_head_dim)
+        return super().flops(tokens, pairs) + 2.0 * pairs * self.heads * self.maps * (self.head_dim + self.v_head_dim)
 
     def kernel_jobs(self, dtype) -> Dict[str, tuple]:
-        return ops.sink_attention_jobs(dtype, self.heads, self.kv_heads, self.head_dim, self.v_head_dim)
+        return ops.sink_attention_jobs(dtype, self.heads * self.maps, self.kv_heads, self.row_dim, self.v_head_dim, pair=self.maps > 1)
+
+    def workspace_per_token(self, dtype) -> int:
+        """Bytes a step keeps per token beside the products' rows: with two maps, the padded queries and (where one kernel does not combine
+        them) both maps' float32 results."""
+        return 2 * self.q_dim * element_size(dtype) + 4 * self.maps * self.o_dim if self.maps > 1 else 0
 
     def decode_plan_key(self):
-        return ("sink_attention", self.heads, self.kv_heads, self.head_dim, self.v_head_dim, self.chunk, self.window, self.keep_first)
+        return ("sink_attention", self.heads * self.maps, self.kv_heads, self.row_dim, self.v_head_dim, self.chunk, self.window, self.keep_first)
 
     def decode_plan(self, requests: int, span: int, rt: Runtime):
-        return ops.sink_decode_plan(rt.dtype, requests, self.heads, self.kv_heads, self.head_dim, self.v_head_dim, span,
+        return ops.sink_decode_plan(rt.dtype, requests, self.heads * self.maps, self.kv_heads, self.row_dim, self.v_head_dim, span,
                                     self.window or 0, self.chunk or 0, keep_first=self.keep_first)
 
     joins_products = True
@@ -465,6 +518,12 @@ class SinkAttention(Mixer):
     def forward(self, x, ctx, cache, residual: torch.Tensor, rows=None, out=None):
         T = x.shape[0]
         ws = ctx.workspace
+        conv = None
+        if self.taps is not None:
+            cache, ring = cache
+            if not (cache.owner and ring.owner):
+                raise ValueError("sink_attention: a layer behind a convolution cannot read another run's cache")
+            conv = ops.ConvRows(self.conv_w, ring.state, ring.slots)
         writes = cache.owner
         if not writes and self.gate:
             raise ValueError("sink_attention: a gated layer cannot read another run's cache")   # its columns lie behind k and v
@@ -474,7 +533,8 @@ class SinkAttention(Mixer):
             rows = ws.get("qkvg", (T, w.shape[0]), x.dtype)
             ops.gemm(x, w, rows)
         ops.stage_name = "heads"
-        q = ws.get("q", (T, self.q_dim), x.dtype)
+        H, maps = self.heads * self.maps, self.maps
+        q = ws.get("q", (T, H * self.row_dim), x.dtype)
         shared = None
         mode = None
         if self.value_mix is not None and writes:
@@ -484,21 +544,23 @@ class SinkAttention(Mixer):
         pos = self.position
         ops.qkv_finish(rows, q, self.q_b, self.k_b, self.v_b, self.qk_norm, self.q_weight, self.k_weight, self.norm_eps, ctx.positions,
                        pos.inv_freq, pos.rotary_dim, pos.magnitude, cache.slot_mapping, cache.k, cache.v, mode, shared, self.lam,
-                       self.heads, self.kv_heads, self.head_dim, self.v_head_dim, writes, pos.interleaved)
+                       H, self.kv_heads * maps, self.head_dim, self.v_head_dim, writes, pos.interleaved, maps, conv, ctx)
         joined = out is not None
         if not joined:
             out = ws.get("attn_out", (T, self.o_dim), x.dtype)
         ops.stage_name = "attention"
         gate = rows[:, self.q_dim + self.k_dim + self.v_dim:] if self.gate else None
         plans = ctx.decode_plans
-        ops.attention_sink(q, cache.k, cache.v, out, ctx, cache.block_table, self.heads, self.kv_heads, self.head_dim, self.v_head_dim,
+        ops.attention_sink(q, cache.k, cache.v, out, ctx, cache.block_table, H, self.kv_heads, self.row_dim, self.v_head_dim,
                            self.scale, self.window or 0, self.chunk or 0, self.sink, gate,
                            plans.get(self.decode_plan_key()) if plans else None, self.sink_logits, self.keep_first, self.softcap or 0.0,
-                           self.out_scale)
+                           self.out_scale * (1.0 - self.diff) if self.pair is not None else self.out_scale, self.pair)
         if joined:
             return None
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
+        if self.row_bias is not None and self.adds_row_bias:
+            ops.add_row_bias(residual, self.row_bias)
         return None
 
 
@@ -846,12 +908,15 @@ class ParallelMixers(Mixer):
     steps is kept side by side: ``cache_need`` answers the tuple of their needs, the view is the tuple of their views.
 
     Where all of them allow it (``Mixer.joins_products``) their first products are one product of the input and, where their
-    results' widths are multiples of 8, their last ones one product of the results side by side."""
+    results' widths are multiples of 8, their last ones one product of the results side by side; with both, they are to whatever is around
+    them one mixer that allows it too.  ``out_scale`` multiplies the sum."""
 
-    def __init__(self, hidden: int, inner: Dict[str, PartSpec], name: str, scales: Optional[Dict[str, float]] = None):
+    def __init__(self, hidden: int, inner: Dict[str, PartSpec], name: str, scales: Optional[Dict[str, float]] = None, out_scale: float = 1.0):
         self.hidden, self.name = int(hidden), name
         scales = scales or {}
-        self.inner = [lookup("mixer", spec.kind)(name=f"{name}.{key}", out_scale=float(scales.get(key, 1.0)), **spec.params) for key, spec in inner.items()]
+        self.inner = [lookup("mixer", spec.kind)(name=f"{name}.{key}", out_scale=float(out_scale) * float(scales.get(key, 1.0)), **spec.params)
+                      for key, spec in inner.items()]
+        self.o_dim = sum(getattr(m, "o_dim", 0) for m in self.inner)
         self.capturable = all(getattr(m, "capturable", True) for m in self.inner)
         windows = {getattr(m, "window", None) for m in self.inner} - {None}
         self.window = windows.pop() if len(windows) == 1 else None
@@ -866,6 +931,11 @@ class ParallelMixers(Mixer):
         for m in self.inner:
             m.load(tensors, rt)
         self.w_in = self.w_o = None
+        biases = [m.row_bias for m in self.inner if m.row_bias is not None]
+        if biases:
+            self.row_bias = torch.stack(biases).sum(dim=0)
+            for m in self.inner:
+                m.adds_row_bias = False
         if all(m.joins_products for m in self.inner):
             # one matrix each; the inner mixers keep views of their blocks of the first (blocks start at multiples of 8 rows, so that
             # every kernel can take them by 16-byte loads)
@@ -882,6 +952,7 @@ class ParallelMixers(Mixer):
                 self.w_o = torch.cat([m.w_o for m in self.inner], dim=1).contiguous()
                 for m in self.inner:
                     m.w_o = None
+                self.joins_products = True
         self.rt = rt
 
     def bytes_read(self, tokens: int, dtype) -> int:
@@ -913,7 +984,7 @@ class ParallelMixers(Mixer):
                 plans[key] = plan
         return plans or None
 
-    def forward(self, x, ctx, cache, residual: torch.Tensor):
+    def forward(self, x, ctx, cache, residual: torch.Tensor, rows=None, out=None):
         own = ctx.decode_plans.get(self.decode_plan_key()) if ctx.decode_plans else None
         outer = ctx.decode_plans
         if own:
@@ -924,16 +995,21 @@ class ParallelMixers(Mixer):
         else:
             if not all(view.owner for view in _leaves(cache)):
                 raise ValueError("parallel_mixers: mixers that share their products cannot read another run's cache")
-            ops.stage_name = "inputs of both"
-            rows = ctx.workspace.get("joined_rows", (x.shape[0], self.w_in.shape[0]), x.dtype)
-            ops.gemm(x, self.w_in, rows)
-            outs = ctx.workspace.get("joined_out", (x.shape[0], self.w_o.shape[1]), x.dtype) if self.w_o is not None else None
+            if rows is None:
+                ops.stage_name = "inputs of both"
+                rows = ctx.workspace.get("joined_rows", (x.shape[0], self.w_in.shape[0]), x.dtype)
+                ops.gemm(x, self.w_in, rows)
+            outs = out
+            if outs is None and self.w_o is not None:
+                outs = ctx.workspace.get("joined_out", (x.shape[0], self.w_o.shape[1]), x.dtype)
             at = 0
             for m, view, (first, n) in zip(self.inner, cache, self.cols):
                 m.forward(x, ctx, view, residual, rows=rows[:, first:first + n], out=outs[:, at:at + m.o_dim] if outs is not None else None)
                 at += m.o_dim
-            if outs is not None:
+            if outs is not None and out is None:
                 ops.stage_name = "o"
                 ops.gemm(outs, self.w_o, residual, accumulate=True)
+        if self.row_bias is not None and self.adds_row_bias:
+            ops.add_row_bias(residual, self.row_bias)
         ctx.decode_plans = outer
         return None

@@ -1,7 +1,7 @@
 """Normalisation parts."""
 from __future__ import annotations
 
-from typing import Dict, List
+from typing import Dict, List, Optional
 
 import torch
 
@@ -32,9 +32,10 @@ class RMSNorm(Part):
     def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
         self.weight = rt.f32(tensors.pop(self.weight_name))
 
-    def forward(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-        """``x`` float32 ``[rows, dim]`` → ``out`` (float32 or bfloat16) ``[rows, dim]``."""
-        ops.rmsnorm(x, self.weight, self.eps, out, self.unit_offset)
+    def forward(self, x: torch.Tensor, out: torch.Tensor, then_add: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``x`` float32 ``[rows, dim]`` → ``out`` (float32 or bfloat16) ``[rows, dim]``; ``then_add`` (float32 ``[dim]``) is added to ``x`` itself
+        once its norm is taken."""
+        ops.rmsnorm(x, self.weight, self.eps, out, self.unit_offset, then_add)
         return out
 
     def coupling(self, out: torch.Tensor) -> "ops.NormOut":

@@ -413,3 +413,99 @@ class DeltaRule(Mixer):
         ops.stage_name = "o"
         ops.gemm(out, self.w_o, residual, accumulate=True)
         return None
+
+
+@register_mixer("gated_linear_attention")
+class GatedLinearAttention(Mixer):
+    """Gated linear attention (Yang, Wang, Shen, Panda, Kim, "Gated Linear Attention Transformers with Hardware-Efficient Training").
+
+    ``q = W_q x dim^(-1/2)``, ``k = W_k x`` (``heads`` x ``dim``), ``v = W_v x`` (``heads`` x ``vdim``); per head
+    ``S <- diag(alpha) S + k v^T``, ``o = S^T q`` (``S`` ``dim`` x ``vdim``, float32, zero at first) with a decay per key channel,
+    ``alpha = sigmoid(z)^(1 / tau)``, ``z = W_a2 (W_a1 x) + bias`` (``decay_rank`` numbers between).  Each head's ``o`` is divided by its root mean square
+    over ``vdim`` (``norm_eps`` under the root), times a weight ``[vdim]``, times ``gate`` ("silu" or "sigmoid") of ``W_g x``; then ``out_scale`` and ``W_o``
+    into the residual."""
+
+    NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "a1": "a1", "a2": "a2", "a_bias": "a2.b", "norm": "norm", "o": "o"}
+
+    def __init__(self, hidden: int, heads: int, dim: int, vdim: int, tau: float, decay_rank: int, name: str, gate: str = "silu", norm_eps: float = 1e-6,
+                 names=None, out_scale: float = 1.0):
+        self.hidden, self.heads, self.dim, self.vdim, self.rank = (int(v) for v in (hidden, heads, dim, vdim, decay_rank))
+        self.name, self.gate, self.tau, self.norm_eps, self.out_scale = name, gate, float(tau), float(norm_eps), float(out_scale)
+        if gate not in ops.DELTA_GATES or not self.tau > 0:
+            raise ValueError(f"gated_linear_attention: gate {gate!r}, tau {tau}")
+        if self.dim > 256 or self.rank > 512:
+            raise ValueError("gated_linear_attention: key heads above 256 or a decay rank above 512 are not supported")
+        self.names = dict(self.NAMES, **(names or {}))
+        self.qk, self.hv = self.heads * self.dim, self.heads * self.vdim
+        self.o_dim = self.hv
+        self.w_in = self.w_2 = self.a_bias = self.norm_w = self.w_o = None
+
+    def _n(self, key: str) -> str:
+        return f"{self.name}.{self.names[key]}"
+
+    def cache_need(self):
+        return StateNeed((self.heads, self.dim, self.vdim), torch.float32)
+
+    def tensor_specs(self) -> List[TensorSpec]:
+        h = self.hidden
+        return [TensorSpec(self._n("q"), (self.qk, h)), TensorSpec(self._n("k"), (self.qk, h)), TensorSpec(self._n("v"), (self.hv, h)),
+                TensorSpec(self._n("g"), (self.hv, h)), TensorSpec(self._n("a1"), (self.rank, h)), TensorSpec(self._n("a2"), (self.qk, self.rank)),
+                TensorSpec(self._n("a_bias"), (self.qk,), "bias"), TensorSpec(self._n("norm"), (self.vdim,), "norm"), TensorSpec(self._n("o"), (h, self.hv))]
+
+    def load(self, tensors: Dict[str, torch.Tensor], rt: Runtime) -> None:
+        # One product of the layer's input: q | k | v | g | what the decays are made of, in blocks padded to multiples of 8 columns (every kernel
+        # can take them by 16-byte loads).  The decays' second matrix is applied inside the recurrence's kernels, in steps of 16 numbers.
+        blocks = {p: tensors.pop(self._n(p)) for p in "qkvg"}
+        first, second = tensors.pop(self._n("a1")), tensors.pop(self._n("a2"))
+        pad = -self.rank % 16
+        blocks["low"] = torch.cat([first, first.new_zeros(pad, first.shape[1])], dim=0)
+        self.w_2 = rt.matrix(torch.cat([second, second.new_zeros(second.shape[0], pad)], dim=1))
+        self.cols, at, rows = {}, 0, []
+        for key, w in blocks.items():
+            self.cols[key] = (at, w.shape[0])
+            rows += [w, w.new_zeros(-w.shape[0] % 8, w.shape[1])]
+            at += w.shape[0] + -w.shape[0] % 8
+        self.w_in = rt.matrix(torch.cat(rows, dim=0))
+        self.a_bias, self.norm_w = rt.f32(tensors.pop(self._n("a_bias"))), rt.f32(tensors.pop(self._n("norm")))
+        self.w_o = rt.matrix(tensors.pop(self._n("o")))
+        self.rt = rt
+
+    def flops(self, tokens: int, pairs: int = 0) -> float:
+        return super().flops(tokens, pairs) + 4.0 * tokens * self.heads * self.dim * self.vdim
+
+    def kernel_jobs(self, dtype) -> Dict[str, tuple]:
+        return ops.gla_jobs(dtype, self.dim, self.vdim)
+
+    def workspace_per_token(self, dtype) -> int:
+        """Bytes a step keeps per token beside the products' rows: the heads' sums, and what the chunked kernels hand over."""
+        return 4 * self.hv
+
+    joins_products = True
+
+    def forward(self, x, ctx, cache, residual: torch.Tensor, rows=None, out=None):
+        T = x.shape[0]
+        ws = ctx.workspace
+        H, d, dv = self.heads, self.dim, self.vdim
+        if rows is None:
+            ops.stage_name = "q|k|v|g"
+            rows = ws.get("gla_rows", (T, self.w_in.shape[0]), x.dtype)
+            ops.gemm(x, self.w_in, rows)
+        block = lambda key: rows[:, self.cols[key][0]:self.cols[key][0] + self.cols[key][1]]
+        inputs = ops.GlaInputs(block("q"), block("k"), block("v"), block("g"), block("low"), self.w_2, self.a_bias, 1.0 / self.tau)
+        joined = out is not None
+        if not joined:
+            out = ws.get("gla_out", (T, self.hv), x.dtype)
+        ops.stage_name = "gated linear attention"
+        single = ctx.num_decode if ops.use_gla_single and ops.gla_single_supported(d, dv) else 0
+        if single:                                             # requests with one token each come first in the batch
+            ops.gla_single(inputs, cache.state, ctx, cache.slots, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, single, H, d, dv)
+        if ctx.num_requests > single:
+            o = ws.get("gla_o", (T, self.hv), torch.float32)
+            ops.gla_scan(inputs, cache.state, ctx, cache.slots, o, H, d, dv, single)
+            ops.stage_name = "norm, gate"
+            ops.delta_norm(o, inputs.gate, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, H, dv, single)
+        if joined:
+            return None
+        ops.stage_name = "o"
+        ops.gemm(out, self.w_o, residual, accumulate=True)
+        return None

@@ -57,10 +57,12 @@ class LayerSpec:
 @dataclass
 class ScheduleEntry:
     """One run of a layer.  ``cache_of`` names an earlier entry whose cache this run reads
-    instead of keeping one of its own (it then writes nothing)."""
+    instead of keeping one of its own (it then writes nothing).  ``enters``: this run starts pass ``enters`` of a loop: the pass's row of
+    ``ModelSpec.pass_vectors`` is added to the stream right before it, and before that, in every pass but the first, the embedding's output."""
 
     layer: int
     cache_of: Optional[int] = None
+    enters: Optional[int] = None
 
 
 @dataclass
@@ -77,3 +79,5 @@ class ModelSpec:
     #: how many copies of the residual stream the blocks keep (hyper-connections): the model then hands its blocks a float32
     #: ``[streams, T, hidden]`` tensor (also for a single copy) and the head reads their sum; 0: one plain ``[T, hidden]`` stream
     streams: int = 0
+    #: a tensor ``[passes, hidden]`` whose rows are added to the stream where passes start (``ScheduleEntry.enters``)
+    pass_vectors: Optional[TensorSpec] = None

@@ -136,12 +136,12 @@ def test_band_scaled_frequencies(rot):
 
 
 def test_which_prompt_kernel_a_head_layout_gets():
-    """The tcgen05 prompt kernel takes keys and values of 64 or 128 alike, or page rows of 64 to 192 numbers whose first 64 or
+    """The tcgen05 prompt kernel takes keys and values of 64 or 128 each, or page rows of 64 to 192 numbers whose first 64 or
     128 are the values; a latent layer asks for the kernels of its own layout and a name tells the layouts apart."""
     from marin_b200.kernels import build, ops
 
     assert ops.tc_sink_attention_supported(64, 64) and ops.tc_sink_attention_supported(128, 128)
-    assert not ops.tc_sink_attention_supported(128, 64) and not ops.tc_sink_attention_supported(96, 96)
+    assert ops.tc_sink_attention_supported(128, 64) and not ops.tc_sink_attention_supported(96, 96)
     for d, dv, ok in ((160, 128, True), (80, 64, True), (192, 128, True), (64, 64, True), (128, 96, False), (208, 128, False),
                       (72, 64, False), (112, 48, False), (256, 128, False)):
         assert ops.tc_sink_attention_supported(d, dv, True) == ok, (d, dv)
