@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine on one B200, with their fractions of roofline.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers N] [--impl ours|reference]
-    python bench.py --arch lakulix|fegarax|nirotar|vogunex|pununex [--model 4b|8b|14b] [--layers 12] [--batch 8] [--profile]
+    python bench.py --arch lakulix|fegarax|nirotar|vogunex|pununex|punolix [--model 4b|8b|14b] [--layers 12] [--batch 8] [--profile]
 
 The default run has the layer sizes of the Qwen3-4B layout with random bfloat16 weights, a batch of 8
 sequences and a context of 4096 positions (the last timed step reaches it).  A "step" is one decode
@@ -29,6 +29,8 @@ layer, attention over a shared latent with a window, in turn; dense and routed f
 mixer) beside the Nirotar layers at the same sizes, the closest of the engine's models.
 ``--arch pununex`` measures Pununex layers (windowed attention with kept first positions beside a gated delta rule, and a delta
 rule alone, in turn; dense and routed feed-forwards, norms on the sublayers' outputs) beside the Vogunex layers at the same sizes.
+``--arch punolix`` measures Punolix layers (differential attention, and chunked attention behind short convolutions beside gated linear
+attention, in turn; a dense feed-forward on the mixer's own norm in each) beside the Pununex layers at the same sizes.
 The default workload and its line are not touched by any of them.
 
 Peaks come from MEASURED_PEAKS.json beside this file if present, else 6.65 TB/s and 1.59 PFLOP/s.
@@ -426,6 +428,27 @@ def pununex_layout(raw: dict, layers: int) -> dict:
             "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": kinds[i % 4][2]} for i in range(layers)]}
 
 
+PUNOLIX_LAYERS = ("in turn: differential attention (the layout's heads, two maps of half a head each over values of a whole one, neighbouring pairs rotated, "
+                  "scores capped); attention with the layout's heads in chunks of 1,024 positions (four taps over q, k and v, q and k normed, half-split "
+                  "pairs with band-scaled frequencies) beside gated linear attention (heads of 128 x 128 filling the width, a decay per key channel out of "
+                  "two matrices of rank 16, a silu gate).  The layout's dense feed-forward (a gelu gate) beside every mixer on the same norm; one pass of a "
+                  "loop around all of them")
+
+
+def punolix_layout(raw: dict, layers: int) -> dict:
+    """A Punolix configuration at a Qwen3 layout's sizes: the same width, vocabulary, attention heads and feed-forward."""
+    head, heads, kv, width = raw["head_dim"], raw["num_attention_heads"], raw["num_key_value_heads"], raw["hidden_size"]
+    diff = {"heads": heads, "kv_heads": kv, "dim": head // 2, "vdim": head, "scale": (head // 2) ** -0.5, "softcap": 50.0, "diff": 0.4,
+            "rot": {"base": 500000.0, "dims": head // 2}}
+    left = {"heads": heads, "kv_heads": kv, "dim": head, "vdim": head, "scale": head ** -0.5, "conv": 4, "mask": {"size": 1024},
+            "rot": {"base": 500000.0, "dims": head, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}
+    right = {"heads": width // 128, "dim": 128, "vdim": 128, "tau": 16.0}
+    kinds = [("attention", diff), ("parallel", {"left": left, "right": right, "left_scale": 0.6, "right_scale": 0.8})]
+    return {"architecture": "Punolix", "vocab": raw["vocab_size"], "width": width, "norm": {"eps": 1e-6}, "max_positions": 2 * CONTEXT, "residual_mult": 0.5,
+            "embedding": {"scale": 1.0}, "loop": {"start": 0, "stop": layers, "times": 1},
+            "layers": [{"type": kinds[i % 2][0], "mixer": kinds[i % 2][1], "mlp": {"kind": "dense", "ff": raw["intermediate_size"]}} for i in range(layers)]}
+
+
 def arch_mode(args, pk, arch: str) -> int:
     """Decode and prompt throughput of another architecture at a Qwen3 layout's sizes, and of that Qwen3 layout at the same
     depth, with their fractions of roofline: one JSON line.  With --profile: the architecture's stage tables."""
@@ -434,7 +457,7 @@ def arch_mode(args, pk, arch: str) -> int:
     import torch
 
     from marin_b200 import Engine
-    from marin_b200.config import FegaraxConfig, LakulixConfig, NirotarConfig, PununexConfig, Qwen3Config, VogunexConfig
+    from marin_b200.config import FegaraxConfig, LakulixConfig, NirotarConfig, PunolixConfig, PununexConfig, Qwen3Config, VogunexConfig
 
     layers = args.layers or 12
     raw = dict(LAYOUTS[args.model], num_hidden_layers=layers)
@@ -443,8 +466,11 @@ def arch_mode(args, pk, arch: str) -> int:
     # the model it is measured beside: the Qwen3 layout, or for Nirotar the engine's closest model, Fegarax at that layout's sizes
     # (for Vogunex: Nirotar, whose windowed and latent attention and experts with a shared one are the nearest kernels)
     # (for Pununex: Vogunex, which keeps recurrent states beside a window of keys and has experts with a shared one)
-    beside = {"nirotar": "fegarax", "vogunex": "nirotar", "pununex": "vogunex"}.get(arch, "qwen3")
-    if arch == "pununex":
+    # (for Punolix: Pununex, whose windowed attention has capped scores and stands beside a recurrent mixer too)
+    beside = {"nirotar": "fegarax", "vogunex": "nirotar", "pununex": "vogunex", "punolix": "pununex"}.get(arch, "qwen3")
+    if arch == "punolix":
+        other = PunolixConfig.from_dict(punolix_layout(raw, layers))
+    elif arch == "pununex":
         other = PununexConfig.from_dict(pununex_layout(raw, layers))
     elif arch == "vogunex":
         other = VogunexConfig.from_dict(vogunex_layout(raw, layers))
@@ -456,7 +482,8 @@ def arch_mode(args, pk, arch: str) -> int:
         other = NirotarConfig.from_dict(nirotar_layout(raw, layers))
     arms = {arch: other, beside: FegaraxConfig.from_dict(fegarax_layout(raw, layers)) if beside == "fegarax" else
             NirotarConfig.from_dict(nirotar_layout(raw, layers)) if beside == "nirotar" else
-            VogunexConfig.from_dict(vogunex_layout(raw, layers)) if beside == "vogunex" else Qwen3Config.from_dict(raw)}
+            VogunexConfig.from_dict(vogunex_layout(raw, layers)) if beside == "vogunex" else
+            PununexConfig.from_dict(pununex_layout(raw, layers)) if beside == "pununex" else Qwen3Config.from_dict(raw)}
     out = {}
     for name, cfg in arms.items():
         if args.profile and name != arch:
@@ -500,7 +527,7 @@ def arch_mode(args, pk, arch: str) -> int:
         "config": {"layers": layers, "width": raw["hidden_size"], "ff": raw["intermediate_size"], "vocab": raw["vocab_size"],
                    "global_batch": args.batch, "seq_len": CONTEXT, "prefill_tokens": PREFILL_TOKENS, "kv_block": PAGE,
                    f"{arch}_layers": FEGARAX_LAYERS if arch == "fegarax" else NIROTAR_LAYERS if arch == "nirotar" else VOGUNEX_LAYERS if arch == "vogunex" else
-                   PUNUNEX_LAYERS if arch == "pununex" else
+                   PUNUNEX_LAYERS if arch == "pununex" else PUNOLIX_LAYERS if arch == "punolix" else
                    "lightning (heads of 128 x 128), attention (the layout's heads), wkv (heads of 64) in turn, a dense feed-forward in each",
                    "l2": "inputs larger than L2 (weights read per step exceed 126 MB)"},
         arch: out[arch], beside: out[beside], "impl": "ours"}))
@@ -528,9 +555,10 @@ def main() -> int:
     ap.add_argument("--model", default="4b", choices=sorted(LAYOUTS), help="layer sizes: Qwen3-4B (the default), 8B or 14B layout")
     ap.add_argument("--context", type=int, default=CONTEXT, help="context length the last timed decode step reaches (default 4096)")
     ap.add_argument("--profile", action="store_true", help="print where a step's time goes, stage by stage, instead of the JSON line")
-    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "lakulix", "fegarax", "nirotar", "vogunex", "pununex"],
+    ap.add_argument("--arch", default="qwen3", choices=["qwen3", "lakulix", "fegarax", "nirotar", "vogunex", "pununex", "punolix"],
                     help="qwen3: the default workload; lakulix, fegarax: that architecture at the layout's sizes beside the Qwen3 layout of "
-                         "equal size; nirotar: beside the Fegarax layers at that layout's sizes; vogunex: beside the Nirotar layers at those sizes; pununex: beside the Vogunex layers")
+                         "equal size; nirotar: beside the Fegarax layers at that layout's sizes; vogunex: beside the Nirotar layers at those sizes; pununex: beside the Vogunex layers; "
+                         "punolix: beside the Pununex layers")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm()

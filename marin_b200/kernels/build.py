@@ -218,13 +218,16 @@ def attention_tc_name(d: int, group: int, dv: int = 0, values_in_keys: bool = Fa
 #: One or two layouts of every source that is otherwise compiled for a model's own sizes when it first runs (the names and
 #: defines are those the wrappers in ``ops`` use): sink attention with keys and values of their own and over a shared latent
 #: with sixteen heads a CTA, sigmoid attention, chunked linear attention, attention over a window and pooled blocks, the chunked
-#: delta rule.
+#: delta rule, chunked gated linear attention, two maps per head.
 PER_LAYOUT_SAMPLES = {
     "mb_attention_sink_fast_d128_v128_g4": (["attention_sink_fast.cu"], ["HEAD_DIM=128", "V_DIM=128", "GROUP=4"]),
     "mb_attention_sink_fast_d160_v128_g16_vk": (["attention_sink_fast.cu"], ["HEAD_DIM=160", "V_DIM=128", "GROUP=16", "V_IN_K"]),
     "mb_attention_sigmoid_fast_d128_v128_g4": (["attention_sigmoid_fast.cu"], ["HEAD_DIM=128", "V_DIM=128", "GROUP=4"]),
     "mb_linear_attention_chunked_d128_v32": (["linear_attention_chunked.cu"], ["QK_DIM=128", "V_SLICE=32"]),
     "mb_delta_rule_chunked_d128_v32": (["delta_rule_chunked.cu"], ["QK_DIM=128", "V_SLICE=32"]),
+    "mb_gated_linear_chunked_d128_v128": (["gated_linear_chunked.cu"], ["QK_DIM=128", "V_SLICE=128"]),
+    "mb_attention_sink_fast_d128_v128_g8": (["attention_sink_fast.cu"], ["HEAD_DIM=128", "V_DIM=128", "GROUP=8"]),
+    "mb_attention_tc_d128_g8_pair": (["attention_tc.cu"], ["HEAD_DIM=128", "GROUP=8", "PAIR"]),
     "mb_attention_pooled_fast_d128_v128_g4_c2": (["attention_pooled_fast.cu"], ["HEAD_DIM=128", "V_DIM=128", "GROUP=4", "VALUE_HEADS=2"]),
 }
 

@@ -2342,5 +2342,66 @@ def gla_single(inp: GlaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, ga
         "gated linear attention (single tokens)")
 
 
-def gla_jobs(dtype, d: int, dv: int) -> dict:
-    return library_jobs("mb_gated_linear", "mb_delta_rule")
+#: portions longer than this go 64 tokens at a time through the tensor-core kernels where the head sizes allow (False: token by token)
+use_chunked_gla = True
+GLA_CHUNKED_FROM = 8
+
+
+def gla_chunked_supported(dtype, d: int, dv: int, rank: int) -> bool:
+    return dtype == torch.bfloat16 and d % 16 == 0 and 16 <= d <= 128 and dv % 16 == 0 and rank % 16 == 0 and 16 <= rank <= 128
+
+
+def _gla_slice(dv: int) -> int:
+    """Value channels a CTA takes: a whole head's up to 128, else the largest part of equal ones up to 128."""
+    return max(n for n in range(16, 129, 16) if dv % n == 0)
+
+
+def _gla_chunked_job(d: int, dv: int) -> tuple:
+    n = _gla_slice(dv)
+    return f"mb_gated_linear_chunked_d{d}_v{n}", (["gated_linear_chunked.cu"], [f"QK_DIM={d}", f"V_SLICE={n}"])
+
+
+def gla_chunk_bytes(d: int, dv: int) -> int:
+    """Bytes a chunk of 64 tokens and a head keep between the chunked kernels."""
+    return 4 * (64 * d + d * dv)
+
+
+def gla_chunked(inp: GlaInputs, state: torch.Tensor, ctx, slots: torch.Tensor, gate: str, norm_w: torch.Tensor, eps: float, factor: float, out: torch.Tensor,
+                H: int, d: int, dv: int, first_req: int = 0) -> None:
+    """Requests ``first_req`` on (those before bring a token each), 64 tokens at a time, from the projections' rows to the gated heads in ``out`` (rows
+    may be strided)."""
+    _need_cuda(state, slots, norm_w)
+    assert gla_chunked_supported(inp.q.dtype, d, dv, inp.low.shape[1]) and state.dtype == torch.float32 and tuple(state.shape[1:]) == (H, d, dv)
+    assert out.stride(1) == 1 and out.shape[1] == H * dv and norm_w.dtype == torch.float32 and norm_w.numel() == dv
+    T = inp.q.shape[0]
+    tokens = T - first_req
+    chunks = tokens // 64 + ctx.num_requests - first_req
+    ws = ctx.workspace
+    floats = ws.get("gla_chunks", (chunks * H * gla_chunk_bytes(d, dv) // 4,), torch.float32)
+    whole = _gla_slice(dv) == dv
+    o = None if whole else ws.get("gla_o", (T, H * dv), torch.float32)
+    name, job = _gla_chunked_job(d, dv)
+    lib = build.load(name, *job)
+    args = list(_gla_args(inp, H, d, dv))
+    del args[5]                                                # (the dtype)
+    args += [_ptr(state), _ptr(ctx.cu_tokens), _ptr(slots), _ptr(floats), _ptr(o), _c_void_p(inp.gate.data_ptr()), _c_int(inp.gate.stride(0)),
+             _c_int(DELTA_GATES[gate]), _ptr(norm_w), _c_float(eps), _c_float(factor), _c_void_p(out.data_ptr()), _c_int(out.stride(0)), _c_int(first_req),
+             _c_int(ctx.num_requests), _c_int(ctx.max_query_len), _c_int(H), _c_int(dv), _stream()]
+    rows = inp.q.element_size() * tokens * H
+    # what the algorithm needs is shared out over the three: its inputs once, the state once, the outputs once
+    _cost(rows * (d + dv) + tokens * inp.low.shape[1] * 2, 2.0 * tokens * H * d * dv)
+    _check(lib.mb_gla_chunked(_c_int(0), *args), "gated linear attention (chunks' parts)")
+    _cost((ctx.num_requests - first_req) * H * d * dv * 8, 0.0)
+    _check(lib.mb_gla_chunked(_c_int(1), *args), "gated linear attention (states carried)")
+    _cost(rows * (d + 2 * dv), 2.0 * tokens * H * d * dv)
+    _check(lib.mb_gla_chunked(_c_int(2), *args), "gated linear attention (outputs)")
+    if not whole:
+        delta_norm(o, inp.gate, gate, norm_w, eps, factor, out, H, dv, first_req)
+
+
+def gla_jobs(dtype, d: int, dv: int, rank: int) -> dict:
+    jobs = library_jobs("mb_gated_linear", "mb_delta_rule")
+    if use_chunked_gla and gla_chunked_supported(dtype, d, dv, rank):
+        name, job = _gla_chunked_job(d, dv)
+        jobs[name] = job
+    return jobs

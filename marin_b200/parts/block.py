@@ -285,7 +285,13 @@ class PostNormBlock(Part):
 class ParallelBlock(Part):
     """``x <- x + m (mixer(h) + feedforward(h))`` with one norm, ``h = norm1(x)``, that both sublayers read (a layer without a feed-forward has the mixer
     alone).  ``block_params["residual_mult"]``: ``m`` (1 without it); mixer and feed-forward take it as their ``out_scale``, so that it multiplies
-    float32 numbers before they are rounded.  A row the mixer adds to every token (``Mixer.row_bias``) rides on the norm's kernel."""
+    float32 numbers before they are rounded.  A row the mixer adds to every token (``Mixer.row_bias``) rides on the norm's kernel.
+
+    In bfloat16, where both sublayers allow it (``joins_products``), what they take from ``h`` is one product, the feed-forward's activation applied to
+    its columns in the epilogue, and what they add to the stream is one product of their results side by side."""
+
+    #: False: the sublayers' products stay their own (the twin the joined ones are compared with); read when a model is loaded
+    join_products = True
 
     def __init__(self, spec: LayerSpec):
         names = spec.names
@@ -309,6 +315,16 @@ class ParallelBlock(Part):
         for p in self.parts():
             p.load(tensors, rt)
         self.mixer.adds_row_bias = False
+        self.w_in = self.w_last = None
+        mixer, ff = self.mixer, self.feedforward
+        if (self.join_products and rt.dtype == torch.bfloat16 and mixer.joins_products and ff is not None and getattr(ff, "joins_products", False)
+                and mixer.o_dim % 8 == 0 and mixer.w_in.shape[1] % 8 == 0):
+            n = mixer.w_in.shape[0]
+            self.plain = n + -n % 32                           # the mixer's rows, in whole steps of the epilogue's warps
+            self.w_in = torch.cat([mixer.w_in, mixer.w_in.new_zeros(self.plain - n, mixer.w_in.shape[1]), ff.w_gate_up], dim=0).contiguous()
+            self.w_last = torch.cat([mixer.w_o, ff.w_down], dim=1).contiguous()
+            mixer.lend_products(self.w_in[:n])
+            ff.w_gate_up, ff.w_down = self.w_in[self.plain:], None
         self.rt = rt
 
     def weight_bytes(self, dtype) -> int:
@@ -329,6 +345,16 @@ class ParallelBlock(Part):
     def forward(self, hidden: torch.Tensor, ctx, cache):
         ops.stage_name = "norm"
         x = self.norm1.forward(hidden, ctx.workspace.get("normed", tuple(hidden.shape), self.rt.dtype), self.mixer.row_bias)
+        if self.w_in is not None:
+            T, n, ff = hidden.shape[0], self.mixer.o_dim, self.feedforward
+            ops.stage_name = "inputs, gate|up"
+            rows = ctx.workspace.get("layer_rows", (T, self.plain), x.dtype)
+            outs = ctx.workspace.get("layer_outs", (T, self.w_last.shape[1]), x.dtype)
+            ops.gemm_glu_rows(x, self.w_in, rows, outs[:, n:], ff.activation, ff.out_scale)
+            self.mixer.forward(x, ctx, cache, hidden, rows=rows[:, :self.mixer.w_in.shape[0]], out=outs[:, :n])
+            ops.stage_name = "o|down"
+            ops.gemm(outs, self.w_last, hidden, accumulate=True)
+            return
         self.mixer.forward(x, ctx, cache, hidden)
         if self.feedforward is not None:
             self.feedforward.forward(x, ctx, hidden)

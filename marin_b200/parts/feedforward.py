@@ -63,6 +63,11 @@ class SwiGLU(FeedForward):
     def couples_norm(self) -> bool:
         return self.out_scale == 1.0
 
+    @property
+    def joins_products(self) -> bool:
+        """Whether a block may take ``w_gate_up`` and ``w_down`` into products shared with the other sublayer (``ops.gemm_glu_rows``)."""
+        return self.fused and self.intermediate % 8 == 0
+
     def forward(self, x, ctx, residual: torch.Tensor, then_norm=None):
         T = x.shape[0]
         ws = ctx.workspace

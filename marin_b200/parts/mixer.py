@@ -112,6 +112,10 @@ class Mixer(Part):
     #: that mixers side by side can share both products.
     joins_products = False
 
+    def lend_products(self, w_in: torch.Tensor) -> None:
+        """Whoever took ``w_in`` and ``w_o`` into products of its own hands back where the first now lies: this mixer keeps no copy."""
+        self.w_in, self.w_o = w_in, None
+
     #: a vector (float32 ``[hidden]``, after ``load``) that the mixer adds to every row of the residual: the output projection's bias, times whatever
     #: multiplies the result.  A block whose norm adds it to the rows (``RMSNorm.forward(then_add=)``) sets ``adds_row_bias`` to False.
     row_bias: Optional[torch.Tensor] = None
@@ -954,6 +958,11 @@ class ParallelMixers(Mixer):
                     m.w_o = None
                 self.joins_products = True
         self.rt = rt
+
+    def lend_products(self, w_in: torch.Tensor) -> None:
+        super().lend_products(w_in)
+        for m, (first, n) in zip(self.inner, self.cols):
+            m.w_in = w_in[first:first + n]
 
     def bytes_read(self, tokens: int, dtype) -> int:
         return sum(m.bytes_read(tokens, dtype) for m in self.inner)

@@ -438,6 +438,7 @@ class GatedLinearAttention(Mixer):
         self.names = dict(self.NAMES, **(names or {}))
         self.qk, self.hv = self.heads * self.dim, self.heads * self.vdim
         self.o_dim = self.hv
+        self.low_dim = self.rank + -self.rank % 16             # the decays' numbers between the matrices, padded with zeros
         self.w_in = self.w_2 = self.a_bias = self.norm_w = self.w_o = None
 
     def _n(self, key: str) -> str:
@@ -457,7 +458,7 @@ class GatedLinearAttention(Mixer):
         # can take them by 16-byte loads).  The decays' second matrix is applied inside the recurrence's kernels, in steps of 16 numbers.
         blocks = {p: tensors.pop(self._n(p)) for p in "qkvg"}
         first, second = tensors.pop(self._n("a1")), tensors.pop(self._n("a2"))
-        pad = -self.rank % 16
+        pad = self.low_dim - self.rank
         blocks["low"] = torch.cat([first, first.new_zeros(pad, first.shape[1])], dim=0)
         self.w_2 = rt.matrix(torch.cat([second, second.new_zeros(second.shape[0], pad)], dim=1))
         self.cols, at, rows = {}, 0, []
@@ -474,11 +475,12 @@ class GatedLinearAttention(Mixer):
         return super().flops(tokens, pairs) + 4.0 * tokens * self.heads * self.dim * self.vdim
 
     def kernel_jobs(self, dtype) -> Dict[str, tuple]:
-        return ops.gla_jobs(dtype, self.dim, self.vdim)
+        return ops.gla_jobs(dtype, self.dim, self.vdim, self.low_dim)
 
     def workspace_per_token(self, dtype) -> int:
         """Bytes a step keeps per token beside the products' rows: the heads' sums, and what the chunked kernels hand over."""
-        return 4 * self.hv
+        chunked = self.heads * ops.gla_chunk_bytes(self.dim, self.vdim) // 64 if ops.gla_chunked_supported(dtype, self.dim, self.vdim, self.low_dim) else 0
+        return 4 * self.hv + chunked
 
     joins_products = True
 
@@ -495,11 +497,14 @@ class GatedLinearAttention(Mixer):
         joined = out is not None
         if not joined:
             out = ws.get("gla_out", (T, self.hv), x.dtype)
-        ops.stage_name = "gated linear attention"
+        ops.stage_name = "gated linear"
         single = ctx.num_decode if ops.use_gla_single and ops.gla_single_supported(d, dv) else 0
         if single:                                             # requests with one token each come first in the batch
             ops.gla_single(inputs, cache.state, ctx, cache.slots, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, single, H, d, dv)
-        if ctx.num_requests > single:
+        if (ctx.num_requests > single and ops.use_chunked_gla and ops.gla_chunked_supported(x.dtype, d, dv, self.low_dim)
+                and ctx.max_query_len > ops.GLA_CHUNKED_FROM):
+            ops.gla_chunked(inputs, cache.state, ctx, cache.slots, self.gate, self.norm_w, self.norm_eps, self.out_scale, out, H, d, dv, single)
+        elif ctx.num_requests > single:
             o = ws.get("gla_o", (T, self.hv), torch.float32)
             ops.gla_scan(inputs, cache.state, ctx, cache.slots, o, H, d, dv, single)
             ops.stage_name = "norm, gate"

@@ -86,7 +86,7 @@ def differential_attention(h: torch.Tensor, t: Dict[str, torch.Tensor], name: st
     q = (h @ t[f"{name}.q"].T + t[f"{name}.q.b"]).reshape(T, H, 2, d)
     k = (h @ t[f"{name}.k"].T + t[f"{name}.k.b"]).reshape(T, G, 2, d)
     v = (h @ t[f"{name}.v"].T + t[f"{name}.v.b"]).reshape(T, G, dv)
-    a1, a2 = (softmax_attention(rotate(q[:, :, n], m["rot"], True), rotate(k[:, :, n], m["rot"], True), v, m["scale"], m["softcap"]) for n in (0, 1))
+    a1, a2 = (softmax_attention(rotate(q[:, :, n], m["rot"], True), rotate(k[:, :, n], m["rot"], True), v, m["scale"], m.get("softcap")) for n in (0, 1))
     o = a1 - lam_of(t, name, m["diff"]) * a2
     o = o / rms(o, eps) * (1.0 - m["diff"])
     return o.reshape(T, H * dv) @ t[f"{name}.o"].T
@@ -107,11 +107,13 @@ def chunked_attention(h: torch.Tensor, t: Dict[str, torch.Tensor], name: str, m:
     head, rotated; the output projection has a bias."""
     T = h.shape[0]
     H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q, k, v = (short_convolution(h @ t[f"{name}.{p}"].T + t[f"{name}.{p}.b"], t[f"{name}.{p}.conv"]) for p in "qkv")
+    q, k, v = (h @ t[f"{name}.{p}"].T + t[f"{name}.{p}.b"] for p in "qkv")
+    if m.get("conv"):
+        q, k, v = (short_convolution(x, t[f"{name}.{p}.conv"]) for p, x in zip("qkv", (q, k, v)))
     q, k = q.reshape(T, H, d), k.reshape(T, G, d)
     q = rotate(q / rms(q, eps) * t[f"{name}.q.norm"], m["rot"], False)
     k = rotate(k / rms(k, eps) * t[f"{name}.k.norm"], m["rot"], False)
-    o = softmax_attention(q, k, v.reshape(T, G, dv), m["scale"], None, m["mask"]["size"])
+    o = softmax_attention(q, k, v.reshape(T, G, dv), m["scale"], None, (m.get("mask") or {}).get("size"))
     return o.reshape(T, H * dv) @ t[f"{name}.o"].T + t[f"{name}.o.b"]
 
 
@@ -188,7 +190,7 @@ def forward(config: dict, tensors: Dict[str, torch.Tensor], tokens: List[int], r
             if entered > 0:
                 x = x + first
             x = x + t["loop.step"][entered]
-        x = parallel_layer(config["layers"][i], x, t, f"l{i}", eps, config["residual_mult"])
+        x = parallel_layer(config["layers"][i], x, t, f"l{i}", eps, config.get("residual_mult", 1.0))
         if residuals is not None:
             residuals.append(x.clone())
     return (x / rms(x, eps) * t["final.norm"]) @ t["head"].T
