@@ -429,14 +429,162 @@ __global__ void __launch_bounds__(RUNS <= 2 ? 1024 : 256) qkv_finish_vec_kernel(
     }
 }
 
+// The same without a barrier, for bf16 heads whose runs of 8 are a power of two and lie in one warp (values of any multiple of 8; no norm over the
+// whole projection, no mixed values): a thread owns one run of 8 neighbouring channels of q, k or v over a run of consecutive tokens, a
+// head's sum of squares and its rotation partners come by shuffles, cosines and sines from a table made once a step (rope: [tokens][rot_dim],
+// cosines then sines).  With a convolution the thread's weights and last TAPS - 1 inputs stay in registers, so that every row is read once a run.
+// TAPS 0: no convolution.
+#define FR_THREADS 128
+#define FR_RUN 8
+
+template <int TAPS>
+__global__ void __launch_bounds__(FR_THREADS, 3) qkv_finish_runs_kernel(
+    const bf16* __restrict__ row, int row_stride, bf16* __restrict__ q_out, const float* __restrict__ q_b, const float* __restrict__ k_b,
+    const float* __restrict__ v_b, int norm, const float* __restrict__ q_w, const float* __restrict__ k_w, float eps, const int* __restrict__ positions,
+    const float* __restrict__ rope, int rot_dim, const int* __restrict__ slot_mapping, bf16* __restrict__ k_cache, bf16* __restrict__ v_cache, int H, int K,
+    int d, int dv, int page_size, int write_kv, int interleaved, int maps, ConvRows cv, int tokens, int run) {
+    PDL_ENTER();
+    row = pdl_fresh(row); rope = pdl_fresh(rope); cv.ring = pdl_fresh(cv.ring);
+    constexpr int RING = TAPS > 0 ? TAPS : 1;
+    const int KG = K / maps, wide = d * maps, half = rot_dim >> 1;
+    const int q_cols = H * d, k_end = q_cols + (write_kv ? K * d : 0), cols = k_end + (write_kv ? KG * dv : 0);
+    const int c = (blockIdx.y * FR_THREADS + threadIdx.x) * 8, lane = threadIdx.x & 31;
+    const bool active = c < cols;
+    const bool is_q = c < q_cols, is_v = c >= k_end;
+    const int rel = is_q ? c : is_v ? c - k_end : c - q_cols;
+    const int width = is_v ? dv : d, head = rel / width, i0 = rel - head * width;
+    const int t0 = blockIdx.x * run, t1 = min(tokens, t0 + run);
+    const bool rotated = !is_v && i0 < rot_dim, low = i0 < half;
+    const int partner = rotated && !interleaved ? lane + (low ? half / 8 : -half / 8) : lane;
+    const int j0 = interleaved ? i0 >> 1 : low ? i0 : i0 - half;      // the first of this run's angles
+    float bias[8], w[8];
+    {
+        const float* b = is_q ? q_b : is_v ? v_b : k_b;
+        const float* ww = is_q ? q_w : k_w;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { bias[e] = 0.0f; w[e] = 1.0f; }
+        if (active && b != nullptr) load8(b + rel, bias);
+        if (active && norm && !is_v) load8(ww + i0, w);
+    }
+    float wt[TAPS > 0 ? TAPS : 1][8], past[TAPS > 1 ? TAPS - 1 : 1][8];      // past[b]: the input b + 1 tokens back
+    if (TAPS > 0 && active)
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) load8(cv.w + (size_t)j * cv.channels + c, wt[j]);
+    uint4 raw[FR_RUN];                                         // every row of the run in flight at once
+#pragma unroll
+    for (int u = 0; u < FR_RUN; ++u) {
+        raw[u] = make_uint4(0, 0, 0, 0);
+        if (active && t0 + u < t1) raw[u] = *reinterpret_cast<const uint4*>(row + (size_t)(t0 + u) * row_stride + c);
+    }
+    int first = 0, end = 0;
+    float* kept = nullptr;
+#pragma unroll
+    for (int u = 0; u < FR_RUN; ++u) {
+        const int t = t0 + u;
+        if (t >= t1) break;                                    // (the same for the whole block)
+        float x[8];
+        unpack8(raw[u], x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += bias[e];
+        if (TAPS > 0) {
+            if (u == 0 || t == end) {                          // another request: its window, from this step's rows, the ring, or nothing
+                const int req = cv.req_index[t], pos = positions[t];
+                first = cv.cu_tokens[req];
+                end = cv.cu_tokens[req + 1];
+                kept = cv.ring + (size_t)cv.slots[req] * TAPS * cv.channels + c;
+                if (TAPS > 1 && active)
+#pragma unroll
+                    for (int b = 0; b < TAPS - 1; ++b) {
+                        if (t - b - 1 >= first) {
+                            unpack8(*reinterpret_cast<const uint4*>(row + (size_t)(t - b - 1) * row_stride + c), past[b]);
+#pragma unroll
+                            for (int e = 0; e < 8; ++e) past[b][e] += bias[e];
+                        } else if (pos - b - 1 >= 0) {
+                            load8(kept + (size_t)((pos - b - 1) % RING) * cv.channels, past[b]);
+                        } else {
+#pragma unroll
+                            for (int e = 0; e < 8; ++e) past[b][e] = 0.0f;
+                        }
+                    }
+            }
+            if (TAPS > 1 && active && t < cv.singles) {
+                float* dst = kept + (size_t)(positions[t] % RING) * cv.channels;
+                *reinterpret_cast<float4*>(dst) = make_float4(x[0], x[1], x[2], x[3]);
+                *reinterpret_cast<float4*>(dst + 4) = make_float4(x[4], x[5], x[6], x[7]);
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                float sum = 0.0f;                              // (the oldest first, as the other kernels add)
+#pragma unroll
+                for (int b = TAPS - 2; b >= 0; --b) sum = fmaf(wt[TAPS - 2 - b][e], past[b][e], sum);
+                const float now = x[e];
+                x[e] = fmaf(wt[TAPS > 0 ? TAPS - 1 : 0][e], now, sum);
+#pragma unroll
+                for (int b = TAPS - 2; b > 0; --b) past[b][e] = past[b - 1][e];
+                if (TAPS > 1) past[0][e] = now;
+            }
+        }
+        if (norm) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+            for (int o = 1; o < d / 8; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);       // (a head's lanes; values do not use theirs)
+            if (!is_v) {
+                const float factor = 1.0f / sqrtf(ss / (float)d + eps);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[e] = x[e] * factor * w[e];
+            }
+        }
+        if (rot_dim > 0) {
+            const float* cs_row = rope + (size_t)t * rot_dim + j0;
+            if (interleaved) {
+                if (rotated) {
+                    const float4 c4 = *reinterpret_cast<const float4*>(cs_row), s4 = *reinterpret_cast<const float4*>(cs_row + half);
+                    const float cs[4] = {c4.x, c4.y, c4.z, c4.w}, sn[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float a = x[2 * e], b = x[2 * e + 1];
+                        x[2 * e] = a * cs[e] - b * sn[e];
+                        x[2 * e + 1] = b * cs[e] + a * sn[e];
+                    }
+                }
+            } else {
+                float b[8];
+#pragma unroll
+                for (int e = 0; e < 8; ++e) b[e] = __shfl_sync(0xffffffffu, x[e], partner);
+                if (rotated) {
+                    float cs[8], sn[8];
+                    load8(cs_row, cs);
+                    load8(cs_row + half, sn);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) x[e] = low ? x[e] * cs[e] - b[e] * sn[e] : x[e] * cs[e] + b[e] * sn[e];
+                }
+            }
+        }
+        if (!active) continue;
+        if (is_q) {
+            const int m = head % maps;
+            bf16* dst = q_out + ((size_t)t * H + head) * wide + i0;
+            for (int o = 0; o < maps; ++o) *reinterpret_cast<uint4*>(dst + o * d) = o == m ? pack8(x) : make_uint4(0, 0, 0, 0);
+        } else {
+            const int slot = slot_mapping[t];
+            if (slot < 0) continue;
+            const size_t page = (size_t)(slot / page_size), at = (size_t)(slot % page_size);
+            if (is_v) *reinterpret_cast<uint4*>(v_cache + ((page * KG + head) * page_size + at) * dv + i0) = pack8(x);
+            else *reinterpret_cast<uint4*>(k_cache + ((page * KG + head / maps) * page_size + at) * wide + (head % maps) * d + i0) = pack8(x);
+        }
+    }
+}
+
 static bool aligned16(const void* p) { return (((uintptr_t)p) & 15) == 0; }
 
+// rope: null, or what qkv_finish_runs_kernel takes (rot_mag is then 1).
 MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out, const float* q_b, const float* k_b, const float* v_b,
                          int norm_mode, const float* q_w, const float* k_w, float eps, const int* positions, const float* inv_freq,
                          int rot_dim, float rot_mag, const int* slot_mapping, void* k_cache, void* v_cache, int v_mode, void* v_shared,
                          const float* v_lambda, int tokens, int H, int K, int d, int dv, int page_size, int write_kv, int interleaved,
                          int maps, const float* conv_w, float* ring, const int* slots, const int* req_index, const int* cu_tokens, int taps, int singles,
-                         cudaStream_t s) {
+                         const float* rope, cudaStream_t s) {
     if (tokens <= 0) return 0;
     if (maps < 1 || H % maps != 0 || K % maps != 0) return MB_ERR_BAD_SIZE;
     if (conv_w != nullptr && (taps < 1 || taps > 64 || !write_kv)) return MB_ERR_BAD_SIZE;
@@ -445,6 +593,22 @@ MB_API int mb_qkv_finish(const void* row, int row_stride, int dtype, void* q_out
     if ((v_mode == 1 || v_mode == 2) && v_shared == nullptr) return MB_ERR_BAD_SIZE;
     if (v_mode == 2 && v_lambda == nullptr) return MB_ERR_BAD_SIZE;
     if (inv_freq == nullptr) rot_dim = 0;
+    const int lanes = d / 8;                                   // of a head: a power of two within a warp
+    if (dtype == MB_BF16 && (rope != nullptr || rot_dim == 0) && norm_mode != 2 && v_mode == 0 && d % 8 == 0 && dv % 8 == 0 && lanes <= 32 && (lanes & (lanes - 1)) == 0 &&
+        (interleaved ? rot_dim % 8 == 0 : rot_dim % 16 == 0) && row_stride % 8 == 0 && (conv_w == nullptr || taps <= 4) && aligned16(row) && aligned16(q_out) &&
+        aligned16(q_b) && aligned16(k_b) && aligned16(v_b) && aligned16(q_w) && aligned16(k_w) && aligned16(k_cache) && aligned16(v_cache) && aligned16(conv_w) &&
+        aligned16(ring) && aligned16(rope)) {
+        const int cols = H * d + (write_kv ? K * d + K / maps * dv : 0);
+        const int run = tokens >= 256 ? FR_RUN : tokens >= 64 ? 2 : 1;
+        dim3 grid((tokens + run - 1) / run, (cols / 8 + FR_THREADS - 1) / FR_THREADS);
+#define FR_CASE(TAPS)                                                                                                                                \
+    if ((conv_w == nullptr ? 0 : taps) == TAPS)                                                                                                      \
+        return launch_kernel(qkv_finish_runs_kernel<TAPS>, grid, FR_THREADS, 0, s, 0, (const bf16*)row, row_stride, (bf16*)q_out, q_b, k_b, v_b, norm_mode, q_w, \
+                             k_w, eps, positions, rope, rot_dim, slot_mapping, (bf16*)k_cache, (bf16*)v_cache, H, K, d, dv, page_size, write_kv,      \
+                             interleaved, maps, cv, tokens, run);
+        FR_CASE(0) FR_CASE(1) FR_CASE(2) FR_CASE(3) FR_CASE(4)
+#undef FR_CASE
+    }
     const size_t smem = ((size_t)(H + K) * d + rot_dim + H + K) * sizeof(float);
     if (smem > 160 * 1024) return MB_ERR_BAD_SIZE;
     const int runs8 = (H + K) * d / 8;

@@ -362,8 +362,8 @@ stream_k = True
 #: pays a fixed part worth 7,700 such units (about 8 us: every CTA parks a partial tile at the start and the last
 #: epilogue, which nothing overlaps, is longer).  Measured times came out up to 0.1 above the predicted ratio, hence
 #: the margin.  Groups walk different k at the same time, so x has to stay in L2 (at 71 MB stream-K lost 6 % where
-#: the fit promised 9 %), and with fewer than four token tiles the fit did not hold (0.98 and 1.07 for 0.75 and 0.91).
-_KBLOCK_FIXED, _STREAM_K_FIXED, _STREAM_K_MARGIN, _STREAM_K_MAX_X_BYTES = 138, 7700, 0.87, 48 << 20
+#: the fit promised 9 %; at 57 and 67 MB and 20 row tiles it gained 22 and 17 %), and with fewer than four token tiles the fit did not hold (0.98 and 1.07 for 0.75 and 0.91).
+_KBLOCK_FIXED, _STREAM_K_FIXED, _STREAM_K_MARGIN, _STREAM_K_MAX_X_BYTES = 138, 7700, 0.87, 64 << 20
 
 
 def stream_k_plan(T: int, N: int, K: int) -> Optional[int]:
@@ -1284,6 +1284,10 @@ NORM_MODES = {None: 0, "head": 1, "whole": 2}
 VALUE_MODES = {None: 0, "leave": 1, "mix": 2}
 
 
+#: heads that allow it are finished by the kernel without barriers, which takes cosines and sines from the step's table (False: by the others)
+use_finish_runs = True
+
+
 def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Optional[str], q_w, k_w, eps: float, positions,
                inv_freq, rot_dim: int, rot_mag: float, slot_mapping, k_cache, v_cache, value_mode: Optional[str], v_shared,
                v_lambda, H: int, K: int, d: int, dv: int, write_kv: bool = True, interleaved: bool = False, maps: int = 1,
@@ -1306,6 +1310,10 @@ def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Opt
     assert k_cache.shape[1] == KG and H % maps == 0 and K % maps == 0
     assert v_shared is None or (v_shared.dtype == rows.dtype and v_shared.numel() >= T * KG * dv)
     page_size = k_cache.shape[2]
+    rope = None
+    if (use_finish_runs and ctx is not None and rows.dtype == torch.bfloat16 and inv_freq is not None and rot_mag == 1.0 and rot_dim % 8 == 0 and norm != "whole"
+            and value_mode is None):
+        rope = rope_table(ctx, positions, inv_freq)
     _cost(2 * T * ((H + K) * d + KG * dv) * rows.element_size(), 10.0 * T * (H + K) * d)
     single = 0
     if conv is not None:
@@ -1323,7 +1331,7 @@ def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Opt
         _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _c_int(VALUE_MODES[value_mode]), _ptr(v_shared), _ptr(v_lambda), _c_int(T),
         _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_int(int(write_kv)), _c_int(int(interleaved)), _c_int(maps),
         *((_ptr(conv.weight), _ptr(conv.ring), _ptr(conv.slots), _ptr(ctx.req_index), _ptr(ctx.cu_tokens), _c_int(taps)) if conv is not None
-          else (None, None, None, None, None, _c_int(0))), _c_int(single), _stream()), "q|k|v heads (sink attention)")
+          else (None, None, None, None, None, _c_int(0))), _c_int(single), _ptr(rope), _stream()), "q|k|v heads (sink attention)")
     if conv is not None and ctx.num_requests > single and taps > 1:
         _cost((ctx.num_requests - single) * (taps - 1) * channels * (4 + rows.element_size()))
         _check(_lib("mb_attention_sink").mb_conv_ring(

@@ -6,13 +6,20 @@ parameters.  ``NoPosition`` hands over nothing and the mixer skips the rotation.
 """
 from __future__ import annotations
 
+import functools
 import math
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
 from .base import Part, Runtime
 from .registry import register_position
+
+
+@functools.lru_cache(maxsize=64)
+def on_device(frequencies: Tuple[float, ...], device) -> torch.Tensor:
+    """The table on the device, one tensor for all layers that turn alike (cosines and sines are then made once a step for all of them)."""
+    return torch.tensor(frequencies, dtype=torch.float64).to(torch.float32).to(device)
 
 
 class PositionEncoding(Part):
@@ -84,7 +91,7 @@ class RescaledRotary(Rotary):
         return out
 
     def load(self, tensors, rt: Runtime) -> None:
-        self.inv_freq = torch.tensor(self.frequencies(), dtype=torch.float64).to(torch.float32).to(rt.device)
+        self.inv_freq = on_device(tuple(self.frequencies()), rt.device)
 
 
 @register_position("rope_llama3")
@@ -117,7 +124,7 @@ class BandScaledRotary(Rotary):
         return out
 
     def load(self, tensors, rt: Runtime) -> None:
-        self.inv_freq = torch.tensor(self.frequencies(), dtype=torch.float64).to(torch.float32).to(rt.device)
+        self.inv_freq = on_device(tuple(self.frequencies()), rt.device)
 
 
 @register_position("none")
