@@ -19,11 +19,13 @@ def embed(ids, table, out, pos_table=None, positions=None, scale=1.0):
         out.add_(pos_table[positions.long()].float())
 
 
-def rmsnorm(x, weight, eps, out, unit_offset=False):
+def rmsnorm(x, weight, eps, out, unit_offset=False, then_add=None):
     xf = x.float()
     ms = (xf * xf).sum(-1, keepdim=True) / xf.shape[-1]
     w = weight.float() + 1.0 if unit_offset else weight.float()
     out.copy_((xf * (1.0 / torch.sqrt(ms + eps)) * w).to(out.dtype))
+    if then_add is not None:
+        x.add_(then_add)
 
 
 def gemm(x, w, out, accumulate=False, then_norm=None):
@@ -103,15 +105,18 @@ def attention(q, k_cache, v_cache, out, ctx, block_table, H, K, d, scale, window
     out.copy_(res.view(T, H * d).to(out.dtype))
 
 
-def swiglu(gate_up, out, interleaved=False, activation="silu"):
+def swiglu(gate_up, out, interleaved=False, activation="silu", factor=1.0):
     T, I = out.shape
     if interleaved:
         blocks = gate_up.float().view(T, I // 16, 2, 16)
         g, u = blocks[:, :, 0, :].reshape(T, I), blocks[:, :, 1, :].reshape(T, I)
     else:
         g, u = gate_up[:, :I].float(), gate_up[:, I:].float()
-    act = torch.clamp(g, min=0.0) if activation == "relu" else g / (1.0 + torch.exp(-g))
-    out.copy_((act * u).to(out.dtype))
+    if activation == "gelu_tanh":
+        act = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+    else:
+        act = torch.clamp(g, min=0.0) if activation == "relu" else g / (1.0 + torch.exp(-g))
+    out.copy_((act * u * factor).to(out.dtype))
 
 
 def interleave_gate_up(gate, up):
@@ -123,9 +128,9 @@ def can_fuse_swiglu(dtype, hidden, intermediate):
     return dtype == torch.bfloat16 and intermediate % 16 == 0 and hidden % 8 == 0
 
 
-def gemm_swiglu(x, w_interleaved, out, workspace=None, activation="silu"):
+def gemm_swiglu(x, w_interleaved, out, workspace=None, activation="silu", factor=1.0):
     y = x.float() @ w_interleaved.float().t()
-    swiglu(y, out, True, activation)
+    swiglu(y, out, True, activation, factor)
 
 
 def gather_rows(src, rows, out):
