@@ -504,9 +504,17 @@ def arch_mode(args, pk, arch: str) -> int:
         state_bytes = sum(n.bytes() for n in engine.cache.state_needs.values())
         # (a layer with a window reads the window's positions, however long the sequence)
         # (one with pooled blocks: the window's positions and one row per block before it)
-        paged = sum(len(g.entries) * (g.need.bytes_read(int(run["mean_context"]), engine.rt.dtype) if g.need.pooled else
-                                      g.need.bytes_per_token(engine.rt.dtype) * min(run["mean_context"], g.need.window or run["mean_context"]))
-                    for g in engine.cache.groups)
+        # (one with a chunked mask: the positions of the current chunk up to its own, on average over the timed steps)
+        def seen(entry, need):
+            mixer = engine.model.blocks[engine.model.spec.schedule[entry].layer].mixer
+            inner = getattr(mixer, "inner", None)
+            chunk = max(getattr(m, "chunk", None) or 0 for m in [mixer] + (inner if isinstance(inner, list) else []))
+            if chunk:
+                return statistics.mean(p % chunk + 1 for p in range(CONTEXT - args.steps, CONTEXT))
+            return min(run["mean_context"], need.window or run["mean_context"])
+
+        paged = sum(g.need.bytes_read(int(run["mean_context"]), engine.rt.dtype) if g.need.pooled else g.need.bytes_per_token(engine.rt.dtype) * seen(e, g.need)
+                    for g in engine.cache.groups for e in g.entries)
         step_bytes = weight_bytes + args.batch * (paged + 2 * state_bytes)
         achieved = step_bytes / (run["ms_per_step"] / 1e3) / 1e9
         out[name] = {

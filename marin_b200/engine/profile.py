@@ -41,13 +41,18 @@ class StageRow:
         return self.flops / (self.share_us * 1e-6) / 1e12 if self.share_us > 0 else 0.0
 
 
-def lengths_of(runner: Runner, entries: Sequence[StepEntry], window: int = 0):
-    """Keys read and (query, key) pairs of the single-token rows and of the portions of a step that is about to run; a
-    position sees the last ``window`` keys only (0: all before it)."""
+def lengths_of(spans: Sequence[tuple], window: int = 0, chunk: int = 0):
+    """Keys read and (query, key) pairs of the single-token rows and of the portions of a step whose requests bring ``n`` tokens behind
+    ``before`` (``spans``: pairs of the two); a position sees the last ``window`` keys only, or (``chunk``) those of its own chunk
+    (0: all before it)."""
     counts = {"decode": [0, 0], "prefill": [0, 0]}
-    for e in entries:
-        before, n = runner.length(e.req_id), len(e.tokens)
+    for before, n in spans:
         which = counts["decode" if n == 1 else "prefill"]
+        if chunk > 0:
+            seen = [min(i % chunk, window - 1 if window > 0 else chunk) + 1 for i in range(before, before + n)]
+            which[0] += seen[0] - 1 + n
+            which[1] += sum(seen)
+            continue
         if window > 0:
             which[0] += min(before + n, window - 1 + n)
             which[1] += sum(min(i + 1, window) for i in range(before, before + n))
@@ -75,10 +80,7 @@ def profile_steps(runner: Runner, make_entries: Callable[[int], Sequence[StepEnt
 
     def one(i, log=None):
         entries = make_entries(i)
-        # (per window an attention kernel named in its launch record; 0: every earlier key is seen)
-        sizes = {0: lengths_of(runner, entries)}
-        for w in sorted({int(getattr(b.mixer, "window", 0) or 0) for b in getattr(runner.model, "blocks", [])} - {0}):
-            sizes[w] = lengths_of(runner, entries, w)
+        spans = [(runner.length(e.req_id), len(e.tokens)) for e in entries]
         ops.launch_log = log
         try:
             logits = runner.step(entries)
@@ -87,7 +89,7 @@ def profile_steps(runner: Runner, make_entries: Callable[[int], Sequence[StepEnt
                     after_step(logits)
         finally:
             ops.launch_log = None
-        return sizes
+        return spans
 
     for i in range(warmup):
         one(i)
@@ -96,7 +98,7 @@ def profile_steps(runner: Runner, make_entries: Callable[[int], Sequence[StepEnt
     with profile(activities=[ProfilerActivity.CUDA]) as prof:
         for i in range(steps):
             log: List[dict] = []
-            sizes = one(warmup + i, log)
+            spans = one(warmup + i, log)
             replayed = runner._replayed
             if replayed is not None:                        # a graph brings the labels recorded at its capture
                 log = [dict(entry) for entry in replayed["labels"]] + log
@@ -124,10 +126,14 @@ def profile_steps(runner: Runner, make_entries: Callable[[int], Sequence[StepEnt
                 shares[k].append(max(0.0, e.time_range.end - events[s * per_step + k - 1].time_range.end))
     rows: List[StageRow] = []
     merged: Dict[tuple, StageRow] = {}
+    sizes: Dict[tuple, dict] = {}                            # per mask that an attention kernel named in its launch record
     if gaps:
         rows.append(StageRow("(between steps)", "the device idle: host work, launch", 0, statistics.median(gaps), 0.0, 0.0, 0.0))
     for k, entry in enumerate(labels):
-        seen = sizes.get(int(entry.get("window", 0)), sizes[0])
+        mask = (int(entry.get("window", 0)), int(entry.get("chunk", 0)))
+        if mask not in sizes:
+            sizes[mask] = lengths_of(spans, *mask)
+        seen = sizes[mask]
         keys, pairs = seen.get(entry.get("rows", "all"), seen["all"])
         nbytes = entry["bytes"] + entry["bytes_per_key"] * keys
         flops = entry["flops"] + entry["flops_per_pair"] * pairs

@@ -1331,7 +1331,8 @@ def qkv_finish(rows: torch.Tensor, q_out: torch.Tensor, q_b, k_b, v_b, norm: Opt
         _ptr(slot_mapping), _ptr(k_cache), _ptr(v_cache), _c_int(VALUE_MODES[value_mode]), _ptr(v_shared), _ptr(v_lambda), _c_int(T),
         _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_int(int(write_kv)), _c_int(int(interleaved)), _c_int(maps),
         *((_ptr(conv.weight), _ptr(conv.ring), _ptr(conv.slots), _ptr(ctx.req_index), _ptr(ctx.cu_tokens), _c_int(taps)) if conv is not None
-          else (None, None, None, None, None, _c_int(0))), _c_int(single), _ptr(rope), _stream()), "q|k|v heads (sink attention)")
+          else (None, None, None, None, None, _c_int(0))), _c_int(single), _ptr(rope), _stream()),
+        "q|k|v heads (sink attention)" if conv is None else "q|k|v heads (convolution, sink attention)")
     if conv is not None and ctx.num_requests > single and taps > 1:
         _cost((ctx.num_requests - single) * (taps - 1) * channels * (4 + rows.element_size()))
         _check(_lib("mb_attention_sink").mb_conv_ring(
@@ -1385,6 +1386,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
     _need_cuda(q, k_cache, v_cache, block_table, sink_logits)
     assert out.is_cuda and out.stride(1) == 1
     maps = 2 if pair is not None else 1
+    what = "sink, two maps" if pair is not None else "sink"
     if pair is not None and (sink or gate is not None or H % 2 != 0):
         raise KernelError("attention_sink: pairs of maps go without a sink and a gate")
     more = (_c_int(keep_first), _c_float(softcap), _c_float(out_scale if pair is None else 1.0), _c_int(out.stride(0)))
@@ -1421,11 +1423,11 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
             ml = ctx.workspace.get("sink_part_sums", (plan.chunks, nd, H, 2), torch.float32)
             if launch_log is not None:
                 _cost(nd * per_row + 2 * _size(acc), 0.0, key_bytes, 2.0 * H * (d // maps + dv))
-                _pending_cost["rows"], _pending_cost["window"] = "decode", window
+                _pending_cost.update(rows="decode", window=window, chunk=chunk)
             _check(lib.mb_attn_sink_decode(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(acc), _ptr(ml), _ptr(block_table),
                                            _c_int(max_pages), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(page_size), _c_float(scale),
                                            _c_int(window), _c_int(chunk), _c_int(plan.split), _c_int(plan.chunks), _c_int(keep_first), _c_float(softcap), _stream()),
-                   "attention (sink, decode)")
+                   f"attention ({what}, decode)")
             _cost(_size(acc) + nd * H // maps * dv * size * (2 if gate is not None else 1))
             if pair is not None:
                 _check(lib.mb_attn_sink_merge_pair(_ptr(acc), _ptr(ml), _c_void_p(out.data_ptr()), _ptr(ctx.seq_lens), _c_int(nd), _c_int(K), _c_int(window),
@@ -1437,7 +1439,7 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
                                               _c_int(keep_first), _c_float(out_scale), _c_int(out.stride(0)), _stream()), "attention (sink, parts merged)")
         if ctx.num_requests > nd and launch_log is not None:
             _cost((T - nd) * per_row, 0.0, key_bytes, 2.0 * H * (d // maps + dv))
-            _pending_cost["rows"], _pending_cost["window"] = "prefill", window
+            _pending_cost.update(rows="prefill", window=window, chunk=chunk)
         if (ctx.num_requests > nd and use_tc_attention and tc_sink_attention_supported(d, dv, values_in_keys) and page_size >= 16
                 and (gate is None or (gate.data_ptr() % 16 == 0 and gate_stride % 8 == 0)) and out.data_ptr() % 16 == 0 and out.stride(0) % 8 == 0):
             # heads of 64 or 128: the tcgen05 kernel that plain causal attention uses takes the chunked
@@ -1451,26 +1453,26 @@ def attention_sink(q, k_cache, v_cache, out, ctx, block_table, H: int, K: int, d
                                          _ptr(_scratch_for(q.device).error), _c_int(chunk), _c_int(int(sink)), _ptr(gate),
                                          _c_int(gate_stride), _ptr(sink_logits), *more[:2], _c_float(out_scale), more[3],
                                          _c_float(pair.lam if pair is not None else 0.0), _c_float(pair.eps if pair is not None else 0.0), _stream()),
-                   "attention (sink, prefill, tensor cores)")
+                   f"attention ({what}, prefill, tensor cores)")
         elif ctx.num_requests > nd:
             wide = ctx.workspace.get("map_results", (T, H * dv), torch.float32) if pair is not None else None
             _check(lib.mb_attn_sink_prefill(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _ptr(block_table), _c_int(max_pages),
                                             _ptr(ctx.cu_tokens), _ptr(ctx.seq_lens), _c_int(nd), _c_int(ctx.num_requests - nd),
                                             _c_int(ctx.max_query_len), _c_int(K), _c_int(page_size), _c_float(scale), _c_int(window),
                                             _c_int(chunk), _c_int(int(sink)), _ptr(gate), _c_int(gate_stride), _ptr(sink_logits), *more, _ptr(wide), _stream()),
-                   "attention (sink, prefill)")
+                   f"attention ({what}, prefill)")
             if pair is not None:
                 pair_combine(wide, pair, out_scale, out, H // 2, dv, nd)      # (requests with one token each come first: token nd is the portions' first)
         return
     wide = ctx.workspace.get("map_results", (T, H * dv), torch.float32) if pair is not None else None
     if launch_log is not None:
         _cost(T * per_row, 0.0, key_bytes, 2.0 * H * (d // maps + dv))
-        _pending_cost["rows"], _pending_cost["window"] = "all", window
+        _pending_cost.update(rows="all", window=window, chunk=chunk)
     _check(_lib("mb_attention_sink").mb_attention_sink(
         _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(out), _code(q), _ptr(block_table), _c_int(block_table.shape[1]), _ptr(ctx.req_index),
         _ptr(ctx.positions), _c_int(T), _c_int(H), _c_int(K), _c_int(d), _c_int(dv), _c_int(page_size), _c_float(scale), _c_int(window),
         _c_int(chunk), _c_int(int(sink)), _ptr(sink_logits), _c_int(v_stride), _ptr(gate), _c_int(gate_stride), *more, _ptr(wide), _stream()),
-        "attention (sink)")
+        f"attention ({what})")
     if pair is not None:
         pair_combine(wide, pair, out_scale, out, H // 2, dv)
 

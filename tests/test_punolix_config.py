@@ -181,3 +181,18 @@ def test_value_slices_of_the_chunked_recurrence(dv, slice_):
 
     assert ops._gla_slice(dv) == slice_ and dv % slice_ == 0
     assert math.isclose(ops.gla_chunk_bytes(64, dv), 4 * (64 * 64 + 64 * dv))
+
+
+@pytest.mark.parametrize("window,chunk", [(0, 0), (5, 0), (0, 7), (3, 7)])
+def test_keys_and_pairs_counted_for_a_step(window, chunk):
+    """What a stage table divides by: keys read and (query, key) pairs under every mask."""
+    from marin_b200.engine.profile import lengths_of
+
+    def sees(i, j):
+        return j <= i and (not window or i - j < window) and (not chunk or i // chunk == j // chunk)
+
+    spans = [(9, 1), (13, 1), (0, 20), (6, 3)]
+    for which, some in (("decode", spans[:2]), ("prefill", spans[2:]), ("all", spans)):
+        pairs = sum(sees(i, j) for before, n in some for i in range(before, before + n) for j in range(i + 1))
+        keys = sum(any(sees(i, j) for i in range(before, before + n)) for before, n in some for j in range(before + n))
+        assert lengths_of(spans, window, chunk)[which] == [keys, pairs]

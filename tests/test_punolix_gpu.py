@@ -142,7 +142,7 @@ def test_one_key_stands_out_in_one_map(dtype, which, dim, vdim, at):
         close(got[-40:], want[-40:], dtype, f"at {at}, cuts {cuts[:3]}")
 
 
-@pytest.mark.parametrize("m", [_diff(4, 2, 32, 64, 0.3, _rot(32, 5000.0), 0.3, softcap=12.0), _diff(2, 1, 64, 128, 0.2, _rot(64, 5000.0), 0.5),
+@pytest.mark.parametrize("m", [_diff(6, 3, 32, 64, 0.3, _rot(32, 5000.0), 0.3, softcap=12.0), _diff(2, 1, 64, 128, 0.2, _rot(64, 5000.0), 0.5),
                                _diff(3, 1, 24, 48, 0.3, _rot(24, 5000.0), 0.2, softcap=9.0)], ids=label)
 def test_long_sequences_split_their_keys_over_blocks_of_work(m):
     """Single tokens of a long sequence: the keys are split over several CTAs, both maps' parts merged and combined; and a prompt of many tiles."""
@@ -359,7 +359,7 @@ def test_a_layer_alone(dtype, kind, join, monkeypatch):
 
     monkeypatch.setattr(ParallelBlock, "join_products", join)
     hidden, T, mult = 64, 130, 0.3
-    raw = {"attention": _layer("attention", _diff(4, 2, 32, 64, 0.2, _rot(32, 700.0), 0.5, softcap=9.0), 96),
+    raw = {"attention": _layer("attention", _diff(6, 3, 32, 64, 0.2, _rot(32, 700.0), 0.5, softcap=9.0), 96),
            "parallel": _layer("parallel", _parallel(_left(4, 2, 32, 48, 0.2, _rot(32, 700.0), conv=4, chunk=40), _right(3, 32, 48, 8.0), 0.4, -1.3), 80),
            "odd": _layer("parallel", _parallel(_left(3, 1, 12, 10, 0.3, _rot(8, 700.0), conv=3, chunk=40), _right(3, 6, 9, 8.0), 0.4, -1.3), 52),
            "alone": _layer("parallel", _parallel(_left(4, 2, 32, 48, 0.2, _rot(32, 700.0), conv=2), _right(3, 32, 48, 8.0), 0.9, 0.6), None)}[kind]
